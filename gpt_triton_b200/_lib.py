@@ -17,6 +17,18 @@ _TORCH_TO_CODE = {torch.float32: F32, torch.float16: F16, torch.bfloat16: BF16}
 c_i64, c_int, c_float, c_void_p, c_size_t = ctypes.c_int64, ctypes.c_int, ctypes.c_float, ctypes.c_void_p, ctypes.c_size_t
 _p_i64 = ctypes.POINTER(ctypes.c_int64)
 
+
+
+class LinearArgs(ctypes.Structure):
+    """b200_linear_args of include/b200_gpt.h, field for field."""
+
+    _fields_ = [("a", c_void_p), ("b", c_void_p), ("M", c_i64), ("N", c_i64), ("K", c_i64), ("lda", c_i64), ("ldb", c_i64),
+                ("row_sumsq", c_void_p), ("row_sumsq_ld", c_i64), ("row_sumsq_cols", c_i64), ("out", c_void_p), ("ld_out", c_i64),
+                ("act_split", c_i64), ("x", c_void_p), ("ld_x", c_i64), ("gain", c_void_p), ("gx", c_void_p), ("ld_gx", c_i64),
+                ("sumsq_out", c_void_p), ("sumsq_out_ld", c_i64), ("status_word", c_void_p), ("op_dtype", c_int), ("out_dtype", c_int),
+                ("row_sumsq_slices", c_int), ("act_lo", c_int), ("act_hi", c_int), ("eps", c_float), ("out_scale", c_float)]
+
+
 # name -> (restype, argtypes); must list every function include/b200_gpt.h declares
 SIGNATURES = {
     "b200_status_string": (ctypes.c_char_p, [c_int]),
@@ -46,6 +58,19 @@ SIGNATURES = {
     "b200_attention_decode": (c_int, [c_void_p, c_void_p, c_void_p, c_i64, c_i64, c_i64, c_i64, c_float, c_int, c_void_p, c_void_p, c_void_p]),
     "b200_decode_append": (c_int, [c_void_p, c_void_p, c_i64, c_i64, c_i64, c_void_p, c_int, c_void_p, c_void_p, c_void_p]),
     "b200_sample_logits": (c_int, [c_void_p, c_i64, c_i64, c_i64, c_int, c_float, c_int, ctypes.c_uint64, c_void_p, c_void_p, c_void_p]),
+    "b200_linear_slice_cols": (c_i64, [c_i64, c_int]),
+    "b200_linear": (c_int, [ctypes.POINTER(LinearArgs), c_void_p]),
+    "b200_embedding_rms": (c_int, [c_void_p] * 6 + [c_i64] * 4 + [c_int, c_void_p]),
+    "b200_latent_append": (c_int, [c_void_p, c_i64, c_void_p, c_float, c_void_p, c_void_p] + [c_i64] * 6 + [c_void_p, c_int, c_void_p]),
+    "b200_latent_gather": (c_int, [c_void_p, c_void_p] + [c_i64] * 6 + [c_int, c_void_p]),
+    "b200_window_attention": (c_int, [c_void_p, c_i64] * 4 + [c_i64] * 7 + [c_float, c_void_p, c_int, c_void_p, c_void_p]),
+    "b200_latent_decode_workspace_bytes": (c_size_t, [c_i64] * 4 + [c_int]),
+    "b200_latent_decode": (c_int, [c_void_p, c_i64, c_void_p, c_void_p, c_void_p, c_void_p] + [c_i64] * 8 + [c_float, c_void_p, c_int, c_void_p, c_void_p,
+                                                                                                        c_size_t, c_void_p]),
+    "b200_decayed_attention_slices": (c_i64, [c_i64] * 4 + [c_int]),
+    "b200_decayed_attention_workspace_bytes": (c_size_t, [c_i64] * 5 + [c_int]),
+    "b200_decayed_attention": (c_int, [c_void_p] + [c_i64] * 4 + [c_void_p] * 3 + [c_int, c_void_p, c_i64, c_void_p] + [c_i64] * 6
+                               + [c_int, c_void_p, c_size_t, c_void_p, c_void_p]),
     "b200_selftest_bounded_wait": (c_int, [c_void_p, c_i64, c_void_p]),
 }
 

@@ -36,7 +36,7 @@ const char* b200_status_string(int status) {
 
 const char* b200_last_cuda_error(void) { return cudaGetErrorString(g_last_cuda); }
 
-int b200_abi_version(void) { return 6; }
+int b200_abi_version(void) { return 7; }
 
 uint64_t b200_launch_count(void) { return b200::launches_so_far(); }
 
@@ -229,6 +229,101 @@ int b200_attention(const void* q, const void* k, const void* v, void* out, int64
   if (!q || !k || !v || !out || !q_strides || !k_strides || !v_strides || !o_strides) return B200_ERR_BAD_ARGUMENT;
   return note(b200::launch_attention(q, k, v, out, B, NH, L, D, q_strides, k_strides, v_strides, o_strides, scale, in_dtype,
                                      out_dtype, status_word, (cudaStream_t)stream));
+}
+
+// ------------------------------------------------------------------ decoders with RMS norms and an fp32 residual stream
+namespace {
+bool model_dtype(int dt) { return dt == B200_BF16 || dt == B200_F32; }
+}  // namespace
+
+int64_t b200_linear_slice_cols(int64_t M, int op_dtype) { return op_dtype == B200_F32 ? b200::linear_f32_slice_cols() : b200::linear_sm100_slice_cols(M); }
+
+int b200_linear(const b200_linear_args* args, void* stream) {
+  if (!args) return B200_ERR_BAD_ARGUMENT;
+  const b200_linear_args& p = *args;
+  if (p.M < 0 || p.N < 0 || p.K < 1 || p.M > kMaxExtent || p.N > kMaxExtent || p.K > kMaxExtent || !valid_dtype(p.op_dtype)) return B200_ERR_BAD_ARGUMENT;
+  if (p.M == 0 || p.N == 0) return B200_OK;
+  if (!p.a || !p.b || p.lda < p.K || p.ldb < p.K || (p.x == nullptr) == (p.out == nullptr)) return B200_ERR_BAD_ARGUMENT;
+  if (p.out && p.ld_out < p.N) return B200_ERR_BAD_ARGUMENT;
+  if (p.x && (p.ld_x < p.N || (p.gain && (!p.gx || p.ld_gx < p.N || !p.sumsq_out || p.sumsq_out_ld < p.M)))) return B200_ERR_BAD_ARGUMENT;
+  if (p.row_sumsq && (p.row_sumsq_slices < 1 || p.row_sumsq_cols < 1 || p.row_sumsq_ld < p.M)) return B200_ERR_BAD_ARGUMENT;
+  if (p.act_lo < 0 || p.act_lo > B200_ACT_GELU_TANH || p.act_hi < 0 || p.act_hi > B200_ACT_GELU_TANH) return B200_ERR_BAD_ARGUMENT;
+  return note(p.op_dtype == B200_F32 ? b200::launch_linear_f32(p, (cudaStream_t)stream) : b200::launch_linear_sm100(p, (cudaStream_t)stream));
+}
+
+int b200_embedding_rms(const int64_t* ids, const void* table, const float* gain, float* x, void* gx, float* sumsq, int64_t T, int64_t V, int64_t W,
+                       int64_t ld_gx, int dtype, void* stream) {
+  if (T < 0 || V < 1 || W < 1 || ld_gx < W || !model_dtype(dtype)) return B200_ERR_BAD_ARGUMENT;
+  if (T == 0) return B200_OK;
+  if (!ids || !table || !gain || !x || !gx || !sumsq) return B200_ERR_BAD_ARGUMENT;
+  return note(b200::launch_embedding_rms(ids, table, gain, x, gx, sumsq, T, V, W, ld_gx, dtype, (cudaStream_t)stream));
+}
+
+int b200_latent_append(const void* raw, int64_t ld_raw, const float* weight, float eps, void* work, void* cache, int64_t B, int64_t T, int64_t R,
+                       int64_t hist, int64_t ring, int64_t start, const int32_t* pos_dev, int dtype, void* stream) {
+  if (B < 0 || T < 0 || R < 1 || ld_raw < R || hist < 0 || start < 0 || (cache && ring < 1) || !model_dtype(dtype)) return B200_ERR_BAD_ARGUMENT;
+  if (B == 0 || T == 0) return B200_OK;
+  if (!raw || !weight || (!work && !cache)) return B200_ERR_BAD_ARGUMENT;
+  return note(b200::launch_latent_append(raw, ld_raw, weight, eps, work, cache, B, T, R, hist, ring < 1 ? 1 : ring, start, pos_dev, dtype, (cudaStream_t)stream));
+}
+
+int b200_latent_gather(const void* cache, void* work, int64_t B, int64_t T, int64_t R, int64_t hist, int64_t ring, int64_t start, int dtype, void* stream) {
+  if (B < 0 || T < 0 || R < 1 || hist < 0 || ring < 1 || hist > ring || start < hist || !model_dtype(dtype)) return B200_ERR_BAD_ARGUMENT;
+  if (B == 0 || hist == 0) return B200_OK;
+  if (!cache || !work) return B200_ERR_BAD_ARGUMENT;
+  return note(b200::launch_latent_gather(cache, work, B, T, R, hist, ring, start, dtype, (cudaStream_t)stream));
+}
+
+int b200_window_attention(const void* q, int64_t ld_q, const void* k, int64_t ld_k, const void* v, int64_t ld_v, void* out, int64_t ld_out, int64_t B,
+                          int64_t T, int64_t hist, int64_t heads, int64_t dim, int64_t vdim, int64_t window, float scale, const float* sink, int dtype,
+                          int* status_word, void* stream) {
+  if (B < 0 || T < 0 || hist < 0 || heads < 1 || dim < 1 || vdim < 1 || window < 1 || !model_dtype(dtype)) return B200_ERR_BAD_ARGUMENT;
+  if (ld_q < heads * dim || ld_k < heads * dim || ld_v < heads * vdim || ld_out < heads * vdim || hist + T > kMaxExtent) return B200_ERR_BAD_ARGUMENT;
+  if (B == 0 || T == 0) return B200_OK;
+  if (!q || !k || !v || !out) return B200_ERR_BAD_ARGUMENT;
+  return note(b200::launch_window_attention(q, ld_q, k, ld_k, v, ld_v, out, ld_out, B, T, hist, heads, dim, vdim, window, scale, sink, dtype, status_word,
+                                            (cudaStream_t)stream));
+}
+
+size_t b200_latent_decode_workspace_bytes(int64_t B, int64_t heads, int64_t R, int64_t window, int dtype) {
+  if (B < 1 || heads < 1 || R < 1 || window < 1) return 0;
+  return b200::latent_decode_workspace_bytes(B, heads, R, window, dtype);
+}
+
+int b200_latent_decode(const void* q, int64_t ld_q, const void* w_uk, const void* w_uv, const void* cache, void* out, int64_t ld_out, int64_t B,
+                       int64_t heads, int64_t dim, int64_t vdim, int64_t R, int64_t ring, int64_t window, float scale, const float* sink, int dtype,
+                       const int32_t* pos_dev, void* workspace, size_t workspace_bytes, void* stream) {
+  if (B < 0 || heads < 1 || dim < 1 || vdim < 1 || R < 1 || window < 1 || ring < window || !model_dtype(dtype)) return B200_ERR_BAD_ARGUMENT;
+  if (ld_q < heads * dim || ld_out < heads * vdim) return B200_ERR_BAD_ARGUMENT;
+  if (B == 0) return B200_OK;
+  if (!q || !w_uk || !w_uv || !cache || !out || !pos_dev) return B200_ERR_BAD_ARGUMENT;
+  if (!workspace || workspace_bytes < b200_latent_decode_workspace_bytes(B, heads, R, window, dtype) || (reinterpret_cast<uintptr_t>(workspace) & 255))
+    return B200_ERR_WORKSPACE;
+  return note(b200::launch_latent_decode(q, ld_q, w_uk, w_uv, cache, out, ld_out, B, heads, dim, vdim, R, ring, window, scale, sink, dtype, pos_dev, workspace,
+                                         (cudaStream_t)stream));
+}
+
+int64_t b200_decayed_attention_slices(int64_t T, int64_t heads, int64_t dim, int64_t vdim, int dtype) {
+  return b200::decayed_attention_slices(T, heads, dim, vdim, dtype);
+}
+
+size_t b200_decayed_attention_workspace_bytes(int64_t B, int64_t T, int64_t heads, int64_t dim, int64_t vdim, int dtype) {
+  if (B < 1 || T < 1 || heads < 1 || dim < 1 || vdim < 1) return 0;
+  return b200::decayed_attention_workspace_bytes(B, T, heads, dim, vdim, dtype);
+}
+
+int b200_decayed_attention(const void* qkvg, int64_t ld, int64_t off_k, int64_t off_v, int64_t off_g, const double* decay, const float* weight, float* state,
+                           int fresh, void* y, int64_t ld_y, float* sumsq, int64_t ld_sumsq, int64_t B, int64_t T, int64_t heads, int64_t dim, int64_t vdim,
+                           int dtype, void* workspace, size_t workspace_bytes, int* status_word, void* stream) {
+  if (B < 0 || T < 0 || heads < 1 || dim < 1 || vdim < 1 || !model_dtype(dtype)) return B200_ERR_BAD_ARGUMENT;
+  if (off_k < heads * dim || off_v < off_k + heads * dim || off_g < off_v + heads * vdim || ld < off_g + heads * vdim || ld_y < heads * vdim)
+    return B200_ERR_BAD_ARGUMENT;
+  if (B == 0 || T == 0) return B200_OK;
+  if (!qkvg || !decay || !weight || !state || !y || !sumsq || ld_sumsq < B * T) return B200_ERR_BAD_ARGUMENT;
+  const size_t need = b200_decayed_attention_workspace_bytes(B, T, heads, dim, vdim, dtype);
+  if (need && (!workspace || workspace_bytes < need || (reinterpret_cast<uintptr_t>(workspace) & 255))) return B200_ERR_WORKSPACE;
+  return note(b200::launch_decayed_attention(qkvg, ld, off_k, off_v, off_g, decay, weight, state, fresh, y, ld_y, sumsq, ld_sumsq, B, T, heads, dim, vdim,
+                                             dtype, workspace, status_word, (cudaStream_t)stream));
 }
 
 int b200_selftest_bounded_wait(int* status_word, int64_t limit_cycles, void* stream) {

@@ -251,6 +251,30 @@ int launch_attention(const void* q, const void* k, const void* v, void* out, int
                      int64_t D, const int64_t* q_strides, const int64_t* k_strides, const int64_t* v_strides,
                      const int64_t* o_strides, float scale, int in_dtype, int out_dtype, int* status_word, cudaStream_t stream);
 
+// Decoders with RMS norms and an fp32 residual stream; see include/b200_gpt.h for the arguments.
+int64_t linear_sm100_slice_cols(int64_t M);
+int64_t linear_f32_slice_cols();
+int launch_linear_sm100(const b200_linear_args& p, cudaStream_t stream);
+int launch_linear_f32(const b200_linear_args& p, cudaStream_t stream);
+int launch_embedding_rms(const int64_t* ids, const void* table, const float* gain, float* x, void* gx, float* sumsq, int64_t T, int64_t V, int64_t W,
+                         int64_t ld_gx, int dtype, cudaStream_t stream);
+int launch_latent_append(const void* raw, int64_t ld_raw, const float* weight, float eps, void* work, void* cache, int64_t B, int64_t T, int64_t R,
+                         int64_t hist, int64_t ring, int64_t start, const int* pos_dev, int dtype, cudaStream_t stream);
+int launch_latent_gather(const void* cache, void* work, int64_t B, int64_t T, int64_t R, int64_t hist, int64_t ring, int64_t start, int dtype,
+                         cudaStream_t stream);
+int launch_window_attention(const void* q, int64_t ld_q, const void* k, int64_t ld_k, const void* v, int64_t ld_v, void* out, int64_t ld_out,
+                            int64_t B, int64_t T, int64_t hist, int64_t heads, int64_t dim, int64_t vdim, int64_t window, float scale,
+                            const float* sink, int dtype, int* status_word, cudaStream_t stream);
+size_t latent_decode_workspace_bytes(int64_t B, int64_t heads, int64_t R, int64_t window, int dtype);
+int launch_latent_decode(const void* q, int64_t ld_q, const void* w_uk, const void* w_uv, const void* cache, void* out, int64_t ld_out, int64_t B,
+                         int64_t heads, int64_t dim, int64_t vdim, int64_t R, int64_t ring, int64_t window, float scale, const float* sink,
+                         int dtype, const int* pos_dev, void* workspace, cudaStream_t stream);
+int64_t decayed_attention_slices(int64_t T, int64_t heads, int64_t dim, int64_t vdim, int dtype);
+size_t decayed_attention_workspace_bytes(int64_t B, int64_t T, int64_t heads, int64_t dim, int64_t vdim, int dtype);
+int launch_decayed_attention(const void* qkvg, int64_t ld, int64_t off_k, int64_t off_v, int64_t off_g, const double* decay, const float* weight,
+                             float* state, int fresh, void* y, int64_t ld_y, float* sumsq, int64_t ld_sumsq, int64_t B, int64_t T, int64_t heads,
+                             int64_t dim, int64_t vdim, int dtype, void* workspace, int* status_word, cudaStream_t stream);
+
 // One warp waiting (bounded) on a barrier that nothing completes: reports B200_ERR_DEVICE_WAIT through status_word.
 int launch_bounded_wait_selftest(int* status_word, int64_t limit_cycles, cudaStream_t stream);
 // tcgen05/TMA attention (head size 64, fp16); B200_ERR_UNSUPPORTED means "use the generic kernel".

@@ -199,6 +199,61 @@ int launch_row_ln_stats(const void* x, float* ln_stats, void* ln_ext, int64_t M,
   return status_from_cuda(e);
 }
 
+// ------------------------------------------------------------------ start of an fp32 residual stream
+// x = table[id] in fp32, gx = gain * x in the operand type and the row's sum of squares (the deferred RMS norm of the
+// first layer).  One warp per token.
+template <typename T, bool VEC>
+__global__ void __launch_bounds__(kWarpsPerBlock * 32)
+embedding_rms_kernel(const int64_t* __restrict__ ids, const T* __restrict__ table, const float* __restrict__ gain, float* __restrict__ x,
+                     T* __restrict__ gx, float* __restrict__ sumsq, int64_t rows, int64_t V, int64_t W, int64_t ld_gx) {
+  const int lane = threadIdx.x & 31;
+  const int64_t stride = (int64_t)gridDim.x * kWarpsPerBlock;
+  for (int64_t t = (int64_t)blockIdx.x * kWarpsPerBlock + (threadIdx.x >> 5); t < rows; t += stride) {
+    const int64_t id = ids[t];
+    const bool ok = id >= 0 && id < V;
+    const T* e = table + (ok ? id : 0) * W;
+    float sq = 0.f;
+    if (VEC) {
+      for (int64_t c = (int64_t)lane * 8; c < W; c += 256) {
+        float f[8], g[8];
+        load8(e + c, f);
+        load8(gain + c, g);
+#pragma unroll
+        for (int i = 0; i < 8; ++i) f[i] = ok ? f[i] : 0.f, sq = fmaf(f[i], f[i], sq), g[i] *= f[i];
+        store8(x + t * W + c, f);
+        store8(gx + t * ld_gx + c, g);
+      }
+    } else {
+      for (int64_t c = lane; c < W; c += 32) {
+        const float f = ok ? to_float(e[c]) : 0.f;
+        sq = fmaf(f, f, sq);
+        x[t * W + c] = f;
+        gx[t * ld_gx + c] = from_float<T>(f * gain[c]);
+      }
+    }
+    sq = warp_sum(sq);
+    if (lane == 0) sumsq[t] = sq;
+  }
+}
+
+template <typename T>
+static int embedding_rms_typed(const int64_t* ids, const void* table, const float* gain, float* x, void* gx, float* sumsq, int64_t rows, int64_t V,
+                               int64_t W, int64_t ld_gx, cudaStream_t stream) {
+  const bool vec = W % 8 == 0 && ld_gx % 8 == 0 &&
+                   ((reinterpret_cast<uintptr_t>(table) | reinterpret_cast<uintptr_t>(gain) | reinterpret_cast<uintptr_t>(x) | reinterpret_cast<uintptr_t>(gx)) & 15) == 0;
+  const unsigned grid = row_grid(rows);
+  if (vec) embedding_rms_kernel<T, true><<<grid, kWarpsPerBlock * 32, 0, stream>>>(ids, (const T*)table, gain, x, (T*)gx, sumsq, rows, V, W, ld_gx);
+  else embedding_rms_kernel<T, false><<<grid, kWarpsPerBlock * 32, 0, stream>>>(ids, (const T*)table, gain, x, (T*)gx, sumsq, rows, V, W, ld_gx);
+  note_launches(1);
+  return status_from_cuda(cudaGetLastError());
+}
+
+int launch_embedding_rms(const int64_t* ids, const void* table, const float* gain, float* x, void* gx, float* sumsq, int64_t rows, int64_t V, int64_t W,
+                         int64_t ld_gx, int dtype, cudaStream_t stream) {
+  return dtype == B200_BF16 ? embedding_rms_typed<__nv_bfloat16>(ids, table, gain, x, gx, sumsq, rows, V, W, ld_gx, stream)
+                            : embedding_rms_typed<float>(ids, table, gain, x, gx, sumsq, rows, V, W, ld_gx, stream);
+}
+
 // ------------------------------------------------------------------ LayerNorm
 // Register-resident row: each lane holds NV vectors of 8 elements (row read from HBM once,
 // written once).  Statistics in fp32: mean, then the centred sum of squares (two passes over

@@ -30,6 +30,8 @@ import torch
 from torch import nn
 
 from . import kernels as K
+from .generation import GeneratesTokens, GenerationSession  # noqa: F401  (GenerationSession: part of this module's surface)
+from .module_base import _EvalOnly, _OperandCache
 
 GPU_TO_FLOPS = {"v100": 130e12, "a100": 312e12, "h100": 989e12, "b200": 2250e12}
 GPU_TO_FLOPS = {k: int(v) for k, v in GPU_TO_FLOPS.items()}
@@ -52,58 +54,6 @@ def _linear_flops(tokens, fan_in, fan_out):
 
 def _ln_flops(tokens, h):
     return 2 * tokens * h
-
-
-class _OperandCache:
-    """Derived operands (PackedWeight and friends) per parameter; rebuilt when the parameter is replaced, cast,
-    moved or written in place.  The tag uses the Parameter's own ``_version``, which ``load_state_dict``,
-    ``param.copy_`` and optimizer steps bump (``param.data`` is a fresh tensor object whose counter always reads 0,
-    so it cannot serve).  Writes made *through* ``param.data`` (``param.data.mul_(2)``) bump no counter torch
-    exposes: after such a write call ``refresh_operands()`` on the model."""
-
-    def __init__(self):
-        self._slots = {}
-
-    def clear(self):
-        self._slots.clear()
-
-    @staticmethod
-    def _tag(param):
-        return (param.data_ptr(), param._version, param.dtype, param.device, tuple(param.shape))
-
-    def derived(self, key, params, make):
-        """`make()` cached under `key` until one of `params` changes."""
-        tag = tuple(self._tag(p) for p in params)
-        slot = self._slots.get(key)
-        if slot is None or slot[0] != tag:
-            slot = (tag, make())
-            self._slots[key] = slot
-        return slot[1]
-
-    def __call__(self, param, weight_is_nk=False):
-        return self.derived(("packed", id(param), weight_is_nk), (param,),
-                            lambda: K.pack_weight(param.data.contiguous(), weight_is_nk=weight_is_nk))
-
-    def folded(self, weight, ln_weight, ln_bias, bias):
-        """FoldedWeight of `weight` with the LayerNorm (ln_weight, ln_bias) in front of it and `bias` behind."""
-        return self.derived(("folded", id(weight)), (weight, ln_weight, ln_bias, bias),
-                            lambda: K.fold_layer_norm(weight.data.contiguous(), ln_weight.data.contiguous(), ln_bias.data.contiguous(),
-                                                      bias.data.contiguous()))
-
-
-class _EvalOnly(nn.Module):
-    def _check_eval(self):
-        if self.training:
-            raise NotImplementedError("libb200gpt implements the forward/eval path only: call .eval() first")
-
-    def refresh_operands(self):
-        """Drop every cached derived operand (packed weights) of this module and its children; the next forward
-        rebuilds them from the parameters.  Needed only after writes through ``param.data``, which torch's version
-        counters do not see; ``load_state_dict``, ``copy_``, casts and moves are noticed without it."""
-        for m in self.modules():
-            cache = getattr(m, "_operand", None)
-            if isinstance(cache, _OperandCache):
-                cache.clear()
 
 
 class FusedAttention(_EvalOnly):
@@ -206,7 +156,8 @@ class GPTConfig:
     dropout: float = 0.1
 
 
-class FusedGPT(_EvalOnly):
+class FusedGPT(GeneratesTokens, _EvalOnly):
+    exact_float32 = False  # fp32 storage still rounds the operands of its products to fp16, as the reference does
     # Fold the LayerNorms of the blocks into the GEMMs behind them (16-bit models; see the module docstring).  The
     # environment variable B200GPT_FOLD_LAYERNORM=0 changes the default for the process; the attribute can also be set
     # per model.
@@ -283,25 +234,47 @@ class FusedGPT(_EvalOnly):
             return logits.argmax(dim=-1)
         return K.sample_logits(logits, temperature=temperature, top_k=top_k, seed=seed, step=pos)
 
-    @torch.no_grad()
-    def generate(self, ids, max_new_tokens, temperature=0.0, top_k=0, seed=0, use_cuda_graph=True):
-        """ids (batch, prompt_len) -> (batch, max_new_tokens) int64 continuation, one token per step with a key/value
-        cache (the inference loop the reference's README.md:55 lists as not built).  temperature 0: greedy; > 0:
-        draws from softmax(logits / temperature) over the top_k largest logits (0 = all), reproducible for a given
-        seed.  The sessions (cache, captured decode step) are kept on the model per
-        (batch, capacity, temperature, top_k, seed) and re-used by later calls of the same shape."""
-        B, L0 = ids.shape
-        need = L0 + max_new_tokens - 1
-        key = (B, temperature, top_k, seed, use_cuda_graph, self.wte_weight.dtype, self.wte_weight.device)
-        sessions = self.__dict__.setdefault("_sessions", {})
-        session = sessions.get(key)
-        if session is None or session.capacity < need or session.tokens.shape[1] < max_new_tokens or session.stale():
-            sessions.pop(key, None)
-            while len(sessions) >= 4:  # every session holds a cache: keep a few
-                sessions.pop(next(iter(sessions)))
-            sessions[key] = session = GenerationSession(self, B, capacity=need, max_new_tokens=max_new_tokens, temperature=temperature,
-                                                        top_k=top_k, seed=seed, use_cuda_graph=use_cuda_graph)
-        return session.generate(ids, max_new_tokens)
+    # ---- what GenerationSession drives (generation.py)
+    def vocab_size(self):
+        return self.config.vocab_size
+
+    def check_capacity(self, capacity):
+        assert capacity <= self.config.block_size, f"{capacity} positions exceed the position table ({self.config.block_size} rows)"
+
+    def new_cache(self, batch, capacity):
+        """Keys and values of every layer: (batch, capacity, 2 * n_embd) each."""
+        w = self.wte_weight
+        return [torch.empty((batch, capacity, 2 * self.config.n_embd), device=w.device, dtype=w.dtype) for _ in range(self.config.n_layer)]
+
+    def prompt_pass(self, ids, cache, start, pos, want=None):
+        """ids (batch, n) of positions start .. start + n - 1 -> final hidden rows at the places `want` (int64 tensor; None:
+        the last one) of every sequence, (batch * len(want), n_embd); keys and values join the cache.  A later portion
+        (start > 0) goes through the one-token step, which reads its position from `pos`."""
+        B, n = ids.shape
+        if start == 0:
+            y = self._body(ids, kv_caches=cache)
+            y = y[:, -1:, :] if want is None else y.index_select(1, want)
+            return K.fused_layer_norm(y.reshape(-1, self.config.n_embd).contiguous(), self.layer_norm_weight.data, self.layer_norm_bias.data)
+        places = {n - 1} if want is None else set(want.tolist())
+        kept = {}
+        for t in range(n):
+            pos[:1].fill_(start + t)
+            row = self.decode_pass(ids[:, t].contiguous(), cache, pos)
+            if t in places:
+                kept[t] = row
+        order = [n - 1] if want is None else want.tolist()
+        return torch.stack([kept[t] for t in order], dim=1).reshape(B * len(order), -1)
+
+    def decode_pass(self, ids, cache, pos):
+        """ids (batch,) of the tokens at position pos[0] -> final hidden rows (batch, n_embd)."""
+        return self._decode_body(ids, cache, pos)
+
+    def pick(self, hidden, temperature, top_k, seed, pos):
+        return self._pick(hidden, temperature, top_k, seed, pos)
+
+    def head_logits(self, hidden):
+        """Final hidden rows -> logits (rows, vocab)."""
+        return self.lm_head(hidden.view(1, *hidden.shape))[0]
 
     @torch.no_grad()
     def lm_head(self, hidden, return_argmax=False, return_lse=False):
@@ -413,78 +386,6 @@ class GraphedForward:
         self.static_ids.copy_(ids)
         self.graph.replay()
         return self.outputs
-
-
-class GenerationSession:
-    """Token-by-token generation for a fixed batch size: the key/value cache of every layer
-    ((batch, capacity, 2 * n_embd) each), the device-side position counter and, after the first two decode steps,
-    a CUDA graph of one decode step that is replayed for every further token of this and later generations (any
-    prompt length: the position lives in device memory).  Prompt + generated tokens - 1 must fit both `capacity`
-    and the model's position table.  No counterpart in the reference (README.md:55)."""
-
-    EAGER_STEPS = 2  # decode steps run eagerly before the capture (kernel attributes, allocator pools)
-
-    def __init__(self, model, batch, capacity, max_new_tokens, temperature=0.0, top_k=0, seed=0, use_cuda_graph=True):
-        cfg = model.config
-        assert capacity <= cfg.block_size, f"{capacity} positions exceed the position table ({cfg.block_size} rows)"
-        assert temperature >= 0.0 and top_k >= 0 and max_new_tokens >= 1
-        dev, dtype = model.wte_weight.device, model.wte_weight.dtype
-        self.model, self.batch, self.capacity = model, batch, max(int(capacity), 1)
-        self.temperature, self.top_k, self.seed, self.use_cuda_graph = float(temperature), int(top_k), int(seed), use_cuda_graph
-        self.kv = [torch.empty((batch, self.capacity, 2 * cfg.n_embd), device=dev, dtype=dtype) for _ in range(cfg.n_layer)]
-        self.pos = torch.zeros(2, device=dev, dtype=torch.int32)  # {tokens in the cache, prompt length}
-        self.tokens = torch.zeros((batch, max_new_tokens), device=dev, dtype=torch.int64)
-        self.feedback = torch.zeros((batch,), device=dev, dtype=torch.int64)  # the ids the next decode step embeds
-        self.graph = None
-        self._sig = self._signature()
-
-    def _signature(self):
-        return tuple(_OperandCache._tag(p) for p in self.model.parameters())
-
-    def stale(self):
-        """True once a parameter has been reloaded, cast or moved: a captured step holds the old operands."""
-        return self._signature() != self._sig
-
-    def _step(self):
-        m = self.model
-        hidden = m._decode_body(self.feedback, self.kv, self.pos)
-        ids = m._pick(hidden, self.temperature, self.top_k, self.seed, self.pos)
-        K.decode_append(ids, self.tokens, self.pos, advance=True, feedback=self.feedback)
-
-    @torch.no_grad()
-    def generate(self, ids, max_new_tokens):
-        m = self.model
-        B, L0 = ids.shape
-        assert B == self.batch and L0 >= 1 and 1 <= max_new_tokens <= self.tokens.shape[1]
-        assert L0 + max_new_tokens - 1 <= self.capacity, "prompt + generated tokens do not fit this session's cache"
-        assert not self.stale(), "the model's parameters changed: make a new session"
-        dev = self.pos.device
-        # prompt: the usual forward, its keys/values copied into the caches; next id from the last position
-        y = m._body(ids, kv_caches=self.kv)
-        last = K.fused_layer_norm(y[:, -1, :].contiguous(), m.layer_norm_weight.data, m.layer_norm_bias.data)
-        self.pos.copy_(torch.tensor([L0, L0], dtype=torch.int32), non_blocking=False)
-        first = m._pick(last, self.temperature, self.top_k, self.seed, self.pos)
-        K.decode_append(first, self.tokens, self.pos, advance=False, feedback=self.feedback)
-        steps = max_new_tokens - 1
-        done = 0
-        if self.graph is None:
-            while done < min(steps, self.EAGER_STEPS):
-                self._step()
-                done += 1
-            if self.use_cuda_graph and done < steps:
-                torch.cuda.synchronize(dev)
-                self.graph = torch.cuda.CUDAGraph()
-                with torch.cuda.graph(self.graph):
-                    self._step()
-        for _ in range(steps - done):
-            if self.graph is not None:
-                self.graph.replay()
-            else:
-                self._step()
-        code = K.device_status(dev)
-        if code:
-            raise RuntimeError(f"generation stopped by a device-side check (code {code}): cache or token buffer out of room")
-        return self.tokens[:, :max_new_tokens].clone()
 
 
 def executed_fwd_flops(config, batch, seqlen, with_lm_head=True):

@@ -604,3 +604,230 @@ def sample_logits(logits, temperature=1.0, top_k=0, seed=0, step=None, out=None)
                                             int(top_k), int(seed) & 0xFFFFFFFFFFFFFFFF, _ptr(step), ids.data_ptr(), stream_ptr(dev))
     check(st, "sample_logits")
     return ids
+
+
+# ----------------------------------------------------------------------------- RMS-normed decoders, fp32 residual stream
+# No counterpart in the reference.  bf16 runs on the tensor cores with fp32 accumulation; fp32 is true 32-bit.
+ACTIVATIONS = {None: 0, "silu": 1, "sigmoid": 2, "gelu_tanh": 3}
+
+
+def _rows_empty(M, cols, dtype, device):
+    """(M, cols) matrix whose rows start 32-byte aligned: what the wide stores and the tensor maps want."""
+    q = 64 // dtype.itemsize
+    return torch.empty((M, (cols + q - 1) // q * q), device=device, dtype=dtype)[:, :cols]
+
+
+class NormedRows:
+    """Rows behind an RMS norm that the consuming product finishes: ``data`` (M, cols) = gain * x in the operand type,
+    ``sumsq`` (slices, M) float32 = sums of x^2 per column slice; the normed row is
+    data / sqrt(sum(sumsq) / norm_cols + eps)."""
+
+    __slots__ = ("data", "sumsq", "norm_cols", "eps")
+
+    def __init__(self, data, sumsq, norm_cols, eps):
+        self.data, self.sumsq, self.norm_cols, self.eps = data, sumsq, norm_cols, eps
+
+    def select(self, index):
+        """The rows `index` (int64 tensor) of this matrix."""
+        out = _rows_empty(index.numel(), self.data.shape[1], self.data.dtype, self.data.device)
+        out.copy_(self.data.index_select(0, index))
+        return NormedRows(out, self.sumsq.index_select(1, index), self.norm_cols, self.eps)
+
+
+def operand_rows(*weights):
+    """Stack (n_i, k) weights into one K-major operand; every section starts at a multiple of 8 rows (the columns of the
+    product), zero rows in between.  Returns (operand, first row of every section)."""
+    k, dtype, dev = weights[0].shape[1], weights[0].dtype, weights[0].device
+    starts, n = [], 0
+    for w in weights:
+        assert w.shape[1] == k and w.dtype == dtype
+        starts.append(n)
+        n = (n + w.shape[0] + 7) // 8 * 8
+    n = starts[-1] + weights[-1].shape[0]
+    if len(weights) == 1 and weights[0].is_contiguous() and weights[0].data_ptr() % 16 == 0 and (k % 8 == 0 or dtype == torch.float32):
+        return weights[0], starts
+    out = torch.zeros((n, (k + 7) // 8 * 8), device=dev, dtype=dtype)[:, :k]
+    for s, w in zip(starts, weights):
+        out[s:s + w.shape[0]] = w
+    return out, starts
+
+
+def _linear_args(rows, weight):
+    normed = rows if isinstance(rows, NormedRows) else None
+    a = normed.data if normed else rows
+    require_cuda(a, weight)
+    assert a.dim() == 2 and weight.dim() == 2 and a.stride(1) == 1 and weight.stride(1) == 1
+    assert a.shape[1] == weight.shape[1] and a.dtype == weight.dtype and a.dtype in (torch.bfloat16, torch.float32)
+    dev = _same_device(a, weight)
+    p = _lib.LinearArgs()
+    p.a, p.b = a.data_ptr(), weight.data_ptr()
+    p.M, p.K = a.shape
+    p.N = weight.shape[0]
+    p.lda = max(a.stride(0), a.shape[1])
+    p.ldb = max(weight.stride(0), weight.shape[1])
+    p.op_dtype = dtype_code(a.dtype)
+    p.out_scale = 1.0
+    p.status_word = _status_ptr(dev)
+    if normed:
+        sq = normed.sumsq
+        assert sq.dtype == torch.float32 and sq.shape[1] >= p.M and (sq.stride(1) == 1 or sq.shape[1] == 1)
+        p.row_sumsq, p.row_sumsq_slices, p.row_sumsq_cols, p.eps = sq.data_ptr(), sq.shape[0], normed.norm_cols, normed.eps
+        p.row_sumsq_ld = max(sq.stride(0), sq.shape[1])
+    return p, a, dev
+
+
+@torch.no_grad()
+def embedding_rms(ids, table, gain, eps):
+    """Start of an fp32 residual stream: ids (n,) int64 -> (x (n, width) float32 = table[ids], NormedRows of x under an RMS
+    norm with weights `gain` (width,) float32)."""
+    require_cuda(ids, table, gain)
+    assert ids.dtype == torch.int64 and ids.is_contiguous() and table.is_contiguous() and gain.dtype == torch.float32 and gain.is_contiguous()
+    V, W = table.shape
+    n = ids.numel()
+    dev = _same_device(ids, table, gain)
+    assert gain.shape == (W,)
+    x = torch.empty((n, W), device=dev, dtype=torch.float32)
+    gx = _rows_empty(n, W, table.dtype, dev)
+    sumsq = torch.empty((1, n), device=dev, dtype=torch.float32)
+    with torch.cuda.device(dev):
+        st = _lib.load().b200_embedding_rms(ids.data_ptr(), table.data_ptr(), gain.data_ptr(), x.data_ptr(), gx.data_ptr(), sumsq.data_ptr(), n, V, W,
+                                            max(gx.stride(0), W), dtype_code(table.dtype), stream_ptr(dev))
+    check(st, "embedding_rms")
+    return x, NormedRows(gx, sumsq, W, eps)
+
+
+@torch.no_grad()
+def linear(rows, weight, *, act=None, act_split=None, act_after=None, out_scale=1.0, out_dtype=None):
+    """act(norm(rows) @ weight^T * out_scale): rows a NormedRows or a plain (M, K) matrix, weight (N, K).  `act` applies to
+    the output columns below `act_split` (default: all), `act_after` to the rest."""
+    p, a, dev = _linear_args(rows, weight)
+    out = _rows_empty(p.M, p.N, out_dtype or a.dtype, dev)
+    p.out, p.ld_out, p.out_dtype = out.data_ptr(), max(out.stride(0), p.N), dtype_code(out.dtype)
+    p.act_lo, p.act_hi = ACTIVATIONS[act], ACTIVATIONS[act_after]
+    p.act_split = p.N if act_split is None else act_split
+    p.out_scale = out_scale
+    with torch.cuda.device(dev):
+        check(_lib.load().b200_linear(ctypes.byref(p), stream_ptr(dev)), "linear")
+    return out
+
+
+@torch.no_grad()
+def linear_residual(rows, weight, x, gain=None, eps=0.0):
+    """x += norm(rows) @ weight^T, in place on the fp32 residual stream x (M, N).  With `gain` (N,) float32 returns the
+    NormedRows of the new x under an RMS norm with those weights."""
+    p, a, dev = _linear_args(rows, weight)
+    require_cuda(x, gain)
+    assert x.dtype == torch.float32 and x.shape == (p.M, p.N) and x.is_contiguous()
+    p.x, p.ld_x = x.data_ptr(), p.N
+    lib = _lib.load()
+    normed = None
+    if gain is not None:
+        assert gain.dtype == torch.float32 and gain.shape == (p.N,) and gain.is_contiguous()
+        gx = _rows_empty(p.M, p.N, a.dtype, dev)
+        cols = lib.b200_linear_slice_cols(p.M, p.op_dtype)
+        sumsq = torch.empty(((p.N + cols - 1) // cols, p.M), device=dev, dtype=torch.float32)
+        p.gain, p.gx, p.ld_gx, p.sumsq_out, p.sumsq_out_ld = gain.data_ptr(), gx.data_ptr(), max(gx.stride(0), p.N), sumsq.data_ptr(), p.M
+        normed = NormedRows(gx, sumsq, p.N, eps)
+    with torch.cuda.device(dev):
+        check(lib.b200_linear(ctypes.byref(p), stream_ptr(dev)), "linear_residual")
+    return normed
+
+
+# ----------------------------------------------------------------------------- latent attention
+@torch.no_grad()
+def latent_append(raw, weight, eps, batch, *, cache=None, hist=0, start=0, pos=None, keep_rows=True):
+    """RMS norm (plain `weight` (R,) float32) of the new tokens' latents raw (batch * n, R).  They join `cache` (batch, ring,
+    R) at the slots position % ring, the first position being `start`, or pos[0] on the device; with `keep_rows` the
+    result is (batch, hist + n, R): the latents of the `hist` tokens before them, from the cache, then the new ones."""
+    require_cuda(raw, weight, cache)
+    assert raw.stride(1) == 1 and weight.dtype == torch.float32 and weight.is_contiguous()
+    M, R = raw.shape
+    n = M // batch
+    dev = _same_device(raw, weight, cache)
+    ring = 0
+    if cache is not None:
+        assert cache.is_contiguous() and cache.dtype == raw.dtype and cache.shape[0] == batch and cache.shape[2] == R
+        ring = cache.shape[1]
+    work = torch.empty((batch, hist + n, R), device=dev, dtype=raw.dtype) if keep_rows else None
+    lib, dt = _lib.load(), dtype_code(raw.dtype)
+    with torch.cuda.device(dev):
+        if hist:
+            check(lib.b200_latent_gather(cache.data_ptr(), work.data_ptr(), batch, n, R, hist, ring, start, dt, stream_ptr(dev)), "latent_gather")
+        st = lib.b200_latent_append(raw.data_ptr(), max(raw.stride(0), R), weight.data_ptr(), float(eps), _ptr(work), _ptr(cache), batch, n, R, hist, ring,
+                                    start, _ptr(pos), dt, stream_ptr(dev))
+    check(st, "latent_append")
+    return work
+
+
+@torch.no_grad()
+def window_attention(q, k, v, batch, heads, dim, vdim, window, scale, sink=None):
+    """Causal sliding-window softmax attention with an optional sink (float32 (heads,), one extra exp(sink) in the
+    denominator).  q (batch * n, heads * dim); k, v (batch * m, heads * dim / vdim), m >= n: the n queries are the last n of
+    the m positions.  A query sees itself and the window - 1 positions before it."""
+    require_cuda(q, k, v, sink)
+    M, rows = q.shape[0], k.shape[0]
+    n, m = M // batch, rows // batch
+    assert q.shape[1] == k.shape[1] == heads * dim and v.shape == (rows, heads * vdim) and m >= n
+    assert q.dtype == k.dtype == v.dtype and q.stride(1) == k.stride(1) == v.stride(1) == 1
+    if sink is not None:
+        assert sink.dtype == torch.float32 and sink.numel() == heads and sink.is_contiguous()
+    dev = _same_device(q, k, v, sink)
+    out = _rows_empty(M, heads * vdim, q.dtype, dev)
+    with torch.cuda.device(dev):
+        st = _lib.load().b200_window_attention(q.data_ptr(), max(q.stride(0), heads * dim), k.data_ptr(), max(k.stride(0), heads * dim), v.data_ptr(),
+                                               max(v.stride(0), heads * vdim), out.data_ptr(), max(out.stride(0), heads * vdim), batch, n, m - n, heads, dim,
+                                               vdim, window, float(scale), _ptr(sink), dtype_code(q.dtype), _status_ptr(dev), stream_ptr(dev))
+    check(st, "window_attention")
+    return out
+
+
+@torch.no_grad()
+def latent_decode(q, w_uk, w_uv, cache, pos, heads, dim, vdim, window, scale, sink=None):
+    """One token per sequence at position pos[0] (its latent is in the cache already): window attention straight on the
+    cached latents, W_uk applied to the query and W_uv to the weighted latent.  q (batch, heads * dim), w_uk (heads * dim,
+    R), w_uv (heads * vdim, R), cache (batch, ring, R)."""
+    require_cuda(q, w_uk, w_uv, cache, pos, sink)
+    B = q.shape[0]
+    R, ring = cache.shape[2], cache.shape[1]
+    assert q.shape == (B, heads * dim) and w_uk.shape == (heads * dim, R) and w_uv.shape == (heads * vdim, R) and cache.shape[0] == B
+    assert w_uk.is_contiguous() and w_uv.is_contiguous() and cache.is_contiguous() and q.stride(1) == 1 and pos.dtype == torch.int32
+    assert q.dtype == w_uk.dtype == w_uv.dtype == cache.dtype
+    dev = _same_device(q, w_uk, w_uv, cache, pos, sink)
+    out = _rows_empty(B, heads * vdim, q.dtype, dev)
+    lib, dt = _lib.load(), dtype_code(q.dtype)
+    window = min(window, ring)
+    need = lib.b200_latent_decode_workspace_bytes(B, heads, R, window, dt)
+    ws = torch.empty((need,), device=dev, dtype=torch.uint8)
+    with torch.cuda.device(dev):
+        st = lib.b200_latent_decode(q.data_ptr(), max(q.stride(0), heads * dim), w_uk.data_ptr(), w_uv.data_ptr(), cache.data_ptr(), out.data_ptr(),
+                                    max(out.stride(0), heads * vdim), B, heads, dim, vdim, R, ring, window, float(scale), _ptr(sink), dt, pos.data_ptr(),
+                                    ws.data_ptr(), need, stream_ptr(dev))
+    check(st, "latent_decode")
+    return out
+
+
+# ----------------------------------------------------------------------------- decayed linear attention
+@torch.no_grad()
+def decayed_attention(qkvg, offsets, decay, weight, state, batch, heads, dim, vdim, eps, *, fresh=False):
+    """S <- decay * S + k v^T, o = S^T q per head over the n tokens of each sequence, then o * weight * gate as NormedRows of
+    an RMS norm over all heads * vdim columns.  qkvg (batch * n, .) holds q | k | v | gate from the columns 0 and
+    `offsets` = (k, v, gate) on; decay (heads,) float64; weight (heads * vdim,) float32; state (batch, heads, dim, vdim)
+    float32, updated in place (`fresh`: taken as zero)."""
+    require_cuda(qkvg, decay, weight, state)
+    M = qkvg.shape[0]
+    n = M // batch
+    assert qkvg.stride(1) == 1 and decay.dtype == torch.float64 and decay.numel() == heads and weight.dtype == torch.float32
+    assert state.dtype == torch.float32 and state.is_contiguous() and state.shape == (batch, heads, dim, vdim) and weight.shape == (heads * vdim,)
+    assert offsets[2] + heads * vdim <= qkvg.shape[1]
+    dev = _same_device(qkvg, decay, weight, state)
+    lib, dt = _lib.load(), dtype_code(qkvg.dtype)
+    y = _rows_empty(M, heads * vdim, qkvg.dtype, dev)
+    sumsq = torch.empty((lib.b200_decayed_attention_slices(n, heads, dim, vdim, dt), M), device=dev, dtype=torch.float32)
+    need = lib.b200_decayed_attention_workspace_bytes(batch, n, heads, dim, vdim, dt)
+    ws = torch.empty((need,), device=dev, dtype=torch.uint8) if need else None
+    with torch.cuda.device(dev):
+        st = lib.b200_decayed_attention(qkvg.data_ptr(), max(qkvg.stride(0), qkvg.shape[1]), *offsets, decay.data_ptr(), weight.data_ptr(), state.data_ptr(),
+                                        int(bool(fresh)), y.data_ptr(), max(y.stride(0), heads * vdim), sumsq.data_ptr(), M, batch, n, heads, dim, vdim, dt,
+                                        _ptr(ws), need, _status_ptr(dev), stream_ptr(dev))
+    check(st, "decayed_attention")
+    return NormedRows(y, sumsq, heads * vdim, eps)

@@ -35,7 +35,7 @@ enum {
 const char* b200_status_string(int status);
 /* cudaGetErrorString of the last failing CUDA call made by this library on this thread. */
 const char* b200_last_cuda_error(void);
-/* ABI version of this header (6); bumped when a signature changes or an entry point is added. */
+/* ABI version of this header (7); bumped when a signature changes or an entry point is added. */
 int b200_abi_version(void);
 /* Number of kernels this library has launched in this process so far (all entry points). */
 uint64_t b200_launch_count(void);
@@ -296,6 +296,110 @@ int b200_decode_append(const int64_t* next_ids, int64_t* tokens, int64_t ld_toke
  */
 int b200_sample_logits(const void* logits, int64_t ld, int64_t B, int64_t V, int dtype, float temperature, int top_k, uint64_t seed,
                        const int32_t* step_dev, int64_t* ids_out, void* stream);
+
+/*
+ * ------------------------------------------------------------------------------------------------------------------
+ * Decoders with RMS norms and a residual stream in 32-bit (no counterpart in the reference).
+ *
+ * A pre-norm RMS norm, x / sqrt(mean(x^2) + eps) * gain, is never computed as a pass of its own.  Whoever writes rows x
+ * of the fp32 residual stream also writes gx = gain * x rounded to the operand type, and, per slice of columns, the
+ * sums of squares of x; the product that consumes the normed rows multiplies gx and applies 1 / sqrt(sum / cols + eps)
+ * to the accumulator.  The rounding of gx is relative to each element, so this is as exact as rounding the normed row.
+ */
+enum { B200_ACT_NONE = 0, B200_ACT_SILU = 1, B200_ACT_SIGMOID = 2, B200_ACT_GELU_TANH = 3 };
+
+/*
+ * acc = A [M,K] . B [N,K]^T (both K-major, op_dtype B200_BF16 on the tensor cores or B200_F32 in true 32-bit), then
+ *   s[row] = out_scale / sqrt(sum_i row_sumsq[i * row_sumsq_ld + row] / row_sumsq_cols + eps)   (row_sumsq NULL: out_scale)
+ *   x == NULL:  out[row, col] = act(s[row] * acc), act = act_lo for col < act_split, act_hi from there on;
+ *   x != NULL:  x[row, col] += s[row] * acc (fp32, in place) and, if gain (fp32 [N]) is given, gx = op_dtype(gain[col] *
+ *               new x) and sumsq_out[slice * sumsq_out_ld + row] = sum of (new x)^2 over slice's columns.  A slice is
+ *               b200_linear_slice_cols(M, op_dtype) columns; the slices are added in order, so results are reproducible.
+ * bf16: A and B 16-byte aligned, lda and ldb multiples of 8.  out_dtype: op_dtype or B200_F32.
+ */
+typedef struct {
+  const void* a;
+  const void* b;
+  int64_t M, N, K, lda, ldb;
+  const float* row_sumsq;
+  int64_t row_sumsq_ld, row_sumsq_cols;
+  void* out;
+  int64_t ld_out;
+  int64_t act_split;
+  float* x;
+  int64_t ld_x;
+  const float* gain;
+  void* gx;
+  int64_t ld_gx;
+  float* sumsq_out;
+  int64_t sumsq_out_ld;
+  int* status_word;
+  int op_dtype, out_dtype, row_sumsq_slices, act_lo, act_hi;
+  float eps, out_scale;
+} b200_linear_args;
+int64_t b200_linear_slice_cols(int64_t M, int op_dtype);
+int b200_linear(const b200_linear_args* args, void* stream);
+
+/*
+ * Start of the residual stream: x[t,:] = table[ids[t],:] (fp32 [T,W]), gx[t,:] = dtype(gain * x) with pitch ld_gx, and
+ * sumsq[t] = sum of x^2 (one slice).  table [V,W] and gx of `dtype` (B200_BF16 or B200_F32).  An id outside [0,V) gives a
+ * zero row.
+ */
+int b200_embedding_rms(const int64_t* ids, const void* table, const float* gain, float* x, void* gx, float* sumsq, int64_t T, int64_t V,
+                       int64_t W, int64_t ld_gx, int dtype, void* stream);
+
+/*
+ * Latent attention: a layer remembers one normed latent vector c of R elements per token; per head keys are W_uk c and
+ * values W_uv c.  The latents of the last `ring` tokens of sequence b live in cache [B, ring, R], the token at position
+ * p in slot p % ring.
+ *
+ * b200_latent_append: c = raw / sqrt(mean(raw^2) + eps) * weight for T new tokens per sequence (raw [B*T, R], pitch
+ * ld_raw; weight fp32 [R]) goes to rows [hist, hist + T) of work [B, hist + T, R] (NULL: nowhere) and, for the last
+ * min(T, ring) tokens, to the cache.  The first new token has position start, or *pos_dev if pos_dev is not NULL.
+ * b200_latent_gather: rows [0, hist) of work = the latents of positions [start - hist, start), from the cache
+ * (hist <= ring; call it before the append that may overwrite them).
+ */
+int b200_latent_append(const void* raw, int64_t ld_raw, const float* weight, float eps, void* work, void* cache, int64_t B, int64_t T, int64_t R,
+                       int64_t hist, int64_t ring, int64_t start, const int32_t* pos_dev, int dtype, void* stream);
+int b200_latent_gather(const void* cache, void* work, int64_t B, int64_t T, int64_t R, int64_t hist, int64_t ring, int64_t start, int dtype,
+                       void* stream);
+
+/*
+ * Causal sliding-window attention with a sink over expanded keys and values: query t of sequence b (row b*T + t of q)
+ * sits at key index hist + t and sees the keys j with 0 <= hist + t - j < window, of the hist + T rows of sequence b in k
+ * and v (row b*(hist+T) + j).  weights = exp(scale * q.k) / (sum over visible keys + exp(sink[head])); sink NULL: no
+ * such term.  Head h of a row starts at column h * dim (q, k) or h * vdim (v, out); pitches in elements.  Any sizes;
+ * window < 1 is refused.
+ */
+int b200_window_attention(const void* q, int64_t ld_q, const void* k, int64_t ld_k, const void* v, int64_t ld_v, void* out, int64_t ld_out,
+                          int64_t B, int64_t T, int64_t hist, int64_t heads, int64_t dim, int64_t vdim, int64_t window, float scale,
+                          const float* sink, int dtype, int* status_word, void* stream);
+
+/*
+ * One new token per sequence (at position p = pos_dev[0], its latent already appended), without expanding keys and
+ * values: with q~ = W_uk[head]^T q the score of a cached latent is (q~ . c) * scale, and the output is W_uv[head] applied
+ * to the weighted sum of the latents.  q [B, heads*dim], w_uk [heads*dim, R], w_uv [heads*vdim, R] (row pitch R), cache
+ * [B, ring, R], out [B, heads*vdim]; sees the last min(p + 1, window) latents, window <= ring.  Workspace:
+ * b200_latent_decode_workspace_bytes(...), 256-byte aligned.
+ */
+size_t b200_latent_decode_workspace_bytes(int64_t B, int64_t heads, int64_t R, int64_t window, int dtype);
+int b200_latent_decode(const void* q, int64_t ld_q, const void* w_uk, const void* w_uv, const void* cache, void* out, int64_t ld_out, int64_t B,
+                       int64_t heads, int64_t dim, int64_t vdim, int64_t R, int64_t ring, int64_t window, float scale, const float* sink,
+                       int dtype, const int32_t* pos_dev, void* workspace, size_t workspace_bytes, void* stream);
+
+/*
+ * Decayed linear attention over T tokens per sequence: per head S <- decay * S + k v^T, o = S^T q, S [dim, vdim] fp32.
+ * q, k, v, g share one row-major buffer per token: row b*T + t of qkvg (pitch ld), sections starting at columns 0, off_k,
+ * off_v, off_g, head h at h*dim (q, k) or h*vdim (v, g).  state [B, heads, dim, vdim] fp32 is read (unless fresh != 0:
+ * zero) and updated in place.  decay: double [heads].  Outputs, ready for a product behind a deferred RMS norm over all
+ * heads*vdim columns: y = dtype(o * weight * g) (pitch ld_y; weight fp32 [heads*vdim]) and sumsq[slice * ld_sumsq + row] =
+ * sum of o^2 over the slice's columns, b200_decayed_attention_slices(...) slices.
+ */
+int64_t b200_decayed_attention_slices(int64_t T, int64_t heads, int64_t dim, int64_t vdim, int dtype);
+size_t b200_decayed_attention_workspace_bytes(int64_t B, int64_t T, int64_t heads, int64_t dim, int64_t vdim, int dtype);
+int b200_decayed_attention(const void* qkvg, int64_t ld, int64_t off_k, int64_t off_v, int64_t off_g, const double* decay, const float* weight,
+                           float* state, int fresh, void* y, int64_t ld_y, float* sumsq, int64_t ld_sumsq, int64_t B, int64_t T, int64_t heads,
+                           int64_t dim, int64_t vdim, int dtype, void* workspace, size_t workspace_bytes, int* status_word, void* stream);
 
 /*
  * Self-test of the bounded waits every tensor-core kernel of this library uses (no reference counterpart): launches
