@@ -1,4 +1,6 @@
-// Causal flash attention on the 5th-generation tensor cores, head size 64, fp16 or bf16 storage.
+// Causal flash attention on the 5th-generation tensor cores, fp16 or bf16 storage: head size 64 (template parameter WIN
+// off), or sliding-window attention with a sink, an earlier part of the sequence in front of the queries and separate
+// key/value sizes of up to 64 or up to 128 (WIN on; smaller sizes are zero-filled by the loads).
 // bf16 Q and K feed S = Q K^T as they are (exact products).  P is fp16 for both storage types, as in the
 // reference, and both operands of one MMA must have the same format, so a bf16 V tile is converted to
 // fp16 in place (exact in fp16's normal range) by the softmax warps before P V.
@@ -35,21 +37,28 @@ namespace attn100 {
 
 using namespace sm100;
 
-constexpr int D = 64;
 constexpr int BLOCK_M = 128;
 constexpr int BLOCK_N = 64;
 constexpr int KV_STAGES = 3;
-constexpr int Q_BYTES = BLOCK_M * D * 2;        // 16 KB
-constexpr int KV_TILE_BYTES = BLOCK_N * D * 2;  // 8 KB each for K and V
-constexpr int KV_STAGE_BYTES = 2 * KV_TILE_BYTES;
 constexpr int P_BYTES = BLOCK_M * BLOCK_N * 2;  // 16 KB
 constexpr int NUM_SOFTMAX_WARPS = 8;  // two threads per query row: warps w and w + 4 share a 32-row quarter, 32 keys each
 constexpr int NUM_THREADS = 32 * (2 + NUM_SOFTMAX_WARPS);
-constexpr int CTAS_PER_SM = 2;
-constexpr int TMEM_COLS = 256;  // S[2] (64 columns each) + O (64 columns); allocations are powers of two
+constexpr int TMEM_COLS = 256;  // S[2] (64 columns each) + O (64 or 128 columns); allocations are powers of two
 constexpr int CTRL_BYTES = 256;
 constexpr int XCHG_BYTES = 3 * 2 * BLOCK_M * 4;  // [slot][half][row]: block maximum / row sum of each half of a row, for its partner thread
-constexpr int SMEM_BYTES = 2 * Q_BYTES + KV_STAGES * KV_STAGE_BYTES + P_BYTES + 1024 + CTRL_BYTES + XCHG_BYTES;
+// A tile is D / 64 swizzle atoms of 64 columns (128 bytes), each [rows][64].
+template <int D>
+struct Cfg {
+  static constexpr int ATOMS = D / 64;
+  static constexpr int CTAS_PER_SM = D == 64 ? 2 : 1;
+  static constexpr int Q_ATOM_BYTES = BLOCK_M * 128;       // 16 KB
+  static constexpr int Q_BYTES = ATOMS * Q_ATOM_BYTES;
+  static constexpr int KV_ATOM_BYTES = BLOCK_N * 128;      // 8 KB
+  static constexpr int KV_TILE_BYTES = ATOMS * KV_ATOM_BYTES;  // each for K and V
+  static constexpr int KV_STAGE_BYTES = 2 * KV_TILE_BYTES;
+  static constexpr int SMEM_BYTES = 2 * Q_BYTES + KV_STAGES * KV_STAGE_BYTES + P_BYTES + 1024 + CTRL_BYTES + XCHG_BYTES;
+  static_assert(CTAS_PER_SM * (SMEM_BYTES + 1024) <= 228 * 1024, "shared memory budget");
+};
 
 struct Params {
   void* out;
@@ -59,6 +68,10 @@ struct Params {
   int out_vec32;      // output rows may be written with 32-byte stores
   int q_head_inner, k_head_inner, v_head_inner;  // tensor map dimension order is {D, head, row, batch} instead of {D, row, head, batch}
   int* status_word;
+  // sliding window (WIN): query l sits at key index hist + l and sees the `window` keys that end there; sink[head] (may
+  // be NULL) adds exp(sink) to the denominator; vdim columns of the output exist
+  int hist, window, vdim;
+  const float* sink;
 };
 
 // K-major operand, 128-byte swizzle (rows of 128 bytes, 8-row groups of 1024 bytes).
@@ -67,20 +80,20 @@ __device__ __forceinline__ uint64_t desc_kmajor(uint32_t addr) {
          ((uint64_t)2 << 61);
 }
 // MN-major operand, 128-byte swizzle: 64 contiguous MN elements per 128-byte row, 8 K-rows per 1024-byte
-// group; groups along K are `stride byte offset` apart, 64-wide MN chunks `leading byte offset` apart
-// (one chunk only here).  This is how a [keys, head_dim] V tile serves as the B operand of P V.
-__device__ __forceinline__ uint64_t desc_mnmajor(uint32_t addr) {
-  return (uint64_t)((addr & 0x3FFFF) >> 4) | ((uint64_t)(1024 >> 4) << 16) | ((uint64_t)(1024 >> 4) << 32) | ((uint64_t)1 << 46) |
+// group; groups along K are `stride byte offset` apart, 64-wide MN chunks `leading byte offset` (= one atom) apart.
+// This is how a [keys, head_dim] V tile serves as the B operand of P V.
+__device__ __forceinline__ uint64_t desc_mnmajor(uint32_t addr, int atom_bytes) {
+  return (uint64_t)((addr & 0x3FFFF) >> 4) | ((uint64_t)(atom_bytes >> 4) << 16) | ((uint64_t)(1024 >> 4) << 32) | ((uint64_t)1 << 46) |
          ((uint64_t)2 << 61);
 }
-// kind::f16 instruction descriptor: fp32 accumulator, M = 128, N = 64.
-__host__ __device__ constexpr uint32_t idesc(int a_fmt, int b_fmt, int b_mn_major) {
-  return (1u << 4) | ((uint32_t)a_fmt << 7) | ((uint32_t)b_fmt << 10) | ((uint32_t)b_mn_major << 16) | ((uint32_t)(BLOCK_N >> 3) << 17) |
+// kind::f16 instruction descriptor: fp32 accumulator, M = 128, N = n.
+__host__ __device__ constexpr uint32_t idesc(int a_fmt, int b_fmt, int b_mn_major, int n) {
+  return (1u << 4) | ((uint32_t)a_fmt << 7) | ((uint32_t)b_fmt << 10) | ((uint32_t)b_mn_major << 16) | ((uint32_t)(n >> 3) << 17) |
          ((uint32_t)(BLOCK_M >> 4) << 24);
 }
 
 struct Item {
-  int b, h, q0, q_end, nblk;
+  int b, h, q0, q_end, k0, nblk;  // k0: first key of the first block
 };
 // Query rows [0, L) are cut into n_qt = ceil(L / 128) tiles of at most 128 rows whose ENDS are as early as they can be:
 // tile i ends at min(L, round_up(L - 128 * (n_qt - 1 - i), 64)) and starts where tile i - 1 ends.  A tile costs one
@@ -93,7 +106,8 @@ __device__ __forceinline__ int tile_end(int i, int n_qt, int L) {
   const int e = (L - BLOCK_M * (n_qt - 1 - i) + BLOCK_N - 1) / BLOCK_N * BLOCK_N;
   return min(L, e);
 }
-__device__ __forceinline__ Item decode_item(int64_t idx, int bh_total, int n_qt, int NH, int L) {
+template <bool WIN>
+__device__ __forceinline__ Item decode_item(int64_t idx, int bh_total, int n_qt, int NH, int L, const Params& p) {
   const int qt = n_qt - 1 - (int)(idx / bh_total);
   const int bh = (int)(idx % bh_total);
   Item it;
@@ -101,7 +115,14 @@ __device__ __forceinline__ Item decode_item(int64_t idx, int bh_total, int n_qt,
   it.h = bh % NH;
   it.q0 = qt == 0 ? 0 : tile_end(qt - 1, n_qt, L);
   it.q_end = tile_end(qt, n_qt, L);
-  it.nblk = (it.q_end - 1) / BLOCK_N + 1;
+  if constexpr (WIN) {
+    // blocks start at the first key the tile's first query sees (a load may start at any row)
+    it.k0 = max(0, p.hist + it.q0 - p.window + 1);
+    it.nblk = (p.hist + it.q_end - it.k0 + BLOCK_N - 1) / BLOCK_N;
+  } else {
+    it.k0 = 0;
+    it.nblk = (it.q_end - 1) / BLOCK_N + 1;
+  }
   return it;
 }
 
@@ -151,11 +172,13 @@ __device__ __forceinline__ void tmem_st_32x32(uint32_t taddr, const uint32_t (&v
 }
 __device__ __forceinline__ void tmem_st_wait() { asm volatile("tcgen05.wait::st.sync.aligned;" ::: "memory"); }
 
-template <typename T>
-__global__ void __launch_bounds__(NUM_THREADS, CTAS_PER_SM)
+template <typename T, int D, bool WIN>
+__global__ void __launch_bounds__(NUM_THREADS, Cfg<D>::CTAS_PER_SM)
 attention_sm100_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k,
                        const __grid_constant__ CUtensorMap map_v, Params p, uint32_t idesc_s, uint32_t idesc_pv) {
   constexpr bool IS_FP16 = DType<T>::code == B200_F16;
+  using C = Cfg<D>;
+  constexpr int Q_BYTES = C::Q_BYTES, KV_TILE_BYTES = C::KV_TILE_BYTES, KV_STAGE_BYTES = C::KV_STAGE_BYTES, ATOMS = C::ATOMS;
   extern __shared__ uint8_t smem_raw[];
   const uint32_t raw = smem_u32(smem_raw);
   const uint32_t base = (raw + 1023u) & ~1023u;
@@ -223,11 +246,13 @@ attention_sm100_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
       uint32_t qi = 0, ki = 0;
       bool alive = true;
       for (int64_t idx = blockIdx.x; idx < n_items && alive; idx += gridDim.x) {
-        const Item it = decode_item(idx, bh_total, n_qt, p.NH, p.L);
+        const Item it = decode_item<WIN>(idx, bh_total, n_qt, p.NH, p.L, p);
         const uint32_t qb = qi & 1;
         if (!mbar_wait(bar_q_empty + 8 * qb, ((qi >> 1) & 1) ^ 1u, abort_flag, p.status_word, 11)) break;
         mbar_arrive_expect_tx(bar_q_full + 8 * qb, Q_BYTES);
-        tma_load_4d(smem_q + qb * Q_BYTES, &map_q, bar_q_full + 8 * qb, 0, p.q_head_inner ? it.h : it.q0, p.q_head_inner ? it.q0 : it.h, it.b);
+#pragma unroll
+        for (int a = 0; a < ATOMS; ++a)
+          tma_load_4d(smem_q + qb * Q_BYTES + a * C::Q_ATOM_BYTES, &map_q, bar_q_full + 8 * qb, 64 * a, p.q_head_inner ? it.h : it.q0, p.q_head_inner ? it.q0 : it.h, it.b);
         ++qi;
         for (int j = 0; j < it.nblk; ++j) {
           const uint32_t st = ki % KV_STAGES;
@@ -236,8 +261,13 @@ attention_sm100_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
             break;
           }
           mbar_arrive_expect_tx(bar_kv_full + 8 * st, KV_STAGE_BYTES);
-          tma_load_4d(smem_kv + st * KV_STAGE_BYTES, &map_k, bar_kv_full + 8 * st, 0, p.k_head_inner ? it.h : j * BLOCK_N, p.k_head_inner ? j * BLOCK_N : it.h, it.b);
-          tma_load_4d(smem_kv + st * KV_STAGE_BYTES + KV_TILE_BYTES, &map_v, bar_kv_full + 8 * st, 0, p.v_head_inner ? it.h : j * BLOCK_N, p.v_head_inner ? j * BLOCK_N : it.h, it.b);
+          const int key = it.k0 + j * BLOCK_N;
+#pragma unroll
+          for (int a = 0; a < ATOMS; ++a) {
+            const uint32_t dst = smem_kv + st * KV_STAGE_BYTES + a * C::KV_ATOM_BYTES;
+            tma_load_4d(dst, &map_k, bar_kv_full + 8 * st, 64 * a, p.k_head_inner ? it.h : key, p.k_head_inner ? key : it.h, it.b);
+            tma_load_4d(dst + KV_TILE_BYTES, &map_v, bar_kv_full + 8 * st, 64 * a, p.v_head_inner ? it.h : key, p.v_head_inner ? key : it.h, it.b);
+          }
           ++ki;
         }
       }
@@ -257,14 +287,16 @@ attention_sm100_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
         const uint64_t da = desc_kmajor(smem_q + qb * Q_BYTES);
         const uint64_t db = desc_kmajor(smem_kv + st * KV_STAGE_BYTES);
 #pragma unroll
-        for (int k = 0; k < D / 16; ++k) umma_f16(tmem_s + sb * BLOCK_N, da + (uint64_t)(2 * k), db + (uint64_t)(2 * k), idesc_s, (uint32_t)(k != 0));
+        for (int k = 0; k < D / 16; ++k)  // 16 elements further = 32 bytes inside the swizzled row, 64 = the next atom
+          umma_f16(tmem_s + sb * BLOCK_N, da + (uint64_t)(2 * (k & 3) + (k >> 2) * (C::Q_ATOM_BYTES >> 4)),
+                   db + (uint64_t)(2 * (k & 3) + (k >> 2) * (C::KV_ATOM_BYTES >> 4)), idesc_s, (uint32_t)(k != 0));
         umma_commit(bar_s_full + 8 * sb);
         ++si;
         ++ks;
         return true;
       };
       for (int64_t idx = blockIdx.x; idx < n_items && alive; idx += gridDim.x) {
-        const Item it = decode_item(idx, bh_total, n_qt, p.NH, p.L);
+        const Item it = decode_item<WIN>(idx, bh_total, n_qt, p.NH, p.L, p);
         const uint32_t qb = qi & 1;
         if (!mbar_wait(bar_q_full + 8 * qb, (qi >> 1) & 1, abort_flag, p.status_word, 15)) break;
         if (!issue_s(qb)) break;
@@ -285,7 +317,7 @@ attention_sm100_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
           }
           tc_fence_after();
           const uint64_t da = desc_kmajor(smem_p);
-          const uint64_t db = desc_mnmajor(smem_kv + st * KV_STAGE_BYTES + KV_TILE_BYTES);
+          const uint64_t db = desc_mnmajor(smem_kv + st * KV_STAGE_BYTES + KV_TILE_BYTES, ATOMS == 1 ? 1024 : C::KV_ATOM_BYTES);
 #pragma unroll
           for (int k = 0; k < BLOCK_N / 16; ++k) {
             // A: +16 keys = +32 bytes inside the swizzled row; B: +16 keys = two 8-key groups = +2048 bytes
@@ -307,7 +339,7 @@ attention_sm100_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
     const uint32_t lane_addr = (uint32_t)(quarter * 32) << 16;
     const uint32_t p_row = smem_p + (uint32_t)r_in_tile * 128u;
     const uint32_t sw = (uint32_t)(r_in_tile & 7);
-    const uint32_t o_addr = tmem_o + lane_addr + (uint32_t)(half * 32);
+    const uint32_t o_addr = tmem_o + lane_addr + (uint32_t)(half * (D / 2));
     // Exchange between the two threads of a row: slot layout [3][2][128] floats.  Block exchanges alternate between
     // slots 0 and 1 (a thread can only be one exchange ahead of its partner), the end-of-item exchange uses slot 2.
     float* my_x = xchg + half * BLOCK_M + r_in_tile;
@@ -327,9 +359,11 @@ attention_sm100_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
     uint32_t it_count = 0;  // 64-key blocks processed so far by this CTA
     bool alive = true;
     for (int64_t idx = blockIdx.x; idx < n_items && alive; idx += gridDim.x) {
-      const Item it = decode_item(idx, bh_total, n_qt, p.NH, p.L);
+      const Item it = decode_item<WIN>(idx, bh_total, n_qt, p.NH, p.L, p);
       const int row = it.q0 + r_in_tile;
       const int warp_row0 = it.q0 + quarter * 32;       // first query row of this warp
+      // (key indices of the same rows: hist further)
+      const int krow = WIN ? row + p.hist : row, warp_krow0 = WIN ? warp_row0 + p.hist : warp_row0;
       const bool warp_live = warp_row0 < it.q_end;      // a warp whose 32 rows all lie beyond the tile's end only keeps the handshakes going
       float m_run = -INFINITY, l_run = 0.f;             // l_run: this thread's half of the row's denominator
       for (int j = 0; j < it.nblk; ++j, ++it_count) {
@@ -339,9 +373,9 @@ attention_sm100_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
           break;
         }
         tc_fence_after();
-        const int k0 = j * BLOCK_N + half * 32;  // first key of this thread's 32
-        // keys above this warp's last row are masked for the whole warp
-        const bool live = warp_live && k0 <= warp_row0 + 31;
+        const int k0 = it.k0 + j * BLOCK_N + half * 32;  // first key of this thread's 32
+        // keys above this warp's last row (or behind the window of its first) are masked for the whole warp
+        const bool live = warp_live && k0 <= warp_krow0 + 31 && (!WIN || k0 + 31 > warp_krow0 - p.window);
         uint32_t v[32];
         if (live) {
           tmem_ld_32x32(tmem_s + lane_addr + sb * BLOCK_N + (uint32_t)(half * 32), v);
@@ -356,11 +390,12 @@ attention_sm100_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
         // exponentials below need no second test.
         float bm = -INFINITY;
         if (live) {
-          if (k0 + 31 > warp_row0) {
-            const int lim = row - k0;  // keys i <= lim are visible to this row
+          if (k0 + 31 > warp_krow0 || (WIN && k0 <= warp_krow0 + 31 - p.window)) {
+            const int lim = krow - k0;  // keys i <= lim are visible to this row
+            const int low = WIN ? lim - p.window : -1;  // ... and so are only keys i > low
 #pragma unroll
             for (int i = 0; i < 32; ++i) {
-              if (i > lim) v[i] = 0xff800000u;
+              if (i > lim || (WIN && i <= low)) v[i] = 0xff800000u;
               bm = fmaxf(bm, __uint_as_float(v[i]));
             }
           } else {
@@ -380,9 +415,11 @@ attention_sm100_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
           break;
         }
         bm = fmaxf(bm, partner_bm);
-        const float m_new = fmaxf(m_run, bm * p.scale_log2e);  // running maximum, in log2 units
-        const float mult = ex2f(m_run - m_new);
+        float m_new = fmaxf(m_run, bm * p.scale_log2e);  // running maximum, in log2 units
+        const float m_old = m_run;
         m_run = m_new;
+        if (WIN && m_new == -INFINITY) m_new = 0.f;  // nothing in this row's window yet: every exponential below is 0
+        const float mult = ex2f(m_old - m_new);
         // the previous block's P V must be complete: it read the P tile that is about to be overwritten, and it
         // produced the O that is about to be rescaled (the first block of an item finds both free: the previous
         // item's last P V was awaited before its output was stored)
@@ -416,10 +453,10 @@ attention_sm100_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
           for (int g = 0; g < 4; ++g) st_shared_v4(p_row + ((((uint32_t)(half * 4 + g)) ^ sw) << 4), 0u, 0u, 0u, 0u);
         }
         if constexpr (sizeof(T) == 2 && !IS_FP16) {
-          // bf16 storage: V_j -> fp16 in place, 32 bytes per softmax thread (the swizzle is address-agnostic)
-          const uint32_t vaddr = smem_kv + (it_count % KV_STAGES) * KV_STAGE_BYTES + KV_TILE_BYTES + (uint32_t)(threadIdx.x - 64) * 32u;
+          // bf16 storage: V_j -> fp16 in place, 32 bytes per softmax thread and atom (the swizzle is address-agnostic)
+          const uint32_t vaddr = smem_kv + (it_count % KV_STAGES) * KV_STAGE_BYTES + KV_TILE_BYTES + (uint32_t)(threadIdx.x - 64) * (32u * ATOMS);
 #pragma unroll
-          for (int g = 0; g < 2; ++g) {
+          for (int g = 0; g < 2 * ATOMS; ++g) {
             uint32_t w4[4];
             ld_shared_v4(vaddr + g * 16, w4);
 #pragma unroll
@@ -433,12 +470,15 @@ attention_sm100_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
         }
         // o = o * exp(m_old - m_new) in tensor memory, for this warp's 32 rows x 32 columns, unless no row's maximum moved
         if (j > 0 && warp_live && __any_sync(0xffffffffu, mult != 1.0f)) {
-          uint32_t a[32];
-          tmem_ld_32x32(o_addr, a);
-          tmem_ld_wait();
 #pragma unroll
-          for (int i = 0; i < 32; ++i) a[i] = __float_as_uint(__uint_as_float(a[i]) * mult);
-          tmem_st_32x32(o_addr, a);
+          for (int c = 0; c < ATOMS; ++c) {
+            uint32_t a[32];
+            tmem_ld_32x32(o_addr + c * 32, a);
+            tmem_ld_wait();
+#pragma unroll
+            for (int i = 0; i < 32; ++i) a[i] = __float_as_uint(__uint_as_float(a[i]) * mult);
+            tmem_st_32x32(o_addr + c * 32, a);
+          }
           tmem_st_wait();
         }
         // P (and, for bf16, the converted V) is complete, O is rescaled: P V of this block may be issued
@@ -457,21 +497,28 @@ attention_sm100_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
       if (!mbar_wait(bar_pv_done, (it_count - 1) & 1, abort_flag, p.status_word, 21)) break;
       tc_fence_after();
       if (warp_live) {  // (warp-uniform: the tensor-memory load below is a warp-wide instruction)
-        const float inv = 1.0f / l_row;
-        T* dst = reinterpret_cast<T*>(p.out) + (int64_t)it.b * p.so_b + (int64_t)it.h * p.so_h + (int64_t)row * p.so_l + half * 32;
-        uint32_t a[32];
-        tmem_ld_32x32(o_addr, a);
-        tmem_ld_wait();
-        uint32_t w[16];
+        float denom = l_row;
+        if (WIN && p.sink) denom += ex2f(__ldg(p.sink + it.h) * 1.4426950408889634f - m_run);
+        const float inv = 1.0f / denom;
+        T* dst = reinterpret_cast<T*>(p.out) + (int64_t)it.b * p.so_b + (int64_t)it.h * p.so_h + (int64_t)row * p.so_l + half * (D / 2);
 #pragma unroll
-        for (int i = 0; i < 16; ++i) w[i] = pack_out<T>(__uint_as_float(a[2 * i]) * inv, __uint_as_float(a[2 * i + 1]) * inv);
-        if (row < it.q_end) {
-          if (p.out_vec32) {
-            st_global_v8(dst, &w[0]);
-            st_global_v8(dst + 16, &w[8]);
-          } else {
+        for (int c = 0; c < ATOMS; ++c) {
+          uint32_t a[32];
+          tmem_ld_32x32(o_addr + c * 32, a);
+          tmem_ld_wait();
+          uint32_t w[16];
 #pragma unroll
-            for (int g = 0; g < 4; ++g) *reinterpret_cast<uint4*>(dst + g * 8) = make_uint4(w[4 * g], w[4 * g + 1], w[4 * g + 2], w[4 * g + 3]);
+          for (int i = 0; i < 16; ++i) w[i] = pack_out<T>(__uint_as_float(a[2 * i]) * inv, __uint_as_float(a[2 * i + 1]) * inv);
+          const int room = WIN ? p.vdim - half * (D / 2) - c * 32 : 32;  // columns of these 32 that exist (a multiple of 8)
+          if (row < it.q_end) {
+            if (p.out_vec32 && room >= 32) {
+              st_global_v8(dst + c * 32, &w[0]);
+              st_global_v8(dst + c * 32 + 16, &w[8]);
+            } else {
+#pragma unroll
+              for (int g = 0; g < 4; ++g)
+                if (g * 8 < room) *reinterpret_cast<uint4*>(dst + c * 32 + g * 8) = make_uint4(w[4 * g], w[4 * g + 1], w[4 * g + 2], w[4 * g + 3]);
+            }
           }
         }
       }
@@ -499,12 +546,12 @@ attention_sm100_kernel(const __grid_constant__ CUtensorMap map_q, const __grid_c
 // 4-D map over a strided (batch, head, row) view with contiguous head_dim.  The two middle dimensions are
 // ordered by ascending stride ({D, row, head, batch} for contiguous [B, NH, L, D] tensors, {D, head, row, batch}
 // for views into a fused [B, L, 3*NH*D] projection); *head_inner tells the kernel which order was used.
-static int make_map(CUtensorMap* map, const void* ptr, int64_t B, int64_t NH, int64_t L, const int64_t* s, int box_rows, int dtype,
+static int make_map(CUtensorMap* map, const void* ptr, int64_t B, int64_t NH, int64_t L, int64_t D, const int64_t* s, int box_rows, int dtype,
                     int* head_inner) {
   *head_inner = s[1] < s[2];
   uint64_t dims[4] = {(uint64_t)D, (uint64_t)L, (uint64_t)NH, (uint64_t)B};
   uint64_t strides[3] = {(uint64_t)s[2] * 2, (uint64_t)s[1] * 2, (uint64_t)s[0] * 2};
-  uint32_t box[4] = {(uint32_t)D, (uint32_t)box_rows, 1, 1};
+  uint32_t box[4] = {64, (uint32_t)box_rows, 1, 1};
   if (*head_inner) {
     dims[1] = (uint64_t)NH, dims[2] = (uint64_t)L;
     strides[0] = (uint64_t)s[1] * 2, strides[1] = (uint64_t)s[2] * 2;
@@ -530,21 +577,24 @@ int launch_attention_sm100(const void* q, const void* k, const void* v, void* ou
                            const int64_t* qs, const int64_t* ks, const int64_t* vs, const int64_t* os, float scale, int in_dtype,
                            int out_dtype, int* status_word, cudaStream_t stream) {
   using namespace attn100;
+  constexpr int D = 64;
+  using C = Cfg<D>;
   if (Dh != D || in_dtype != out_dtype || (in_dtype != B200_F16 && in_dtype != B200_BF16)) return B200_ERR_UNSUPPORTED;
   if (!view_ok(q, qs, B, NH) || !view_ok(k, ks, B, NH) || !view_ok(v, vs, B, NH) || !view_ok(out, os, B, NH)) return B200_ERR_UNSUPPORTED;
   if (B * NH > 0x7fffffffLL || L > 0x7fffff00LL || B > 0x7fffffffLL) return B200_ERR_UNSUPPORTED;
   CUtensorMap mq, mk, mv;
   Params p;
-  int st = make_map(&mq, q, B, NH, L, qs, BLOCK_M, in_dtype, &p.q_head_inner);
-  if (st == B200_OK) st = make_map(&mk, k, B, NH, L, ks, BLOCK_N, in_dtype, &p.k_head_inner);
-  if (st == B200_OK) st = make_map(&mv, v, B, NH, L, vs, BLOCK_N, in_dtype, &p.v_head_inner);
+  p.hist = 0, p.window = 0, p.vdim = D, p.sink = nullptr;
+  int st = make_map(&mq, q, B, NH, L, D, qs, BLOCK_M, in_dtype, &p.q_head_inner);
+  if (st == B200_OK) st = make_map(&mk, k, B, NH, L, D, ks, BLOCK_N, in_dtype, &p.k_head_inner);
+  if (st == B200_OK) st = make_map(&mv, v, B, NH, L, D, vs, BLOCK_N, in_dtype, &p.v_head_inner);
   if (st != B200_OK) return B200_ERR_UNSUPPORTED;  // e.g. strides the tensor map cannot express
   static std::atomic<bool> attr_set[kMaxDevices];  // kernel attributes are per device
   const int slot = device_slot();
   if (slot < 0) return B200_ERR_CUDA;
   if (!attr_set[slot].load(std::memory_order_acquire)) {
-    if (cudaFuncSetAttribute(attention_sm100_kernel<__half>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES) != cudaSuccess ||
-        cudaFuncSetAttribute(attention_sm100_kernel<__nv_bfloat16>, cudaFuncAttributeMaxDynamicSharedMemorySize, SMEM_BYTES) != cudaSuccess)
+    if (cudaFuncSetAttribute(attention_sm100_kernel<__half, D, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, C::SMEM_BYTES) != cudaSuccess ||
+        cudaFuncSetAttribute(attention_sm100_kernel<__nv_bfloat16, D, false>, cudaFuncAttributeMaxDynamicSharedMemorySize, C::SMEM_BYTES) != cudaSuccess)
       return B200_ERR_CUDA;
     attr_set[slot].store(true, std::memory_order_release);
   }
@@ -555,15 +605,63 @@ int launch_attention_sm100(const void* q, const void* k, const void* v, void* ou
   p.out_vec32 = (reinterpret_cast<uintptr_t>(out) & 31) == 0 && os[0] % 16 == 0 && os[1] % 16 == 0 && os[2] % 16 == 0;
   p.status_word = status_word;
   const int64_t n_items = ((L + BLOCK_M - 1) / BLOCK_M) * B * NH;
-  int64_t grid = (int64_t)sm_count() * CTAS_PER_SM;
+  int64_t grid = (int64_t)sm_count() * C::CTAS_PER_SM;
   if (grid > n_items) grid = n_items;
   // S = Q K^T in the storage format; P V always fp16 x fp16 (see the top of this file)
-  LaunchSetup ls(dim3((unsigned)grid), dim3(NUM_THREADS), SMEM_BYTES, stream);
+  LaunchSetup ls(dim3((unsigned)grid), dim3(NUM_THREADS), C::SMEM_BYTES, stream);
   const cudaError_t e = in_dtype == B200_BF16
-                            ? cudaLaunchKernelEx(&ls.cfg, attention_sm100_kernel<__nv_bfloat16>, mq, mk, mv, p, idesc(1, 1, 0), idesc(0, 0, 1))
-                            : cudaLaunchKernelEx(&ls.cfg, attention_sm100_kernel<__half>, mq, mk, mv, p, idesc(0, 0, 0), idesc(0, 0, 1));
+                            ? cudaLaunchKernelEx(&ls.cfg, attention_sm100_kernel<__nv_bfloat16, D, false>, mq, mk, mv, p, idesc(1, 1, 0, BLOCK_N), idesc(0, 0, 1, D))
+                            : cudaLaunchKernelEx(&ls.cfg, attention_sm100_kernel<__half, D, false>, mq, mk, mv, p, idesc(0, 0, 0, BLOCK_N), idesc(0, 0, 1, D));
   note_launches(1);
   return status_from_cuda(e);
+}
+
+namespace attn100 {
+// Sliding-window attention, bf16, D = 64 or 128 covering both head sizes.
+template <int D>
+static int launch_window(const CUtensorMap& mq, const CUtensorMap& mk, const CUtensorMap& mv, const Params& p, int64_t n_items, cudaStream_t stream) {
+  using C = Cfg<D>;
+  auto* kernel = attention_sm100_kernel<__nv_bfloat16, D, true>;
+  static std::atomic<bool> attr_set[kMaxDevices];
+  const int slot = device_slot();
+  if (slot < 0) return B200_ERR_CUDA;
+  if (!attr_set[slot].load(std::memory_order_acquire)) {
+    if (cudaFuncSetAttribute(kernel, cudaFuncAttributeMaxDynamicSharedMemorySize, C::SMEM_BYTES) != cudaSuccess) return B200_ERR_CUDA;
+    attr_set[slot].store(true, std::memory_order_release);
+  }
+  int64_t grid = (int64_t)sm_count() * C::CTAS_PER_SM;
+  if (grid > n_items) grid = n_items;
+  LaunchSetup ls(dim3((unsigned)grid), dim3(NUM_THREADS), C::SMEM_BYTES, stream);
+  const cudaError_t e = cudaLaunchKernelEx(&ls.cfg, kernel, mq, mk, mv, p, idesc(1, 1, 0, BLOCK_N), idesc(0, 0, 1, D));
+  note_launches(1);
+  return status_from_cuda(e);
+}
+}  // namespace attn100
+
+int launch_window_attention_sm100(const void* q, int64_t ld_q, const void* k, int64_t ld_k, const void* v, int64_t ld_v, void* out, int64_t ld_out,
+                                  int64_t B, int64_t n_new, int64_t hist, int64_t heads, int64_t dim, int64_t vdim, int64_t window, float scale,
+                                  const float* sink, int dtype, int* status_word, cudaStream_t stream) {
+  using namespace attn100;
+  const int64_t keys = hist + n_new;
+  if (dtype != B200_BF16 || dim > 128 || vdim > 128 || dim % 8 || vdim % 8 || !(scale > 0.f)) return B200_ERR_UNSUPPORTED;
+  const int64_t qs[3] = {n_new * ld_q, dim, ld_q}, ks[3] = {keys * ld_k, dim, ld_k}, vs[3] = {keys * ld_v, vdim, ld_v}, os[3] = {n_new * ld_out, vdim, ld_out};
+  if (!view_ok(q, qs, B, heads) || !view_ok(k, ks, B, heads) || !view_ok(v, vs, B, heads) || !view_ok(out, os, B, heads)) return B200_ERR_UNSUPPORTED;
+  if (B * heads > 0x7fffffffLL || keys > 0x7fffff00LL || B > 0x7fffffffLL) return B200_ERR_UNSUPPORTED;
+  CUtensorMap mq, mk, mv;
+  Params p;
+  int st = make_map(&mq, q, B, heads, n_new, dim, qs, BLOCK_M, dtype, &p.q_head_inner);
+  if (st == B200_OK) st = make_map(&mk, k, B, heads, keys, dim, ks, BLOCK_N, dtype, &p.k_head_inner);
+  if (st == B200_OK) st = make_map(&mv, v, B, heads, keys, vdim, vs, BLOCK_N, dtype, &p.v_head_inner);
+  if (st != B200_OK) return B200_ERR_UNSUPPORTED;
+  p.out = out;
+  p.so_b = os[0], p.so_h = os[1], p.so_l = os[2];
+  p.B = (int)B, p.NH = (int)heads, p.L = (int)n_new;
+  p.scale_log2e = scale * 1.4426950408889634f;
+  p.out_vec32 = (reinterpret_cast<uintptr_t>(out) & 31) == 0 && os[0] % 16 == 0 && os[1] % 16 == 0 && os[2] % 16 == 0;
+  p.status_word = status_word;
+  p.hist = (int)hist, p.window = (int)(window < keys ? window : keys), p.vdim = (int)vdim, p.sink = sink;
+  const int64_t n_items = ((n_new + BLOCK_M - 1) / BLOCK_M) * B * heads;
+  return dim <= 64 && vdim <= 64 ? launch_window<64>(mq, mk, mv, p, n_items, stream) : launch_window<128>(mq, mk, mv, p, n_items, stream);
 }
 
 }  // namespace b200

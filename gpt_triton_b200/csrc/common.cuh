@@ -265,10 +265,19 @@ int launch_latent_gather(const void* cache, void* work, int64_t B, int64_t T, in
 int launch_window_attention(const void* q, int64_t ld_q, const void* k, int64_t ld_k, const void* v, int64_t ld_v, void* out, int64_t ld_out,
                             int64_t B, int64_t T, int64_t hist, int64_t heads, int64_t dim, int64_t vdim, int64_t window, float scale,
                             const float* sink, int dtype, int* status_word, cudaStream_t stream);
+// tcgen05/TMA version (bf16, head sizes up to 128 in multiples of 8); B200_ERR_UNSUPPORTED means "use the generic kernel".
+int launch_window_attention_sm100(const void* q, int64_t ld_q, const void* k, int64_t ld_k, const void* v, int64_t ld_v, void* out, int64_t ld_out,
+                                  int64_t B, int64_t n_new, int64_t hist, int64_t heads, int64_t dim, int64_t vdim, int64_t window, float scale,
+                                  const float* sink, int dtype, int* status_word, cudaStream_t stream);
 size_t latent_decode_workspace_bytes(int64_t B, int64_t heads, int64_t R, int64_t window, int dtype);
 int launch_latent_decode(const void* q, int64_t ld_q, const void* w_uk, const void* w_uv, const void* cache, void* out, int64_t ld_out, int64_t B,
                          int64_t heads, int64_t dim, int64_t vdim, int64_t R, int64_t ring, int64_t window, float scale, const float* sink,
                          int dtype, const int* pos_dev, void* workspace, cudaStream_t stream);
+// Tensor-core version (bf16, sizes in multiples of 8, R up to 512); B200_ERR_UNSUPPORTED means "use the generic kernels".
+size_t latent_decode_mma_workspace_bytes(int64_t B, int64_t heads, int64_t R, int64_t window);
+int launch_latent_decode_mma(const void* q, int64_t ld_q, const void* w_uk, const void* w_uv, const void* cache, void* out, int64_t ld_out, int64_t B,
+                             int64_t heads, int64_t dim, int64_t vdim, int64_t R, int64_t ring, int64_t window, float scale, const float* sink,
+                             const int* pos_dev, void* workspace, cudaStream_t stream);
 int64_t decayed_attention_slices(int64_t T, int64_t heads, int64_t dim, int64_t vdim, int dtype);
 size_t decayed_attention_workspace_bytes(int64_t B, int64_t T, int64_t heads, int64_t dim, int64_t vdim, int dtype);
 int launch_decayed_attention(const void* qkvg, int64_t ld, int64_t off_k, int64_t off_v, int64_t off_g, const double* decay, const float* weight,

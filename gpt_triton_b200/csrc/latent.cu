@@ -253,21 +253,31 @@ int launch_latent_gather(const void* cache, void* work, int64_t B, int64_t n_new
 int launch_window_attention(const void* q, int64_t ld_q, const void* k, int64_t ld_k, const void* v, int64_t ld_v, void* out, int64_t ld_out,
                             int64_t B, int64_t n_new, int64_t hist, int64_t heads, int64_t dim, int64_t vdim, int64_t window, float scale,
                             const float* sink, int dtype, int* status_word, cudaStream_t stream) {
-  (void)status_word;
+  {
+    const int st = launch_window_attention_sm100(q, ld_q, k, ld_k, v, ld_v, out, ld_out, B, n_new, hist, heads, dim, vdim, window, scale, sink, dtype,
+                                                 status_word, stream);
+    if (st != B200_ERR_UNSUPPORTED) return st;
+  }
   if (dtype == B200_BF16)
     return window_typed<__nv_bfloat16>(q, ld_q, k, ld_k, v, ld_v, out, ld_out, B, n_new, hist, heads, dim, vdim, window, scale, sink, stream);
   return window_typed<float>(q, ld_q, k, ld_k, v, ld_v, out, ld_out, B, n_new, hist, heads, dim, vdim, window, scale, sink, stream);
 }
 
 size_t latent_decode_workspace_bytes(int64_t B, int64_t heads, int64_t R, int64_t window, int dtype) {
-  (void)window, (void)dtype;
-  return (size_t)(2 * B * heads * R) * 4;
+  const size_t simple = (size_t)(2 * B * heads * R) * 4;
+  if (dtype != B200_BF16) return simple;
+  const size_t mma = latent_decode_mma_workspace_bytes(B, heads, R, window);
+  return mma > simple ? mma : simple;
 }
 
 int launch_latent_decode(const void* q, int64_t ld_q, const void* w_uk, const void* w_uv, const void* cache, void* out, int64_t ld_out, int64_t B,
                          int64_t heads, int64_t dim, int64_t vdim, int64_t R, int64_t ring, int64_t window, float scale, const float* sink,
                          int dtype, const int* pos_dev, void* workspace, cudaStream_t stream) {
   if (B * heads > 0x7fffffffLL || heads > 65535 || B > 65535 * kBatchTile) return B200_ERR_BAD_ARGUMENT;
+  if (dtype == B200_BF16) {
+    const int st = launch_latent_decode_mma(q, ld_q, w_uk, w_uv, cache, out, ld_out, B, heads, dim, vdim, R, ring, window, scale, sink, pos_dev, workspace, stream);
+    if (st != B200_ERR_UNSUPPORTED) return st;
+  }
   if (dtype == B200_BF16)
     return decode_typed<__nv_bfloat16>(q, ld_q, w_uk, w_uv, cache, out, ld_out, B, heads, dim, vdim, R, ring, window, scale, sink, pos_dev, workspace, stream);
   return decode_typed<float>(q, ld_q, w_uk, w_uv, cache, out, ld_out, B, heads, dim, vdim, R, ring, window, scale, sink, pos_dev, workspace, stream);

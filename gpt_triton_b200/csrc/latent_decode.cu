@@ -1,0 +1,350 @@
+// One-token latent attention on tensor cores (bf16): the heads of a sequence share its cached latents, so a block takes
+// 16 heads of one sequence and streams the latents once.
+//   head_product_kernel   q~ = W_uk[head]^T q  before, and  W_uv[head] o~  after: one small product per head
+//   latent_stream_kernel  scores q~ . c, online softmax and the weighted latent sum o~ over a range of the window
+//   latent_merge_kernel   merges the ranges of one (sequence, head), adds the sink's term, normalises
+// q~ and the softmax weights are fp32 by definition; they enter the MMAs as two bf16 parts each.
+#include <atomic>
+
+#include "mma_sync.cuh"
+
+namespace b200 {
+namespace {
+
+using namespace warp_mma;
+
+// ------------------------------------------------------------------ one product per head
+// out[b, h, n] = sum_k a[b, h, k] * w[h, n, k] (K_MAJOR) or w[h, k, n].  Tile: 16 * MB sequences x 64 columns; MB = 1: the
+// four warps take 16 columns each, MB = 4: 16 sequences each.  k, n multiples of 8.
+template <bool K_MAJOR, int MB, typename OutT>
+__global__ void __launch_bounds__(128)
+head_product_kernel(const __nv_bfloat16* __restrict__ a, int64_t lda, int64_t a_head, const __nv_bfloat16* __restrict__ w, int64_t w_head, int64_t ldw,
+                    OutT* __restrict__ out, int64_t ld_out, int64_t out_head, int B, int N, int K) {
+  constexpr int ROWS = 16 * MB, NT = MB == 1 ? 2 : 8;
+  __shared__ __align__(128) uint8_t tiles[2][(ROWS + 64) * 128];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g8 = lane >> 2, t4 = lane & 3;
+  const int n0 = blockIdx.x * 64, h = blockIdx.y, b0 = blockIdx.z * ROWS;
+  const int row_w = MB == 1 ? 0 : warp * 16, col_w = MB == 1 ? warp * 16 : 0;
+  a += h * a_head, w += h * w_head, out += h * out_head;
+  auto load = [&](int k0, int stage) {
+    const uint32_t sa = (uint32_t)__cvta_generic_to_shared(tiles[stage]), sw = sa + ROWS * 128;
+    for (int i = threadIdx.x; i < ROWS * 8; i += 128) {
+      const int r = i >> 3, c = i & 7;
+      const bool ok = b0 + r < B && k0 + c * 8 < K;
+      cp_async16(sa + swz<128>(r, c), ok ? a + (int64_t)(b0 + r) * lda + k0 + c * 8 : a, ok);
+    }
+    for (int i = threadIdx.x; i < 64 * 8; i += 128) {
+      const int r = i >> 3, c = i & 7;
+      const int n = n0 + (K_MAJOR ? r : c * 8), k = k0 + (K_MAJOR ? c * 8 : r);
+      const bool ok = n < N && k < K;
+      cp_async16(sw + swz<128>(r, c), ok ? w + (K_MAJOR ? (int64_t)n * ldw + k : (int64_t)k * ldw + n) : w, ok);
+    }
+    cp_async_commit();
+  };
+  float acc[NT][4];
+#pragma unroll
+  for (int i = 0; i < NT; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
+  load(0, 0);
+  int stage = 0;
+  for (int k0 = 0; k0 < K; k0 += 64, stage ^= 1) {
+    __syncthreads();
+    if (k0 + 64 < K) {
+      load(k0 + 64, stage ^ 1);
+      cp_async_wait<1>();
+    } else {
+      cp_async_wait<0>();
+    }
+    __syncthreads();
+    const uint32_t sa = (uint32_t)__cvta_generic_to_shared(tiles[stage]), sw = sa + ROWS * 128;
+#pragma unroll
+    for (int ks = 0; ks < 4; ++ks) {
+      uint32_t af[4];
+      ldsm4(af, sa + swz<128>(row_w + (lane & 15), ks * 2 + (lane >> 4)));
+#pragma unroll
+      for (int np = 0; np < NT / 2; ++np) {
+        uint32_t wf[4];
+        const int n = col_w + np * 16;
+        if (K_MAJOR) ldsm4(wf, sw + swz<128>(n + (lane & 7) + ((lane >> 4) << 3), ks * 2 + ((lane >> 3) & 1)));
+        else ldsm4_trans(wf, sw + swz<128>(ks * 16 + (lane & 7) + ((lane >> 3) & 1) * 8, n / 8 + (lane >> 4)));
+        mma_bf16(acc[2 * np], af, wf[0], wf[1]);
+        mma_bf16(acc[2 * np + 1], af, wf[2], wf[3]);
+      }
+    }
+  }
+#pragma unroll
+  for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      const int b = b0 + row_w + g8 + r * 8, n = n0 + col_w + nt * 8 + t4 * 2;
+      if (b < B && n < N) {
+        OutT* p = out + (int64_t)b * ld_out + n;
+        p[0] = from_float<OutT>(acc[nt][2 * r]), p[1] = from_float<OutT>(acc[nt][2 * r + 1]);
+      }
+    }
+}
+
+// ------------------------------------------------------------------ streaming the latents
+constexpr int kHeads = 16, kKeys = 64, kStreamThreads = 256;
+
+template <int RP>  // latent size, padded to 128, 256 or 512
+struct StreamSmem {
+  static constexpr int ROW = RP * 2;
+  static constexpr int C_BYTES = kKeys * ROW;
+  static constexpr int Q_BYTES = kHeads * ROW;
+  static constexpr int P_BYTES = kHeads * kKeys * 2;
+  static constexpr int BYTES = 2 * C_BYTES + 2 * Q_BYTES + 2 * P_BYTES;
+};
+
+// blockIdx.x = sequence, y = group of 16 heads, z = range of the window.  Partial results per (sequence, head, range):
+// part_ml = (maximum in log2 units, denominator), part_o = unnormalised sum of latents.
+template <int RP>
+__global__ void __launch_bounds__(kStreamThreads)
+latent_stream_kernel(const float* __restrict__ qt, const __nv_bfloat16* __restrict__ cache, float* __restrict__ part_o, float2* __restrict__ part_ml,
+                     int heads, int R, int64_t ring, int64_t window, float scale_log2e, const int* __restrict__ pos_dev) {
+  using M = StreamSmem<RP>;
+  constexpr int ROW = M::ROW, NT = RP / 64;  // 8-column output tiles per warp (eight warps)
+  extern __shared__ __align__(128) uint8_t smem[];
+  __shared__ float s_max[8][kHeads], s_sum[8][kHeads];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g8 = lane >> 2, t4 = lane & 3;
+  const int64_t b = blockIdx.x;
+  const int h0 = blockIdx.y * kHeads, split = blockIdx.z, n_split = gridDim.z;
+  const uint32_t base = (uint32_t)__cvta_generic_to_shared(smem);
+  const uint32_t q_hi = base + 2 * M::C_BYTES, q_lo = q_hi + M::Q_BYTES, p_hi = q_lo + M::Q_BYTES, p_lo = p_hi + M::P_BYTES;
+  const int64_t pos = pos_dev[0], first = pos + 1 > window ? pos + 1 - window : 0;
+  const int n_keys = pos < 0 ? 0 : (int)(pos - first + 1);
+  const int tiles = (n_keys + kKeys - 1) / kKeys, per = (tiles + n_split - 1) / n_split;
+  const int tile0 = split * per, tile1 = min(tiles, tile0 + per);
+
+  for (int i = threadIdx.x; i < kHeads * (RP / 2); i += kStreamThreads) {
+    const int r = i / (RP / 2), c = (i % (RP / 2)) * 2;
+    float2 v = make_float2(0.f, 0.f);
+    if (h0 + r < heads && c < R) v = *reinterpret_cast<const float2*>(qt + (b * heads + h0 + r) * R + c);
+    uint32_t hi, lo;
+    split_pair(v.x, v.y, hi, lo);
+    const uint32_t at = swz<ROW>(r, c >> 3) + (c & 7) * 2;
+    asm volatile("st.shared.b32 [%0], %1;" ::"r"(q_hi + at), "r"(hi) : "memory");
+    asm volatile("st.shared.b32 [%0], %1;" ::"r"(q_lo + at), "r"(lo) : "memory");
+  }
+  const __nv_bfloat16* cb = cache + b * ring * R;
+  const int64_t slot0 = first % ring;
+  auto load = [&](int tile, int stage) {
+    const uint32_t dst = base + stage * M::C_BYTES;
+    for (int i = threadIdx.x; i < kKeys * (RP / 8); i += kStreamThreads) {
+      const int r = i / (RP / 8), c = i % (RP / 8);
+      const int key = tile * kKeys + r;
+      const bool ok = key < n_keys && c * 8 < R;
+      int64_t slot = slot0 + key;  // (key < window <= ring: one wrap at most)
+      if (slot >= ring) slot -= ring;
+      cp_async16(dst + swz<ROW>(r, c), ok ? cb + slot * R + c * 8 : cb, ok);
+    }
+    cp_async_commit();
+  };
+
+  float o[NT][4];
+#pragma unroll
+  for (int i = 0; i < NT; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
+  float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};  // heads g8 and g8 + 8
+  if (tile0 < tile1) load(tile0, 0);
+  int stage = 0;
+  for (int tile = tile0; tile < tile1; ++tile, stage ^= 1) {
+    __syncthreads();  // the other stage and the weights of the tile before are no longer read
+    if (tile + 1 < tile1) {
+      load(tile + 1, stage ^ 1);
+      cp_async_wait<1>();
+    } else {
+      cp_async_wait<0>();
+    }
+    __syncthreads();
+    const uint32_t sc = base + stage * M::C_BYTES;
+    // scores of 16 heads x this warp's 8 keys
+    float s[4] = {0.f, 0.f, 0.f, 0.f};
+#pragma unroll 8
+    for (int ks = 0; ks < RP / 16; ++ks) {
+      uint32_t qh[4], ql[4], cf[2];
+      const uint32_t at = swz<ROW>(lane & 15, ks * 2 + (lane >> 4));
+      ldsm4(qh, q_hi + at);
+      ldsm4(ql, q_lo + at);
+      ldsm2(cf, sc + swz<ROW>(warp * 8 + (lane & 7), ks * 2 + ((lane >> 3) & 1)));
+      mma_bf16(s, qh, cf[0], cf[1]);
+      mma_bf16(s, ql, cf[0], cf[1]);
+    }
+    const int key = tile * kKeys + warp * 8 + t4 * 2;
+    float bm[2];
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      s[2 * r] = key < n_keys ? s[2 * r] * scale_log2e : -INFINITY;
+      s[2 * r + 1] = key + 1 < n_keys ? s[2 * r + 1] * scale_log2e : -INFINITY;
+      bm[r] = fmaxf(s[2 * r], s[2 * r + 1]);
+      bm[r] = fmaxf(bm[r], __shfl_xor_sync(0xffffffffu, bm[r], 1));
+      bm[r] = fmaxf(bm[r], __shfl_xor_sync(0xffffffffu, bm[r], 2));
+      if (t4 == 0) s_max[warp][g8 + r * 8] = bm[r];
+    }
+    __syncthreads();
+    float mult[2];
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      float m_new = m_run[r];
+#pragma unroll
+      for (int w2 = 0; w2 < 8; ++w2) m_new = fmaxf(m_new, s_max[w2][g8 + r * 8]);  // finite: a tile has at least one key
+      mult[r] = exp2f(m_run[r] - m_new);
+      m_run[r] = m_new;
+      const float p0 = exp2f(s[2 * r] - m_new), p1 = exp2f(s[2 * r + 1] - m_new);
+      uint32_t hi, lo;
+      split_pair(p0, p1, hi, lo);
+      const uint32_t at = swz<128>(g8 + r * 8, warp) + t4 * 4;
+      asm volatile("st.shared.b32 [%0], %1;" ::"r"(p_hi + at), "r"(hi) : "memory");
+      asm volatile("st.shared.b32 [%0], %1;" ::"r"(p_lo + at), "r"(lo) : "memory");
+      float ps = p0 + p1;
+      ps += __shfl_xor_sync(0xffffffffu, ps, 1);
+      ps += __shfl_xor_sync(0xffffffffu, ps, 2);
+      if (t4 == 0) s_sum[warp][g8 + r * 8] = ps;
+    }
+    __syncthreads();
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      float ps = 0.f;
+#pragma unroll
+      for (int w2 = 0; w2 < 8; ++w2) ps += s_sum[w2][g8 + r * 8];
+      l_run[r] = l_run[r] * mult[r] + ps;
+    }
+#pragma unroll
+    for (int i = 0; i < NT; ++i) o[i][0] *= mult[0], o[i][1] *= mult[0], o[i][2] *= mult[1], o[i][3] *= mult[1];
+    // o~ += P c for this warp's RP / 8 columns
+#pragma unroll
+    for (int kk = 0; kk < kKeys / 16; ++kk) {
+      uint32_t ph[4], pl[4];
+      const uint32_t at = swz<128>(lane & 15, kk * 2 + (lane >> 4));
+      ldsm4(ph, p_hi + at);
+      ldsm4(pl, p_lo + at);
+#pragma unroll
+      for (int np = 0; np < NT / 2; ++np) {
+        uint32_t cf[4];
+        ldsm4_trans(cf, sc + swz<ROW>(kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8, warp * NT + np * 2 + (lane >> 4)));
+        mma_bf16(o[2 * np], ph, cf[0], cf[1]);
+        mma_bf16(o[2 * np + 1], ph, cf[2], cf[3]);
+        mma_bf16(o[2 * np], pl, cf[0], cf[1]);
+        mma_bf16(o[2 * np + 1], pl, cf[2], cf[3]);
+      }
+    }
+  }
+#pragma unroll
+  for (int r = 0; r < 2; ++r) {
+    const int h = h0 + g8 + r * 8;
+    if (h >= heads) continue;
+    const int64_t item = (b * heads + h) * n_split + split;
+    if (warp == 0 && t4 == 0) part_ml[item] = make_float2(m_run[r], l_run[r]);
+#pragma unroll
+    for (int i = 0; i < NT; ++i) {
+      const int c = (warp * NT + i) * 8 + t4 * 2;
+      if (c < R) *reinterpret_cast<float2*>(part_o + item * R + c) = make_float2(o[i][2 * r], o[i][2 * r + 1]);
+    }
+  }
+}
+
+// One block per (sequence, head).
+__global__ void __launch_bounds__(128)
+latent_merge_kernel(const float* __restrict__ part_o, const float2* __restrict__ part_ml, __nv_bfloat16* __restrict__ ot, int heads, int R, int n_split,
+                    const float* __restrict__ sink) {
+  const int64_t item = blockIdx.x;
+  const int h = (int)(item % heads);
+  float m = -INFINITY;
+  for (int s = 0; s < n_split; ++s) m = fmaxf(m, part_ml[item * n_split + s].x);
+  float l = 0.f;
+  for (int s = 0; s < n_split; ++s) {
+    const float2 ml = part_ml[item * n_split + s];
+    l = fmaf(ml.y, exp2f(ml.x - m), l);
+  }
+  if (sink) l += exp2f(sink[h] * 1.4426950408889634f - m);
+  const float inv = 1.0f / l;
+  for (int r = threadIdx.x; r < R; r += 128) {
+    float v = 0.f;
+    for (int s = 0; s < n_split; ++s) {
+      const float f = exp2f(part_ml[item * n_split + s].x - m);
+      if (f > 0.f) v = fmaf(part_o[(item * n_split + s) * R + r], f, v);
+    }
+    ot[item * R + r] = __float2bfloat16_rn(v * inv);
+  }
+}
+
+size_t round256(size_t v) { return (v + 255) & ~(size_t)255; }
+
+struct Plan {
+  int n_split;
+  size_t off_po, off_ml, off_ot, bytes;
+};
+Plan make_plan(int64_t B, int64_t heads, int64_t R, int64_t window) {
+  Plan p;
+  const int64_t groups = B * ((heads + kHeads - 1) / kHeads), tiles = (window + kKeys - 1) / kKeys;
+  int64_t n = (sm_count() + groups - 1) / groups;
+  if (n > tiles) n = tiles;
+  if (n > 64) n = 64;
+  if (n < 1) n = 1;
+  p.n_split = (int)n;
+  size_t at = round256((size_t)(B * heads * R) * 4);  // q~
+  p.off_po = at, at += round256((size_t)(B * heads * n * R) * 4);
+  p.off_ml = at, at += round256((size_t)(B * heads * n) * 8);
+  p.off_ot = at, at += round256((size_t)(B * heads * R) * 2);
+  p.bytes = at;
+  return p;
+}
+
+template <int RP>
+int launch_stream(const float* qt, const void* cache, float* po, float2* ml, int64_t B, int64_t heads, int64_t R, int64_t ring, int64_t window,
+                  float scale, int n_split, const int* pos_dev, cudaStream_t stream) {
+  constexpr int smem = StreamSmem<RP>::BYTES;
+  static std::atomic<bool> attr_set[kMaxDevices];
+  const int slot = device_slot();
+  if (slot < 0) return B200_ERR_CUDA;
+  if (!attr_set[slot].load(std::memory_order_acquire)) {
+    if (cudaFuncSetAttribute(latent_stream_kernel<RP>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return B200_ERR_CUDA;
+    attr_set[slot].store(true, std::memory_order_release);
+  }
+  latent_stream_kernel<RP><<<dim3((unsigned)B, (unsigned)((heads + kHeads - 1) / kHeads), (unsigned)n_split), kStreamThreads, smem, stream>>>(
+      qt, static_cast<const __nv_bfloat16*>(cache), po, ml, (int)heads, (int)R, ring, window, scale * 1.4426950408889634f, pos_dev);
+  note_launches(1);
+  return status_from_cuda(cudaGetLastError());
+}
+
+template <bool K_MAJOR, typename OutT>
+void head_product(const __nv_bfloat16* a, int64_t lda, int64_t a_head, const __nv_bfloat16* w, int64_t w_head, int64_t ldw, OutT* out, int64_t ld_out,
+                  int64_t out_head, int64_t B, int64_t heads, int64_t N, int64_t K, cudaStream_t stream) {
+  const unsigned nb = (unsigned)((N + 63) / 64);
+  if (B <= 16)
+    head_product_kernel<K_MAJOR, 1, OutT><<<dim3(nb, (unsigned)heads, 1), 128, 0, stream>>>(a, lda, a_head, w, w_head, ldw, out, ld_out, out_head, (int)B, (int)N, (int)K);
+  else
+    head_product_kernel<K_MAJOR, 4, OutT><<<dim3(nb, (unsigned)heads, (unsigned)((B + 63) / 64)), 128, 0, stream>>>(a, lda, a_head, w, w_head, ldw, out, ld_out,
+                                                                                                                    out_head, (int)B, (int)N, (int)K);
+  note_launches(1);
+}
+
+bool aligned16_all(const void* a, const void* b, const void* c, const void* d) {
+  return ((reinterpret_cast<uintptr_t>(a) | reinterpret_cast<uintptr_t>(b) | reinterpret_cast<uintptr_t>(c) | reinterpret_cast<uintptr_t>(d)) & 15) == 0;
+}
+
+}  // namespace
+
+size_t latent_decode_mma_workspace_bytes(int64_t B, int64_t heads, int64_t R, int64_t window) { return make_plan(B, heads, R, window).bytes; }
+
+int launch_latent_decode_mma(const void* q, int64_t ld_q, const void* w_uk, const void* w_uv, const void* cache, void* out, int64_t ld_out, int64_t B,
+                             int64_t heads, int64_t dim, int64_t vdim, int64_t R, int64_t ring, int64_t window, float scale, const float* sink,
+                             const int* pos_dev, void* workspace, cudaStream_t stream) {
+  if (R > 512 || R % 8 || dim % 8 || vdim % 8 || ld_q % 8 || !aligned16_all(q, w_uk, w_uv, cache)) return B200_ERR_UNSUPPORTED;
+  if (B > 65535 || heads > 65535 || window > (1 << 30)) return B200_ERR_UNSUPPORTED;
+  const Plan p = make_plan(B, heads, R, window);
+  uint8_t* ws = static_cast<uint8_t*>(workspace);
+  float* qt = reinterpret_cast<float*>(ws);
+  float* po = reinterpret_cast<float*>(ws + p.off_po);
+  float2* ml = reinterpret_cast<float2*>(ws + p.off_ml);
+  __nv_bfloat16* ot = reinterpret_cast<__nv_bfloat16*>(ws + p.off_ot);
+  head_product<false, float>((const __nv_bfloat16*)q, ld_q, dim, (const __nv_bfloat16*)w_uk, dim * R, R, qt, heads * R, R, B, heads, R, dim, stream);
+  int st = R <= 128   ? launch_stream<128>(qt, cache, po, ml, B, heads, R, ring, window, scale, p.n_split, pos_dev, stream)
+           : R <= 256 ? launch_stream<256>(qt, cache, po, ml, B, heads, R, ring, window, scale, p.n_split, pos_dev, stream)
+                      : launch_stream<512>(qt, cache, po, ml, B, heads, R, ring, window, scale, p.n_split, pos_dev, stream);
+  if (st != B200_OK) return st;
+  latent_merge_kernel<<<(unsigned)(B * heads), 128, 0, stream>>>(po, ml, ot, (int)heads, (int)R, p.n_split, sink);
+  note_launches(1);
+  head_product<true, __nv_bfloat16>(ot, heads * R, R, (const __nv_bfloat16*)w_uv, vdim * R, R, (__nv_bfloat16*)out, ld_out, vdim, B, heads, vdim, R, stream);
+  return status_from_cuda(cudaGetLastError());
+}
+
+}  // namespace b200
