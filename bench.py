@@ -616,7 +616,7 @@ def kernel_trace(replay):
     gaps = [(b[0] - a[1], a[2][:60], b[2][:60]) for a, b in zip(recs, recs[1:])]
     by_name = {}
     for st, en, name in recs:
-        key = name.split("(")[0][:90]
+        key = name.replace("(anonymous namespace)::", "").split("(")[0][:90]
         n, t = by_name.get(key, (0, 0.0))
         by_name[key] = (n + 1, t + (en - st))
     return {
@@ -775,6 +775,209 @@ def run_decode(args):
     }))
 
 
+# Fogilix beside GPT-2-shaped FusedGPT models of the same width, depth, feed-forward and vocabulary (bf16 both).
+FOGILIX_SIZES = {
+    "w1024": {"width": 1024, "layers": 8, "vocab": 32768, "kv_rank": 256, "window": 512},
+    "w2048": {"width": 2048, "layers": 8, "vocab": 32768, "kv_rank": 512, "window": 1024},
+    "w4096": {"width": 4096, "layers": 4, "vocab": 32768, "kv_rank": 512, "window": 1024},
+}
+
+
+def fogilix_config(width, layers, vocab, kv_rank, window):
+    """Lightning and latent attention layers in turn (heads of 128), every second latent layer reading the latents of the
+    one before it, a 4x feed-forward everywhere."""
+    heads, out, owner = width // 128, [], None
+    for i in range(layers):
+        mlp = {"kind": "dense", "ff": 4 * width}
+        if i % 2 == 0:
+            mixer = {"heads": heads, "dim": 128, "vdim": 128, "decay": [1.0 - 2.0 ** -(3 + 7 * h / max(heads - 1, 1)) for h in range(heads)]}
+            out.append({"type": "lightning", "mixer": mixer, "mlp": mlp})
+        else:
+            mixer = {"heads": heads, "dim": 128, "vdim": 128, "kv_rank": kv_rank, "mask": {"size": window}, "scale": 128 ** -0.5}
+            if owner is None:
+                owner = i
+            else:
+                mixer["kv_from"], owner = owner, None
+            out.append({"type": "latent_attention", "mixer": mixer, "mlp": mlp})
+    return {"architecture": "Fogilix", "vocab": vocab, "width": width, "layers": out, "norm": {"eps": 1e-5}, "logit_scale": 1.0}
+
+
+def _random_parameters(model):
+    with torch.no_grad():
+        for name, prm in model.named_parameters():
+            if prm.dim() == 2:
+                prm.normal_(0.0, prm.shape[1] ** -0.5 if "embed" not in name and "wte" not in name and "wpe" not in name else 1.0)
+            else:
+                prm.zero_()
+                if name.endswith("layer_norm_weight") or name.endswith("mix.norm") or name.endswith("dkv_norm"):
+                    prm.fill_(1.0)
+    return model
+
+
+def fogilix_work(cfg, batch, n, cached, decode):
+    """Algorithmic flop and bytes of one pass, by kernel family: matrix products, window/latent attention, lightning."""
+    T, w = batch * n, cfg["width"]
+    gemm = attn = light = 0.0
+    gemm_b = attn_b = light_b = 0.0
+
+    def product(m, nn, k, out_bytes):
+        nonlocal gemm, gemm_b
+        gemm += 2.0 * m * nn * k
+        gemm_b += 2.0 * (m * k + nn * k) + out_bytes * m * nn
+
+    for layer in cfg["layers"]:
+        m = layer["mixer"]
+        hd, hv = m["heads"] * m["dim"], m["heads"] * m["vdim"]
+        if layer["type"] == "lightning":
+            product(T, 2 * hd + 2 * hv, w, 2)
+            # the recurrence itself: k v^T and S^T q per token
+            light += 4.0 * T * m["heads"] * m["dim"] * m["vdim"]
+            light_b += 2.0 * T * (2 * hd + 3 * hv) + 8.0 * batch * m["heads"] * m["dim"] * m["vdim"]
+        else:
+            R, win = m["kv_rank"], m["mask"]["size"]
+            product(T, hd + (0 if "kv_from" in m else R), w, 2)
+            if decode:
+                keys = min(cached + 1, win)
+                attn += 2.0 * T * m["heads"] * R * (m["dim"] + m["vdim"] + 2 * keys)
+                attn_b += 2.0 * T * keys * R + 2.0 * (hd + hv) * R + 2.0 * T * (hd + hv)
+            else:
+                product(T, hd + hv, R, 2)
+                pairs = sum(min(i + 1, win) for i in range(n)) * batch
+                attn += 2.0 * pairs * (hd + hv)
+                attn_b += 2.0 * T * (2 * hd + 2 * hv)
+        product(T, w, hv, 8 + 2)
+        product(T, layer["mlp"]["ff"], w, 2)
+        product(T, w, layer["mlp"]["ff"], 8 + 2)
+    product(batch, cfg["vocab"], w, 4)
+    return {"gemm": (gemm, gemm_b), "attention": (attn, attn_b), "lightning": (light, light_b)}
+
+
+def gpt_work(c, batch, n, cached, decode):
+    T, h = batch * n, c.n_embd
+    gemm = 2.0 * T * 12 * h * h * c.n_layer + 2.0 * batch * h * c.vocab_size
+    gemm_b = c.n_layer * (2.0 * 12 * h * h + 2.0 * T * (h + 3 * h + h + 2 * h + h + 4 * h + 4 * h + 2 * h)) + 2.0 * (c.vocab_size * h + batch * c.vocab_size)
+    if decode:
+        attn, attn_b = 4.0 * T * h * (cached + 1) * c.n_layer, c.n_layer * T * (cached + 1) * 2 * h * 2.0
+    else:
+        attn, attn_b = 4.0 * batch * h * (n * (n + 1) / 2) * c.n_layer, c.n_layer * T * 4 * h * 2.0
+    return {"gemm": (gemm, gemm_b), "attention": (attn, attn_b)}
+
+
+_FAMILY = (("gemm_", "gemm"), ("argmax_reduce", "gemm"), ("ln_stats_from", "gemm"), ("attention_sm100", "attention"), ("attention_decode", "attention"),
+           ("attention_kernel", "attention"), ("latent_append", "latents"), ("latent_gather", "latents"), ("latent_", "attention"),
+           ("head_product", "attention"), ("chunked_kernel", "lightning"), ("segment_scan", "lightning"), ("recurrent_kernel", "lightning"))
+
+
+def family_table(trace, work, peaks):
+    """Time per kernel family of one traced pass, against the family's roofline (the slower of flop / tensor peak and bytes /
+    copy bandwidth)."""
+    fam = {}
+    for name, rec in trace["per_kernel"].items():
+        key = next((f for pat, f in _FAMILY if pat in name), "other")
+        n, ms = fam.get(key, (0, 0.0))
+        fam[key] = (n + rec["launches"], ms + rec["total_ms"])
+    out = {}
+    for key, (n, ms) in fam.items():
+        out[key] = {"launches": n, "ms": round(ms, 4)}
+        if key == "other":
+            out[key]["kernels"] = {name[-60:]: round(rec["total_ms"], 4) for name, rec in trace["per_kernel"].items() if not any(pat in name for pat, _ in _FAMILY)}
+        if key in work:
+            flop, nbytes = work[key]
+            floor = max(flop / (peaks["bf16_tflops"] * 1e12), nbytes / (peaks["hbm_gbs"] * 1e9)) * 1e3
+            out[key].update({"roofline_ms": round(floor, 4), "frac": round(floor / ms, 3), "tflops": round(flop / ms * 1e-9, 1), "gbs": round(nbytes / ms * 1e-6, 1)})
+    return out
+
+
+def run_fogilix(args):
+    """Prefill and decode throughput of the Fogilix decoder at a few sizes (random weights, bf16), beside a FusedGPT of the
+    same width, depth, feed-forward and vocabulary: one JSON line per size, with the time of each kernel family against its
+    roofline.  Prefill: the prompt pass of a session (cache filled, first logits); decode: replays of the captured step."""
+    from gpt_triton_b200 import kernels as K
+    from gpt_triton_b200.fogilix import Fogilix, FogilixConfig
+    from gpt_triton_b200.generation import GenerationSession
+    from gpt_triton_b200.gpt import FusedGPT, GPTConfig
+
+    dev = torch.device("cuda", 0)
+    torch.cuda.set_device(dev)
+    peaks, peak_src = load_peaks()
+    s, e = torch.cuda.Event(enable_timing=True), torch.cuda.Event(enable_timing=True)
+
+    def timed(fn, reps):
+        for _ in range(3):
+            fn()
+        torch.cuda.synchronize()
+        s.record()
+        for _ in range(reps):
+            fn()
+        e.record()
+        torch.cuda.synchronize()
+        return s.elapsed_time(e) / reps
+
+    for size in (args.fogilix_size.split(",") if args.fogilix_size else list(FOGILIX_SIZES)):
+        z = FOGILIX_SIZES[size]
+        line = {"model": f"fogilix_{size}", **z, "dtype": "bf16", "data": "synthetic", "peak_source": peak_src, "runs": []}
+        for kind in ("fogilix", "gpt"):
+            torch.manual_seed(0)
+            with torch.device(dev):
+                if kind == "fogilix":
+                    cfg = fogilix_config(**z)
+                    model = Fogilix(FogilixConfig.from_dict(cfg))
+                else:
+                    cfg = GPTConfig(vocab_size=z["vocab"], block_size=4096, n_layer=z["layers"], n_head=z["width"] // 64, n_embd=z["width"])
+                    model = FusedGPT(cfg)
+            model = _random_parameters(model).to(torch.bfloat16).eval()
+            count = lambda b, n, cached, dec: (fogilix_work if kind == "fogilix" else gpt_work)(cfg, b, n, cached, dec)
+            for batch, n in ((16, 2048), (1, 4096)):
+                ids = torch.randint(0, z["vocab"], (batch, n), device=dev)
+                sess = GenerationSession(model, batch, n)
+
+                def prefill():
+                    sess.reset()
+                    with torch.no_grad():
+                        rows = sess.extend(ids)
+                        model.pick(rows, 0.0, 0, 0, sess.pos)
+
+                ms = timed(prefill, max(args.steps // 2, 3))
+                fam = family_table(kernel_trace(prefill), count(batch, n, 0, False), peaks)
+                if args.gap_table:
+                    print(json.dumps({"size": size, "arch": kind, "batch": batch, "tokens": n, **kernel_trace(prefill)}), file=sys.stderr)
+                line["runs"].append({"arch": kind, "phase": "prefill", "batch": batch, "tokens": n, "ms": round(ms, 4), "tokens_per_s": round(batch * n / ms * 1e3),
+                                     "families": fam})
+                del sess
+            for batch, cached in ((1, 2048), (16, 2048), (128, 2048)):
+                sess = GenerationSession(model, batch, cached + 40, max_new_tokens=40)
+                ids = torch.randint(0, z["vocab"], (batch, cached), device=dev)
+                sess.generate(ids, 8, portion=cached)
+                assert sess.graph is not None
+
+                def rewind():
+                    sess.pos.copy_(torch.tensor([cached, cached], dtype=torch.int32))
+
+                best = []
+                for _ in range(3):
+                    rewind()
+                    torch.cuda.synchronize()
+                    s.record()
+                    for _ in range(30):
+                        sess.graph.replay()
+                    e.record()
+                    torch.cuda.synchronize()
+                    best.append(s.elapsed_time(e) / 30)
+                ms = sorted(best)[1]
+                rewind()
+                fam = family_table(kernel_trace(sess.graph.replay), count(batch, 1, cached, True), peaks)
+                if args.gap_table:
+                    rewind()
+                    print(json.dumps({"size": size, "arch": kind, "batch": batch, "cached": cached, **kernel_trace(sess.graph.replay)}), file=sys.stderr)
+                line["runs"].append({"arch": kind, "phase": "decode", "batch": batch, "cached": cached, "ms_per_step": round(ms, 4),
+                                     "tokens_per_s": round(batch / ms * 1e3), "families": fam})
+                del sess
+            del model
+            torch.cuda.empty_cache()
+        assert K.device_status(dev) == 0
+        print(json.dumps(line), flush=True)
+
+
 def main():
     ap = argparse.ArgumentParser()
     ap.add_argument("--gpus", type=int, default=1)
@@ -792,7 +995,12 @@ def main():
     ap.add_argument("--gap-table", action="store_true", help="per-kernel time and idle gaps of one replayed forward (diagnosis)")
     ap.add_argument("--decode", action="store_true", help="time token-by-token generation (key/value cache) instead of the forward")
     ap.add_argument("--new-tokens", type=int, default=64, help="--decode: tokens generated per sequence")
+    ap.add_argument("--fogilix", action="store_true", help="prefill and decode throughput of the Fogilix decoder beside a FusedGPT of equal size")
+    ap.add_argument("--fogilix-size", default="", help=f"--fogilix: sizes to run, with commas between them (of {', '.join(FOGILIX_SIZES)}; default all)")
     args = ap.parse_args()
+    if args.fogilix:
+        run_fogilix(args)
+        return
     if args.decode:  # (with --gap-table: the per-kernel trace of one decode step instead of the timing line)
         run_decode(args)
         return

@@ -659,6 +659,9 @@ def _linear_args(rows, weight):
     assert a.dim() == 2 and weight.dim() == 2 and a.stride(1) == 1 and weight.stride(1) == 1
     assert a.shape[1] == weight.shape[1] and a.dtype == weight.dtype and a.dtype in (torch.bfloat16, torch.float32)
     dev = _same_device(a, weight)
+    if a.dtype == torch.bfloat16 and (max(a.stride(0), a.shape[1]) % 8 or a.data_ptr() % 16):
+        padded = _rows_empty(*a.shape, a.dtype, dev)  # rows a tensor map cannot express (a latent size that is no multiple of 8)
+        a = padded.copy_(a)
     p = _lib.LinearArgs()
     p.a, p.b = a.data_ptr(), weight.data_ptr()
     p.M, p.K = a.shape

@@ -133,10 +133,10 @@ def test_window_attention(dtype, B, n, hist, heads, dim, vdim, window):
     wide = lambda t: torch.nn.functional.pad(t, (0, -t.shape[1] % 8)).to(DEV)[:, :t.shape[1]]  # pitch of a multiple of 8
     got = K.window_attention(wide(q), wide(k), wide(v), B, heads, dim, vdim, window, scale, sink.to(DEV))
     ref = _window_reference(q, k, v, B, heads, dim, vdim, window, scale, sink)
-    assert (got.double().cpu() - ref).abs().max() < (1e-5 if dtype == torch.float32 else 2.5e-2)
+    assert (got.double().cpu() - ref).abs().max() < (4e-5 if dtype == torch.float32 else 2.5e-2)
     no_sink = K.window_attention(wide(q), wide(k), wide(v), B, heads, dim, vdim, window, scale)
     ref = _window_reference(q, k, v, B, heads, dim, vdim, window, scale, torch.full((heads,), -1e4))
-    assert (no_sink.double().cpu() - ref).abs().max() < (1e-5 if dtype == torch.float32 else 2.5e-2)
+    assert (no_sink.double().cpu() - ref).abs().max() < (4e-5 if dtype == torch.float32 else 2.5e-2)
     _clean()
 
 
@@ -247,7 +247,7 @@ def test_decayed_attention_over_portions(dtype, B, heads, dim, vdim, decay, port
             sl = slice(start, start + part)
             o, ref_state[b] = orc.decayed_linear_attention(q[b, sl].double(), k[b, sl].double(), v[b, sl].double(), lam, ref_state[b])
             ref = orc.rms_norm_plain(o.reshape(part, -1), wn.double(), 1e-2) * g[b, sl].reshape(part, -1).double()
-            assert (got[b].double().cpu() - ref).abs().max() < (2e-5 if dtype == torch.float32 else 4e-2)
+            assert ((got[b].double().cpu() - ref).abs() / (1 + ref.abs())).max() < (6e-5 if dtype == torch.float32 else 1e-2)
             top = ref_state[b].abs().max()
             assert (state[b].double().cpu() - ref_state[b]).abs().max() < 3e-5 * top
         start += part
