@@ -7,8 +7,9 @@ namespace b200 {
 namespace {
 
 // ------------------------------------------------------------------ latents in and out of the cache
-// One warp per new token: RMS norm over R, then to the work rows and, for the last `ring` tokens, to the cache.
-template <typename T>
+// One warp per new token: RMS norm over R, then to the work rows and, for the last `ring` tokens, to the cache.  VEC: rows
+// of up to 1024 elements move as 8-element vectors and stay in registers.
+template <typename T, bool VEC>
 __global__ void __launch_bounds__(256)
 latent_append_kernel(const T* __restrict__ raw, int64_t ld_raw, const float* __restrict__ weight, float eps, T* __restrict__ work,
                      T* __restrict__ cache, int64_t rows, int64_t n_new, int64_t R, int64_t hist, int64_t ring, int64_t start,
@@ -19,6 +20,35 @@ latent_append_kernel(const T* __restrict__ raw, int64_t ld_raw, const float* __r
   const int64_t b = row / n_new, t = row % n_new;
   const int64_t pos = (pos_dev ? (int64_t)pos_dev[0] : start) + t;
   const T* src = raw + row * ld_raw;
+  if constexpr (VEC) {
+    constexpr int NV = 4;
+    T* w = work ? work + (b * (hist + n_new) + hist + t) * R : nullptr;
+    T* k = (cache && t + ring >= n_new && pos >= 0) ? cache + (b * ring + pos % ring) * R : nullptr;
+    float f[NV][8], s = 0.f;
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (i * 32 + lane) * 8;
+      if (c < R) {
+        load8(src + c, f[i]);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) s = fmaf(f[i][e], f[i][e], s);
+      }
+    }
+    const float inv = 1.0f / sqrtf(warp_sum(s) / (float)R + eps);
+#pragma unroll
+    for (int i = 0; i < NV; ++i) {
+      const int c = (i * 32 + lane) * 8;
+      if (c < R) {
+        float g[8];
+        load8(weight + c, g);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) g[e] *= f[i][e] * inv;
+        if (w) store8(w + c, g);
+        if (k) store8(k + c, g);
+      }
+    }
+    return;
+  }
   float s = 0.f;
   for (int64_t c = lane; c < R; c += 32) {
     const float v = to_float(src[c]);
@@ -224,18 +254,25 @@ int window_typed(const void* q, int64_t ld_q, const void* k, int64_t ld_k, const
 
 }  // namespace
 
-int launch_latent_append(const void* raw, int64_t ld_raw, const float* weight, float eps, void* work, void* cache, int64_t B, int64_t n_new, int64_t R,
-                         int64_t hist, int64_t ring, int64_t start, const int* pos_dev, int dtype, cudaStream_t stream) {
+template <typename T>
+static int append_typed(const void* raw, int64_t ld_raw, const float* weight, float eps, void* work, void* cache, int64_t B, int64_t n_new, int64_t R,
+                        int64_t hist, int64_t ring, int64_t start, const int* pos_dev, cudaStream_t stream) {
   const int64_t rows = B * n_new, blocks = (rows + 7) / 8;
   if (blocks > 0x7fffffffLL) return B200_ERR_BAD_ARGUMENT;
-  if (dtype == B200_BF16)
-    latent_append_kernel<__nv_bfloat16><<<(unsigned)blocks, 256, 0, stream>>>((const __nv_bfloat16*)raw, ld_raw, weight, eps, (__nv_bfloat16*)work,
-                                                                              (__nv_bfloat16*)cache, rows, n_new, R, hist, ring, start, pos_dev);
+  const bool vec = R <= 1024 && R % 8 == 0 && ld_raw % 8 == 0 &&
+                   ((reinterpret_cast<uintptr_t>(raw) | reinterpret_cast<uintptr_t>(weight) | reinterpret_cast<uintptr_t>(work) | reinterpret_cast<uintptr_t>(cache)) & 15) == 0;
+  if (vec)
+    latent_append_kernel<T, true><<<(unsigned)blocks, 256, 0, stream>>>((const T*)raw, ld_raw, weight, eps, (T*)work, (T*)cache, rows, n_new, R, hist, ring, start, pos_dev);
   else
-    latent_append_kernel<float><<<(unsigned)blocks, 256, 0, stream>>>((const float*)raw, ld_raw, weight, eps, (float*)work, (float*)cache, rows, n_new, R,
-                                                                      hist, ring, start, pos_dev);
+    latent_append_kernel<T, false><<<(unsigned)blocks, 256, 0, stream>>>((const T*)raw, ld_raw, weight, eps, (T*)work, (T*)cache, rows, n_new, R, hist, ring, start, pos_dev);
   note_launches(1);
   return status_from_cuda(cudaGetLastError());
+}
+
+int launch_latent_append(const void* raw, int64_t ld_raw, const float* weight, float eps, void* work, void* cache, int64_t B, int64_t n_new, int64_t R,
+                         int64_t hist, int64_t ring, int64_t start, const int* pos_dev, int dtype, cudaStream_t stream) {
+  return dtype == B200_BF16 ? append_typed<__nv_bfloat16>(raw, ld_raw, weight, eps, work, cache, B, n_new, R, hist, ring, start, pos_dev, stream)
+                            : append_typed<float>(raw, ld_raw, weight, eps, work, cache, B, n_new, R, hist, ring, start, pos_dev, stream);
 }
 
 int launch_latent_gather(const void* cache, void* work, int64_t B, int64_t n_new, int64_t R, int64_t hist, int64_t ring, int64_t start, int dtype,

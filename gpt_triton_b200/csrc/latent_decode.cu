@@ -3,7 +3,8 @@
 //   head_product_kernel   q~ = W_uk[head]^T q  before, and  W_uv[head] o~  after: one small product per head
 //   latent_stream_kernel  scores q~ . c, online softmax and the weighted latent sum o~ over a range of the window
 //   latent_merge_kernel   merges the ranges of one (sequence, head), adds the sink's term, normalises
-// q~ and the softmax weights are fp32 by definition; they enter the MMAs as two bf16 parts each.
+// q~ is the output of a product, in bf16 like every other; the softmax weights are fp32 by definition and enter their MMA
+// as two bf16 parts.
 #include <atomic>
 
 #include "mma_sync.cuh"
@@ -16,10 +17,10 @@ using namespace warp_mma;
 // ------------------------------------------------------------------ one product per head
 // out[b, h, n] = sum_k a[b, h, k] * w[h, n, k] (K_MAJOR) or w[h, k, n].  Tile: 16 * MB sequences x 64 columns; MB = 1: the
 // four warps take 16 columns each, MB = 4: 16 sequences each.  k, n multiples of 8.
-template <bool K_MAJOR, int MB, typename OutT>
+template <bool K_MAJOR, int MB>
 __global__ void __launch_bounds__(128)
 head_product_kernel(const __nv_bfloat16* __restrict__ a, int64_t lda, int64_t a_head, const __nv_bfloat16* __restrict__ w, int64_t w_head, int64_t ldw,
-                    OutT* __restrict__ out, int64_t ld_out, int64_t out_head, int B, int N, int K) {
+                    __nv_bfloat16* __restrict__ out, int64_t ld_out, int64_t out_head, int B, int N, int K) {
   constexpr int ROWS = 16 * MB, NT = MB == 1 ? 2 : 8;
   __shared__ __align__(128) uint8_t tiles[2][(ROWS + 64) * 128];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g8 = lane >> 2, t4 = lane & 3;
@@ -77,53 +78,50 @@ head_product_kernel(const __nv_bfloat16* __restrict__ a, int64_t lda, int64_t a_
     for (int r = 0; r < 2; ++r) {
       const int b = b0 + row_w + g8 + r * 8, n = n0 + col_w + nt * 8 + t4 * 2;
       if (b < B && n < N) {
-        OutT* p = out + (int64_t)b * ld_out + n;
-        p[0] = from_float<OutT>(acc[nt][2 * r]), p[1] = from_float<OutT>(acc[nt][2 * r + 1]);
+        *reinterpret_cast<__nv_bfloat162*>(out + (int64_t)b * ld_out + n) = __floats2bfloat162_rn(acc[nt][2 * r], acc[nt][2 * r + 1]);
       }
     }
 }
 
 // ------------------------------------------------------------------ streaming the latents
-constexpr int kHeads = 16, kKeys = 64, kStreamThreads = 256;
+constexpr int kHeads = 16, kKeys = 32, kStreamThreads = 128, kStreamCtasPerSm = 2;
+static_assert(kKeys == 8 * kStreamThreads / 32, "a warp scores eight keys of a tile");
 
 template <int RP>  // latent size, padded to 128, 256 or 512
 struct StreamSmem {
   static constexpr int ROW = RP * 2;
   static constexpr int C_BYTES = kKeys * ROW;
   static constexpr int Q_BYTES = kHeads * ROW;
-  static constexpr int P_BYTES = kHeads * kKeys * 2;
-  static constexpr int BYTES = 2 * C_BYTES + 2 * Q_BYTES + 2 * P_BYTES;
+  static constexpr int P_BYTES = kHeads * 128;  // one bf16 part of the weights; rows of 128 bytes, kKeys * 2 of them used
+  static constexpr int BYTES = 2 * C_BYTES + Q_BYTES + 2 * P_BYTES;
 };
 
 // blockIdx.x = sequence, y = group of 16 heads, z = range of the window.  Partial results per (sequence, head, range):
 // part_ml = (maximum in log2 units, denominator), part_o = unnormalised sum of latents.
 template <int RP>
-__global__ void __launch_bounds__(kStreamThreads)
-latent_stream_kernel(const float* __restrict__ qt, const __nv_bfloat16* __restrict__ cache, float* __restrict__ part_o, float2* __restrict__ part_ml,
+__global__ void __launch_bounds__(kStreamThreads, kStreamCtasPerSm)
+latent_stream_kernel(const __nv_bfloat16* __restrict__ qt, const __nv_bfloat16* __restrict__ cache, float* __restrict__ part_o, float2* __restrict__ part_ml,
                      int heads, int R, int64_t ring, int64_t window, float scale_log2e, const int* __restrict__ pos_dev) {
   using M = StreamSmem<RP>;
-  constexpr int ROW = M::ROW, NT = RP / 64;  // 8-column output tiles per warp (eight warps)
+  constexpr int WARPS = kStreamThreads / 32;
+  constexpr int ROW = M::ROW, NT = RP / 8 / WARPS;  // 8-column output tiles per warp
   extern __shared__ __align__(128) uint8_t smem[];
-  __shared__ float s_max[8][kHeads], s_sum[8][kHeads];
+  __shared__ float s_max[WARPS][kHeads], s_sum[WARPS][kHeads];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g8 = lane >> 2, t4 = lane & 3;
   const int64_t b = blockIdx.x;
   const int h0 = blockIdx.y * kHeads, split = blockIdx.z, n_split = gridDim.z;
   const uint32_t base = (uint32_t)__cvta_generic_to_shared(smem);
-  const uint32_t q_hi = base + 2 * M::C_BYTES, q_lo = q_hi + M::Q_BYTES, p_hi = q_lo + M::Q_BYTES, p_lo = p_hi + M::P_BYTES;
+  const uint32_t sq = base + 2 * M::C_BYTES, p_hi = sq + M::Q_BYTES, p_lo = p_hi + M::P_BYTES;
   const int64_t pos = pos_dev[0], first = pos + 1 > window ? pos + 1 - window : 0;
   const int n_keys = pos < 0 ? 0 : (int)(pos - first + 1);
   const int tiles = (n_keys + kKeys - 1) / kKeys, per = (tiles + n_split - 1) / n_split;
   const int tile0 = split * per, tile1 = min(tiles, tile0 + per);
 
-  for (int i = threadIdx.x; i < kHeads * (RP / 2); i += kStreamThreads) {
-    const int r = i / (RP / 2), c = (i % (RP / 2)) * 2;
-    float2 v = make_float2(0.f, 0.f);
-    if (h0 + r < heads && c < R) v = *reinterpret_cast<const float2*>(qt + (b * heads + h0 + r) * R + c);
-    uint32_t hi, lo;
-    split_pair(v.x, v.y, hi, lo);
-    const uint32_t at = swz<ROW>(r, c >> 3) + (c & 7) * 2;
-    asm volatile("st.shared.b32 [%0], %1;" ::"r"(q_hi + at), "r"(hi) : "memory");
-    asm volatile("st.shared.b32 [%0], %1;" ::"r"(q_lo + at), "r"(lo) : "memory");
+  // (lands together with the first tile of latents)
+  for (int i = threadIdx.x; i < kHeads * (RP / 8); i += kStreamThreads) {
+    const int r = i / (RP / 8), c = i % (RP / 8);
+    const bool ok = h0 + r < heads && c * 8 < R;
+    cp_async16(sq + swz<ROW>(r, c), ok ? qt + (b * heads + h0 + r) * R + c * 8 : qt, ok);
   }
   const __nv_bfloat16* cb = cache + b * ring * R;
   const int64_t slot0 = first % ring;
@@ -157,17 +155,16 @@ latent_stream_kernel(const float* __restrict__ qt, const __nv_bfloat16* __restri
     __syncthreads();
     const uint32_t sc = base + stage * M::C_BYTES;
     // scores of 16 heads x this warp's 8 keys
-    float s[4] = {0.f, 0.f, 0.f, 0.f};
+    float s[4] = {0.f, 0.f, 0.f, 0.f}, s1[4] = {0.f, 0.f, 0.f, 0.f};
 #pragma unroll 8
     for (int ks = 0; ks < RP / 16; ++ks) {
-      uint32_t qh[4], ql[4], cf[2];
-      const uint32_t at = swz<ROW>(lane & 15, ks * 2 + (lane >> 4));
-      ldsm4(qh, q_hi + at);
-      ldsm4(ql, q_lo + at);
+      uint32_t qf[4], cf[2];
+      ldsm4(qf, sq + swz<ROW>(lane & 15, ks * 2 + (lane >> 4)));
       ldsm2(cf, sc + swz<ROW>(warp * 8 + (lane & 7), ks * 2 + ((lane >> 3) & 1)));
-      mma_bf16(s, qh, cf[0], cf[1]);
-      mma_bf16(s, ql, cf[0], cf[1]);
+      mma_bf16(ks & 1 ? s1 : s, qf, cf[0], cf[1]);
     }
+#pragma unroll
+    for (int i = 0; i < 4; ++i) s[i] += s1[i];
     const int key = tile * kKeys + warp * 8 + t4 * 2;
     float bm[2];
 #pragma unroll
@@ -185,7 +182,7 @@ latent_stream_kernel(const float* __restrict__ qt, const __nv_bfloat16* __restri
     for (int r = 0; r < 2; ++r) {
       float m_new = m_run[r];
 #pragma unroll
-      for (int w2 = 0; w2 < 8; ++w2) m_new = fmaxf(m_new, s_max[w2][g8 + r * 8]);  // finite: a tile has at least one key
+      for (int w2 = 0; w2 < WARPS; ++w2) m_new = fmaxf(m_new, s_max[w2][g8 + r * 8]);  // finite: a tile has at least one key
       mult[r] = exp2f(m_run[r] - m_new);
       m_run[r] = m_new;
       const float p0 = exp2f(s[2 * r] - m_new), p1 = exp2f(s[2 * r + 1] - m_new);
@@ -204,12 +201,12 @@ latent_stream_kernel(const float* __restrict__ qt, const __nv_bfloat16* __restri
     for (int r = 0; r < 2; ++r) {
       float ps = 0.f;
 #pragma unroll
-      for (int w2 = 0; w2 < 8; ++w2) ps += s_sum[w2][g8 + r * 8];
+      for (int w2 = 0; w2 < WARPS; ++w2) ps += s_sum[w2][g8 + r * 8];
       l_run[r] = l_run[r] * mult[r] + ps;
     }
 #pragma unroll
     for (int i = 0; i < NT; ++i) o[i][0] *= mult[0], o[i][1] *= mult[0], o[i][2] *= mult[1], o[i][3] *= mult[1];
-    // o~ += P c for this warp's RP / 8 columns
+    // o~ += P c for this warp's RP / WARPS columns
 #pragma unroll
     for (int kk = 0; kk < kKeys / 16; ++kk) {
       uint32_t ph[4], pl[4];
@@ -227,6 +224,8 @@ latent_stream_kernel(const float* __restrict__ qt, const __nv_bfloat16* __restri
       }
     }
   }
+  cp_async_commit();
+  cp_async_wait<0>();  // (a block without tiles still has its queries in flight)
 #pragma unroll
   for (int r = 0; r < 2; ++r) {
     const int h = h0 + g8 + r * 8;
@@ -242,27 +241,43 @@ latent_stream_kernel(const float* __restrict__ qt, const __nv_bfloat16* __restri
 }
 
 // One block per (sequence, head).
+constexpr int kMaxSplit = 64;
 __global__ void __launch_bounds__(128)
 latent_merge_kernel(const float* __restrict__ part_o, const float2* __restrict__ part_ml, __nv_bfloat16* __restrict__ ot, int heads, int R, int n_split,
                     const float* __restrict__ sink) {
+  __shared__ float factor[kMaxSplit];
   const int64_t item = blockIdx.x;
-  const int h = (int)(item % heads);
-  float m = -INFINITY;
-  for (int s = 0; s < n_split; ++s) m = fmaxf(m, part_ml[item * n_split + s].x);
-  float l = 0.f;
-  for (int s = 0; s < n_split; ++s) {
-    const float2 ml = part_ml[item * n_split + s];
-    l = fmaf(ml.y, exp2f(ml.x - m), l);
-  }
-  if (sink) l += exp2f(sink[h] * 1.4426950408889634f - m);
-  const float inv = 1.0f / l;
-  for (int r = threadIdx.x; r < R; r += 128) {
-    float v = 0.f;
-    for (int s = 0; s < n_split; ++s) {
-      const float f = exp2f(part_ml[item * n_split + s].x - m);
-      if (f > 0.f) v = fmaf(part_o[(item * n_split + s) * R + r], f, v);
+  const int h = (int)(item % heads), lane = threadIdx.x & 31;
+  if (threadIdx.x < 32) {
+    float2 ml[kMaxSplit / 32];
+    float m = -INFINITY, l = 0.f;
+#pragma unroll
+    for (int i = 0; i < kMaxSplit / 32; ++i) {
+      const int s = i * 32 + lane;
+      ml[i] = s < n_split ? part_ml[item * n_split + s] : make_float2(-INFINITY, 0.f);
+      m = fmaxf(m, ml[i].x);
     }
-    ot[item * R + r] = __float2bfloat16_rn(v * inv);
+#pragma unroll
+    for (int o = 16; o > 0; o >>= 1) m = fmaxf(m, __shfl_xor_sync(0xffffffffu, m, o));
+#pragma unroll
+    for (int i = 0; i < kMaxSplit / 32; ++i) l = fmaf(ml[i].y, exp2f(ml[i].x - m), l);
+    l = warp_sum(l);
+    if (sink) l += exp2f(sink[h] * 1.4426950408889634f - m);
+    const float inv = 1.0f / l;
+#pragma unroll
+    for (int i = 0; i < kMaxSplit / 32; ++i) factor[i * 32 + lane] = exp2f(ml[i].x - m) * inv;
+  }
+  __syncthreads();
+  for (int r = threadIdx.x * 4; r < R; r += 512) {  // (R is a multiple of 8)
+    float4 v = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll 4
+    for (int s = 0; s < n_split; ++s) {
+      const float f = factor[s];
+      const float4 o = *reinterpret_cast<const float4*>(part_o + (item * n_split + s) * R + r);
+      v.x = fmaf(o.x, f, v.x), v.y = fmaf(o.y, f, v.y), v.z = fmaf(o.z, f, v.z), v.w = fmaf(o.w, f, v.w);
+    }
+    __nv_bfloat162 lo = __floats2bfloat162_rn(v.x, v.y), hi = __floats2bfloat162_rn(v.z, v.w);
+    *reinterpret_cast<uint2*>(ot + item * R + r) = make_uint2(*reinterpret_cast<uint32_t*>(&lo), *reinterpret_cast<uint32_t*>(&hi));
   }
 }
 
@@ -275,12 +290,16 @@ struct Plan {
 Plan make_plan(int64_t B, int64_t heads, int64_t R, int64_t window) {
   Plan p;
   const int64_t groups = B * ((heads + kHeads - 1) / kHeads), tiles = (window + kKeys - 1) / kKeys;
-  int64_t n = (sm_count() + groups - 1) / groups;
-  if (n > tiles) n = tiles;
-  if (n > 64) n = 64;
-  if (n < 1) n = 1;
+  // ranges per sequence: the fewest rounds of blocks, counted in tiles (a block's start-up and its share of the merge are
+  // worth about three)
+  const int64_t slots = (int64_t)sm_count() * kStreamCtasPerSm;
+  int64_t n = 1, best = -1;
+  for (int64_t k = 1; k <= tiles && k <= kMaxSplit; ++k) {
+    const int64_t cost = ((groups * k + slots - 1) / slots) * ((tiles + k - 1) / k + 3);
+    if (best < 0 || cost < best) best = cost, n = k;
+  }
   p.n_split = (int)n;
-  size_t at = round256((size_t)(B * heads * R) * 4);  // q~
+  size_t at = round256((size_t)(B * heads * R) * 2);  // q~
   p.off_po = at, at += round256((size_t)(B * heads * n * R) * 4);
   p.off_ml = at, at += round256((size_t)(B * heads * n) * 8);
   p.off_ot = at, at += round256((size_t)(B * heads * R) * 2);
@@ -289,7 +308,7 @@ Plan make_plan(int64_t B, int64_t heads, int64_t R, int64_t window) {
 }
 
 template <int RP>
-int launch_stream(const float* qt, const void* cache, float* po, float2* ml, int64_t B, int64_t heads, int64_t R, int64_t ring, int64_t window,
+int launch_stream(const __nv_bfloat16* qt, const void* cache, float* po, float2* ml, int64_t B, int64_t heads, int64_t R, int64_t ring, int64_t window,
                   float scale, int n_split, const int* pos_dev, cudaStream_t stream) {
   constexpr int smem = StreamSmem<RP>::BYTES;
   static std::atomic<bool> attr_set[kMaxDevices];
@@ -305,14 +324,14 @@ int launch_stream(const float* qt, const void* cache, float* po, float2* ml, int
   return status_from_cuda(cudaGetLastError());
 }
 
-template <bool K_MAJOR, typename OutT>
-void head_product(const __nv_bfloat16* a, int64_t lda, int64_t a_head, const __nv_bfloat16* w, int64_t w_head, int64_t ldw, OutT* out, int64_t ld_out,
+template <bool K_MAJOR>
+void head_product(const __nv_bfloat16* a, int64_t lda, int64_t a_head, const __nv_bfloat16* w, int64_t w_head, int64_t ldw, __nv_bfloat16* out, int64_t ld_out,
                   int64_t out_head, int64_t B, int64_t heads, int64_t N, int64_t K, cudaStream_t stream) {
   const unsigned nb = (unsigned)((N + 63) / 64);
   if (B <= 16)
-    head_product_kernel<K_MAJOR, 1, OutT><<<dim3(nb, (unsigned)heads, 1), 128, 0, stream>>>(a, lda, a_head, w, w_head, ldw, out, ld_out, out_head, (int)B, (int)N, (int)K);
+    head_product_kernel<K_MAJOR, 1><<<dim3(nb, (unsigned)heads, 1), 128, 0, stream>>>(a, lda, a_head, w, w_head, ldw, out, ld_out, out_head, (int)B, (int)N, (int)K);
   else
-    head_product_kernel<K_MAJOR, 4, OutT><<<dim3(nb, (unsigned)heads, (unsigned)((B + 63) / 64)), 128, 0, stream>>>(a, lda, a_head, w, w_head, ldw, out, ld_out,
+    head_product_kernel<K_MAJOR, 4><<<dim3(nb, (unsigned)heads, (unsigned)((B + 63) / 64)), 128, 0, stream>>>(a, lda, a_head, w, w_head, ldw, out, ld_out,
                                                                                                                     out_head, (int)B, (int)N, (int)K);
   note_launches(1);
 }
@@ -328,22 +347,22 @@ size_t latent_decode_mma_workspace_bytes(int64_t B, int64_t heads, int64_t R, in
 int launch_latent_decode_mma(const void* q, int64_t ld_q, const void* w_uk, const void* w_uv, const void* cache, void* out, int64_t ld_out, int64_t B,
                              int64_t heads, int64_t dim, int64_t vdim, int64_t R, int64_t ring, int64_t window, float scale, const float* sink,
                              const int* pos_dev, void* workspace, cudaStream_t stream) {
-  if (R > 512 || R % 8 || dim % 8 || vdim % 8 || ld_q % 8 || !aligned16_all(q, w_uk, w_uv, cache)) return B200_ERR_UNSUPPORTED;
+  if (R > 512 || R % 8 || dim % 8 || vdim % 8 || ld_q % 8 || ld_out % 2 || (reinterpret_cast<uintptr_t>(out) & 3) || !aligned16_all(q, w_uk, w_uv, cache)) return B200_ERR_UNSUPPORTED;
   if (B > 65535 || heads > 65535 || window > (1 << 30)) return B200_ERR_UNSUPPORTED;
   const Plan p = make_plan(B, heads, R, window);
   uint8_t* ws = static_cast<uint8_t*>(workspace);
-  float* qt = reinterpret_cast<float*>(ws);
+  __nv_bfloat16* qt = reinterpret_cast<__nv_bfloat16*>(ws);
   float* po = reinterpret_cast<float*>(ws + p.off_po);
   float2* ml = reinterpret_cast<float2*>(ws + p.off_ml);
   __nv_bfloat16* ot = reinterpret_cast<__nv_bfloat16*>(ws + p.off_ot);
-  head_product<false, float>((const __nv_bfloat16*)q, ld_q, dim, (const __nv_bfloat16*)w_uk, dim * R, R, qt, heads * R, R, B, heads, R, dim, stream);
+  head_product<false>((const __nv_bfloat16*)q, ld_q, dim, (const __nv_bfloat16*)w_uk, dim * R, R, qt, heads * R, R, B, heads, R, dim, stream);
   int st = R <= 128   ? launch_stream<128>(qt, cache, po, ml, B, heads, R, ring, window, scale, p.n_split, pos_dev, stream)
            : R <= 256 ? launch_stream<256>(qt, cache, po, ml, B, heads, R, ring, window, scale, p.n_split, pos_dev, stream)
                       : launch_stream<512>(qt, cache, po, ml, B, heads, R, ring, window, scale, p.n_split, pos_dev, stream);
   if (st != B200_OK) return st;
   latent_merge_kernel<<<(unsigned)(B * heads), 128, 0, stream>>>(po, ml, ot, (int)heads, (int)R, p.n_split, sink);
   note_launches(1);
-  head_product<true, __nv_bfloat16>(ot, heads * R, R, (const __nv_bfloat16*)w_uv, vdim * R, R, (__nv_bfloat16*)out, ld_out, vdim, B, heads, vdim, R, stream);
+  head_product<true>(ot, heads * R, R, (const __nv_bfloat16*)w_uv, vdim * R, R, (__nv_bfloat16*)out, ld_out, vdim, B, heads, vdim, R, stream);
   return status_from_cuda(cudaGetLastError());
 }
 

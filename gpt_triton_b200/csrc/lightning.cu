@@ -1,7 +1,7 @@
 // Decayed linear attention: per head S <- decay * S + k v^T, o = S^T q with an fp32 state, over one token or many.
 //
 // recurrent kernel: token by token, exactly the recurrence, any sizes, both storage types.  A block owns 32 columns of
-// one head's state in registers (four warps split the rows); tokens are staged 16 at a time in shared memory.
+// one head's state in registers (four warps split the rows); tokens are staged a few at a time in shared memory.
 //
 // chunked kernel (bf16, many tokens): 64 tokens at a time on the tensor cores.  With the state S before a chunk and
 // i, j = 0..63 inside it,
@@ -21,13 +21,14 @@ namespace {
 
 using namespace warp_mma;
 
-constexpr int kCols = 32, kRowWarps = 4, kTokens = 16;
+constexpr int kCols = 32, kRowWarps = 4;
 
 template <typename T, int RPW>  // RPW: state rows per warp
 __global__ void __launch_bounds__(32 * kRowWarps)
 recurrent_kernel(const T* __restrict__ qkvg, int64_t ld, int64_t off_k, int64_t off_v, int64_t off_g, const double* __restrict__ decay,
                  const float* __restrict__ weight, float* __restrict__ state, int fresh, T* __restrict__ y, int64_t ld_y, float* __restrict__ sumsq,
                  int64_t ld_sumsq, int n_tok, int heads, int dim, int vdim) {
+  constexpr int kTokens = RPW <= 64 ? 16 : 4;  // tokens staged at a time
   __shared__ __align__(16) float qs[kTokens][RPW * kRowWarps], ks[kTokens][RPW * kRowWarps];
   __shared__ float vs[kTokens][kCols];
   __shared__ float part[kTokens][kRowWarps][kCols];
@@ -115,6 +116,7 @@ int launch_recurrent(const Args& a, cudaStream_t stream) {
   else if (a.dim <= 64) B200_RECURRENT(16);
   else if (a.dim <= 128) B200_RECURRENT(32);
   else if (a.dim <= 256) B200_RECURRENT(64);
+  else if (a.dim <= 512) B200_RECURRENT(128);
   else return B200_ERR_UNSUPPORTED;
 #undef B200_RECURRENT
   note_launches(1);

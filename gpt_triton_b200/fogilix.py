@@ -112,6 +112,12 @@ class Fogilix(GeneratesTokens, _EvalOnly):
         name = tensor.replace("final.norm", "final_norm").replace("dkv.norm", "dkv_norm")
         return "layers." + name[1:] if name[:1] == "l" and name[1:2].isdigit() else name
 
+    @staticmethod
+    def tensor_name(parameter):
+        """The other way round."""
+        name = parameter.replace("final_norm", "final.norm").replace("dkv_norm", "dkv.norm")
+        return "l" + name.removeprefix("layers.") if name.startswith("layers.") else name
+
     @classmethod
     def from_checkpoint(cls, config, tensors):
         """config: the parsed config.json; tensors: name -> tensor of model.safetensors."""

@@ -123,7 +123,8 @@ def _window_reference(q, k, v, B, heads, dim, vdim, window, scale, sink):
 @pytest.mark.parametrize("B,n,hist,heads,dim,vdim,window", [
     (1, 1, 0, 1, 16, 16, 1), (2, 7, 0, 3, 10, 6, 3), (1, 70, 0, 2, 32, 48, 1), (2, 65, 12, 3, 64, 64, 13), (1, 130, 63, 2, 64, 32, 64),
     (1, 129, 64, 5, 40, 64, 65), (1, 200, 0, 2, 128, 128, 64), (2, 300, 127, 2, 96, 128, 128), (1, 2, 99, 4, 128, 72, 100), (1, 333, 0, 3, 24, 24, 1000),
-    (1, 260, 5, 1, 72, 8, 6), (3, 128, 0, 2, 64, 64, 2)])
+    (1, 260, 5, 1, 72, 8, 6), (3, 128, 0, 2, 64, 64, 2),
+    (1, 90, 17, 2, 160, 200, 30), (1, 1100, 0, 2, 64, 128, 400)])
 def test_window_attention(dtype, B, n, hist, heads, dim, vdim, window):
     from gpt_triton_b200 import kernels as K
 
@@ -217,7 +218,7 @@ def test_latent_decode(dtype, B, heads, dim, vdim, R, ring, window, pos):
 # ------------------------------------------------------------------ decayed linear attention
 @pytest.mark.parametrize("dtype", DTYPES)
 @pytest.mark.parametrize("B,heads,dim,vdim,decay", [(1, 2, 32, 32, (0.2, 0.999)), (2, 3, 24, 40, (0.5, 0.9, 1.0)), (1, 2, 10, 14, (0.3, 0.99)), (1, 1, 128, 136, (0.9999,)),
-                                                    (2, 2, 72, 64, (0.05, 0.98)), (1, 1, 200, 24, (0.9,))])
+                                                    (2, 2, 72, 64, (0.05, 0.98)), (1, 1, 200, 24, (0.9,)), (1, 1, 320, 40, (0.95,))])
 @pytest.mark.parametrize("portions", [(1, 1, 1), (5, 1, 31), (32, 2, 64), (65, 63, 1, 70), (600, 40, 257)])
 def test_decayed_attention_over_portions(dtype, B, heads, dim, vdim, decay, portions):
     """Any cut of the tokens gives the recurrence's outputs and state (600 tokens of one sequence run in segments)."""
@@ -296,6 +297,27 @@ def test_any_cut_of_a_prompt_gives_the_same_logits(name, dtype, portions):
             at, i = at + n, i + 1
         assert relative_error(torch.cat(got), ref).max() < MODEL_TOL[dtype]
         session.reset()
+    _clean()
+
+
+@pytest.mark.parametrize("dtype", DTYPES)
+def test_a_long_prompt_with_wide_heads(dtype):
+    """Enough rows for the persistent GEMM, heads of 128, several segments of the chunked recurrence, windows that reach
+    across query tiles; whole, and cut once where the second part has a full window of history."""
+    from gpt_triton_b200.generation import GenerationSession
+
+    cfg = config(520, 384, [lightning(2, 128, 128, [0.8, 0.9995], ff=640), latent(3, 128, 96, 136, 190), latent(2, 112, 128, 136, 257, kv_from=1, ff=520)])
+    w = weights(cfg, seed=12)
+    model = build(cfg, w, dtype)
+    ids = tokens(cfg, 1300, seed=4)
+    ref = oracle_logits(cfg, w, ids)
+    got = model.logits(ids[None].to(DEV))[0]
+    assert relative_error(got, ref).max() < MODEL_TOL[dtype]
+    session = GenerationSession(model, 1, 1300)
+    cut = []
+    for lo, hi in ((0, 611), (611, 1300)):
+        cut.append(model.head_logits(session.extend(ids[None, lo:hi].to(DEV), torch.arange(hi - lo, device=DEV))))
+    assert relative_error(torch.cat(cut), ref).max() < MODEL_TOL[dtype]
     _clean()
 
 
