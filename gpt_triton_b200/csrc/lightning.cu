@@ -24,7 +24,7 @@ using namespace warp_mma;
 constexpr int kCols = 32, kRowWarps = 4;
 
 template <typename T, int RPW>  // RPW: state rows per warp
-__global__ void __launch_bounds__(32 * kRowWarps)
+__global__ void __launch_bounds__(32 * kRowWarps, RPW <= 32 ? 5 : 1)
 recurrent_kernel(const T* __restrict__ qkvg, int64_t ld, int64_t off_k, int64_t off_v, int64_t off_g, const double* __restrict__ decay,
                  const float* __restrict__ weight, float* __restrict__ state, int fresh, T* __restrict__ y, int64_t ld_y, float* __restrict__ sumsq,
                  int64_t ld_sumsq, int n_tok, int heads, int dim, int vdim) {
@@ -148,6 +148,7 @@ chunked_kernel(const __nv_bfloat16* __restrict__ qkvg, int64_t ld, int64_t off_k
   constexpr int QROW = DIM * 2, VROW = kVCols * 2;
   extern __shared__ __align__(128) uint8_t smem[];
   __shared__ float pw[kChunk + 1];  // powers of the decay
+  __shared__ float ws[kVCols];      // norm weights of this block's columns
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g8 = lane >> 2, t4 = lane & 3;
   const int vblocks = (vdim + kVCols - 1) / kVCols;
   const int vb = blockIdx.x % vblocks, h = (blockIdx.x / vblocks) % heads;
@@ -156,6 +157,7 @@ chunked_kernel(const __nv_bfloat16* __restrict__ qkvg, int64_t ld, int64_t off_k
   const int seg = blockIdx.y, tok0 = seg * seg_len, tok1 = min(n_tok, tok0 + seg_len);
   const uint32_t base = (uint32_t)__cvta_generic_to_shared(smem);
   const uint32_t s_hi = base + 2 * M::STAGE_BYTES, s_lo = s_hi + M::S_BYTES;
+  if (threadIdx.x < kVCols) ws[threadIdx.x] = OUTPUT && c0 + threadIdx.x < vdim ? weight[h * vdim + c0 + threadIdx.x] : 0.f;
   if (threadIdx.x <= kChunk) pw[threadIdx.x] = (float)pow(decay[h], (double)threadIdx.x);
 
   const __nv_bfloat16* rows = qkvg + b * n_tok * ld;
@@ -251,6 +253,15 @@ chunked_kernel(const __nv_bfloat16* __restrict__ qkvg, int64_t ld, int64_t off_k
         }
       }
       const int i0 = warp * 16 + g8;
+      // gates of this thread's outputs, on their way while the scores are applied (pairs of columns; vdim is a multiple of 8)
+      uint32_t gate[2][8];
+#pragma unroll
+      for (int r = 0; r < 2; ++r) {
+        const __nv_bfloat16* src = qkvg + (b * n_tok + t0 + i0 + r * 8) * ld + off_g + (int64_t)h * vdim + c0 + t4 * 2;
+#pragma unroll
+        for (int nt = 0; nt < 8; ++nt)
+          gate[r][nt] = i0 + r * 8 < n && c0 + nt * 8 < vdim ? __ldg(reinterpret_cast<const unsigned int*>(src + nt * 8)) : 0u;
+      }
       const float p0 = pw[i0 + 1], p1 = pw[i0 + 9];
 #pragma unroll
       for (int nt = 0; nt < 8; ++nt) {
@@ -289,14 +300,12 @@ chunked_kernel(const __nv_bfloat16* __restrict__ qkvg, int64_t ld, int64_t off_k
         if (t < n) {
 #pragma unroll
           for (int nt = 0; nt < 8; ++nt) {
-            const int c = c0 + nt * 8 + t4 * 2;  // (vdim is a multiple of 8)
-            if (c < vdim) {
-              const int64_t col = (int64_t)h * vdim + c;
-              const float2 w = *reinterpret_cast<const float2*>(weight + col);
-              const float2 gt = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(qkvg + row * ld + off_g + col));
+            const int c = nt * 8 + t4 * 2;
+            if (c0 + c < vdim) {
+              const float2 gt = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(&gate[r][nt]));
               const float o0 = o[nt][2 * r], o1 = o[nt][2 * r + 1];
               sq2 = fmaf(o0, o0, fmaf(o1, o1, sq2));
-              *reinterpret_cast<__nv_bfloat162*>(y + row * ld_y + col) = __floats2bfloat162_rn(o0 * w.x * gt.x, o1 * w.y * gt.y);
+              *reinterpret_cast<__nv_bfloat162*>(y + row * ld_y + (int64_t)h * vdim + c0 + c) = __floats2bfloat162_rn(o0 * ws[c] * gt.x, o1 * ws[c + 1] * gt.y);
             }
           }
         }
@@ -379,11 +388,18 @@ segment_scan_kernel(const float* __restrict__ state, int fresh, float* __restric
 bool takes_chunks(int64_t n_tok, int64_t dim, int64_t vdim, int dtype) {
   return dtype == B200_BF16 && n_tok >= kChunk / 2 && dim <= 128 && dim % 8 == 0 && vdim % 8 == 0;
 }
-// Segments per sequence: enough blocks for two per SM, at least four chunks each.
+// Segments per sequence: the fewest rounds of blocks (two per SM), counted in chunks; the first pass over all but the last
+// segment costs about 0.4 of a full one, and extra launches a few chunks.
 int64_t segment_count(int64_t B, int64_t n_tok, int64_t heads, int64_t vdim) {
-  const int64_t blocks = B * heads * ((vdim + kVCols - 1) / kVCols), want = ((int64_t)sm_count() * 2 + blocks - 1) / blocks;
-  const int64_t most = n_tok / (4 * kChunk);
-  return want < 2 || most < 2 ? 1 : (want < most ? want : most);
+  const int64_t blocks = B * heads * ((vdim + kVCols - 1) / kVCols), slots = (int64_t)sm_count() * 2, chunks = (n_tok + kChunk - 1) / kChunk;
+  auto rounds = [&](int64_t n) { return (double)((blocks * n + slots - 1) / slots); };
+  int64_t best = 1;
+  double cost = rounds(1) * chunks;
+  for (int64_t n = 2; n <= 64 && n * 4 <= chunks; ++n) {
+    const double per = (double)((chunks + n - 1) / n), c = rounds(n) * per + 0.4 * rounds(n - 1) * per + 3.0;
+    if (c < cost) cost = c, best = n;
+  }
+  return best;
 }
 
 template <int DIM>
@@ -400,7 +416,7 @@ int launch_chunked(const Args& a, void* workspace, cudaStream_t stream) {
   }
   const int64_t blocks = a.B * a.heads * ((a.vdim + kVCols - 1) / kVCols);
   if (blocks > 0x7fffffffLL || a.n_tok > 0x7fffffffLL - kChunk) return B200_ERR_BAD_ARGUMENT;
-  int64_t n_seg = segment_count(a.B, a.n_tok, a.heads, a.vdim);
+  int64_t n_seg = segment_count(a.B, a.n_tok, a.heads, a.vdim);  // (the workspace is sized for this many)
   const int64_t chunks = (a.n_tok + kChunk - 1) / kChunk, per = (chunks + n_seg - 1) / n_seg;
   const int seg_len = (int)(per * kChunk);
   n_seg = (chunks + per - 1) / per;
