@@ -1,5 +1,5 @@
 // One-token latent attention on tensor cores (bf16): the heads of a sequence share its cached latents, so a block takes
-// 16 heads of one sequence and streams the latents once.
+// 16 or 32 heads of one sequence and streams the latents once.
 //   head_product_kernel   q~ = W_uk[head]^T q  before, and  W_uv[head] o~  after: one small product per head
 //   latent_stream_kernel  scores q~ . c, online softmax and the weighted latent sum o~ over a range of the window
 //   latent_merge_kernel   merges the ranges of one (sequence, head), adds the sink's term, normalises
@@ -21,8 +21,8 @@ template <bool K_MAJOR, int MB>
 __global__ void __launch_bounds__(128)
 head_product_kernel(const __nv_bfloat16* __restrict__ a, int64_t lda, int64_t a_head, const __nv_bfloat16* __restrict__ w, int64_t w_head, int64_t ldw,
                     __nv_bfloat16* __restrict__ out, int64_t ld_out, int64_t out_head, int B, int N, int K) {
-  constexpr int ROWS = 16 * MB, NT = MB == 1 ? 2 : 8;
-  __shared__ __align__(128) uint8_t tiles[2][(ROWS + 64) * 128];
+  constexpr int ROWS = 16 * MB, NT = MB == 1 ? 2 : 8, STAGES = MB == 1 ? 4 : 3;
+  __shared__ __align__(128) uint8_t tiles[STAGES][(ROWS + 64) * 128];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g8 = lane >> 2, t4 = lane & 3;
   const int n0 = blockIdx.x * 64, h = blockIdx.y, b0 = blockIdx.z * ROWS;
   const int row_w = MB == 1 ? 0 : warp * 16, col_w = MB == 1 ? warp * 16 : 0;
@@ -45,17 +45,17 @@ head_product_kernel(const __nv_bfloat16* __restrict__ a, int64_t lda, int64_t a_
   float acc[NT][4];
 #pragma unroll
   for (int i = 0; i < NT; ++i) acc[i][0] = acc[i][1] = acc[i][2] = acc[i][3] = 0.f;
-  load(0, 0);
+#pragma unroll
+  for (int i = 0; i < STAGES - 1; ++i) {
+    if (i * 64 < K) load(i * 64, i);
+    else cp_async_commit();  // (one group per step, so that the wait below can count them)
+  }
   int stage = 0;
-  for (int k0 = 0; k0 < K; k0 += 64, stage ^= 1) {
-    __syncthreads();
-    if (k0 + 64 < K) {
-      load(k0 + 64, stage ^ 1);
-      cp_async_wait<1>();
-    } else {
-      cp_async_wait<0>();
-    }
-    __syncthreads();
+  for (int k0 = 0; k0 < K; k0 += 64) {
+    cp_async_wait<STAGES - 2>();
+    __syncthreads();  // this step's tiles are in place, and the stage filled next is no longer read
+    if (k0 + (STAGES - 1) * 64 < K) load(k0 + (STAGES - 1) * 64, stage == 0 ? STAGES - 1 : stage - 1);
+    else cp_async_commit();
     const uint32_t sa = (uint32_t)__cvta_generic_to_shared(tiles[stage]), sw = sa + ROWS * 128;
 #pragma unroll
     for (int ks = 0; ks < 4; ++ks) {
@@ -71,6 +71,7 @@ head_product_kernel(const __nv_bfloat16* __restrict__ a, int64_t lda, int64_t a_
         mma_bf16(acc[2 * np + 1], af, wf[2], wf[3]);
       }
     }
+    if (++stage == STAGES) stage = 0;
   }
 #pragma unroll
   for (int nt = 0; nt < NT; ++nt)
@@ -84,160 +85,200 @@ head_product_kernel(const __nv_bfloat16* __restrict__ a, int64_t lda, int64_t a_
 }
 
 // ------------------------------------------------------------------ streaming the latents
-constexpr int kHeads = 16, kKeys = 32, kStreamThreads = 128, kStreamCtasPerSm = 2;
-static_assert(kKeys == 8 * kStreamThreads / 32, "a warp scores eight keys of a tile");
+constexpr int kKeys = 32, kStreamThreads = 256, kStreamCtasPerSm = 2;
+static_assert(2 * kKeys == 8 * kStreamThreads / 32, "a warp scores eight keys of a tile over half of the latent");
 
-template <int RP>  // latent size, padded to 128, 256 or 512
+template <int RP, int HT>  // latent size, padded to 128, 256 or 512; 16-head tiles per block
 struct StreamSmem {
+  static constexpr int HEADS = 16 * HT;
   static constexpr int ROW = RP * 2;
   static constexpr int C_BYTES = kKeys * ROW;
-  static constexpr int Q_BYTES = kHeads * ROW;
-  static constexpr int P_BYTES = kHeads * 128;  // one bf16 part of the weights; rows of 128 bytes, kKeys * 2 of them used
-  static constexpr int BYTES = 2 * C_BYTES + Q_BYTES + 2 * P_BYTES;
+  static constexpr int Q_BYTES = HEADS * ROW;
+  static constexpr int P_BYTES = HEADS * 128;  // one bf16 part of the weights; rows of 128 bytes, kKeys * 2 of them used
+  static constexpr int S_BYTES = 2 * HEADS * kKeys * 4;  // scores, one partial sum per half of the latent
+  static constexpr int BYTES = 2 * C_BYTES + Q_BYTES + 2 * P_BYTES + S_BYTES;
 };
 
-// blockIdx.x = sequence, y = group of 16 heads, z = range of the window.  Partial results per (sequence, head, range):
+// Per tile of 32 latents: scores (a warp takes 8 keys and half of the latent), softmax (a warp takes whole heads, one key
+// per lane), weighted sum (a warp takes an eighth of the latent), with a barrier in front of each.
+// blockIdx.x = sequence, y = group of 16 * HT heads, z = range of the window.  Partial results per (sequence, head, range):
 // part_ml = (maximum in log2 units, denominator), part_o = unnormalised sum of latents.
-template <int RP>
+// Shared-memory addresses: a row's 16-byte pieces are permuted inside groups of eight by the row's low three bits, so a
+// lane's address of piece 2 i + b is one of four precomputed offsets (i mod 4) plus 128 bytes for every further four.
+template <int RP, int HT>
 __global__ void __launch_bounds__(kStreamThreads, kStreamCtasPerSm)
 latent_stream_kernel(const __nv_bfloat16* __restrict__ qt, const __nv_bfloat16* __restrict__ cache, float* __restrict__ part_o, float2* __restrict__ part_ml,
                      int heads, int R, int64_t ring, int64_t window, float scale_log2e, const int* __restrict__ pos_dev) {
-  using M = StreamSmem<RP>;
-  constexpr int WARPS = kStreamThreads / 32;
+  using M = StreamSmem<RP, HT>;
+  constexpr int WARPS = kStreamThreads / 32, HEADS = M::HEADS;
   constexpr int ROW = M::ROW, NT = RP / 8 / WARPS;  // 8-column output tiles per warp
+  constexpr int PIECES = RP / 8, ROWS_PER_PASS = kStreamThreads / PIECES, PASSES = kKeys / ROWS_PER_PASS;
+  static_assert(kStreamThreads % PIECES == 0 && kKeys % ROWS_PER_PASS == 0, "a thread keeps its column of pieces");
   extern __shared__ __align__(128) uint8_t smem[];
-  __shared__ float s_max[WARPS][kHeads], s_sum[WARPS][kHeads];
+  __shared__ float s_mult[HEADS];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g8 = lane >> 2, t4 = lane & 3;
   const int64_t b = blockIdx.x;
-  const int h0 = blockIdx.y * kHeads, split = blockIdx.z, n_split = gridDim.z;
+  const int h0 = blockIdx.y * HEADS, split = blockIdx.z, n_split = gridDim.z;
   const uint32_t base = (uint32_t)__cvta_generic_to_shared(smem);
   const uint32_t sq = base + 2 * M::C_BYTES, p_hi = sq + M::Q_BYTES, p_lo = p_hi + M::P_BYTES;
+  float* s_part = reinterpret_cast<float*>(smem + 2 * M::C_BYTES + M::Q_BYTES + 2 * M::P_BYTES);  // [2][HEADS][kKeys]
   const int64_t pos = pos_dev[0], first = pos + 1 > window ? pos + 1 - window : 0;
   const int n_keys = pos < 0 ? 0 : (int)(pos - first + 1);
   const int tiles = (n_keys + kKeys - 1) / kKeys, per = (tiles + n_split - 1) / n_split;
   const int tile0 = split * per, tile1 = min(tiles, tile0 + per);
 
   // (lands together with the first tile of latents)
-  for (int i = threadIdx.x; i < kHeads * (RP / 8); i += kStreamThreads) {
-    const int r = i / (RP / 8), c = i % (RP / 8);
+  for (int i = threadIdx.x; i < HEADS * PIECES; i += kStreamThreads) {
+    const int r = i / PIECES, c = i % PIECES;
     const bool ok = h0 + r < heads && c * 8 < R;
     cp_async16(sq + swz<ROW>(r, c), ok ? qt + (b * heads + h0 + r) * R + c * 8 : qt, ok);
   }
   const __nv_bfloat16* cb = cache + b * ring * R;
-  const int64_t slot0 = first % ring;
+  const int slot0 = (int)(first % ring), n_ring = (int)ring;
+  // this thread's 16-byte pieces of a tile: always column ld_c, rows ld_r, ld_r + ROWS_PER_PASS, ...
+  const int ld_c = threadIdx.x % PIECES, ld_r = threadIdx.x / PIECES;
+  const bool col_ok = ld_c * 8 < R;
+  const __nv_bfloat16* ld_src = cb + ld_c * 8;
   auto load = [&](int tile, int stage) {
     const uint32_t dst = base + stage * M::C_BYTES;
-    for (int i = threadIdx.x; i < kKeys * (RP / 8); i += kStreamThreads) {
-      const int r = i / (RP / 8), c = i % (RP / 8);
-      const int key = tile * kKeys + r;
-      const bool ok = key < n_keys && c * 8 < R;
-      int64_t slot = slot0 + key;  // (key < window <= ring: one wrap at most)
-      if (slot >= ring) slot -= ring;
-      cp_async16(dst + swz<ROW>(r, c), ok ? cb + slot * R + c * 8 : cb, ok);
+    const int key0 = tile * kKeys + ld_r;
+#pragma unroll
+    for (int i = 0; i < PASSES; ++i) {
+      const int key = key0 + i * ROWS_PER_PASS;
+      int slot = slot0 + key;  // (key < window <= ring: one wrap at most)
+      if (slot >= n_ring) slot -= n_ring;
+      const bool ok = key < n_keys && col_ok;
+      cp_async16(dst + swz<ROW>(ld_r + i * ROWS_PER_PASS, ld_c), ok ? ld_src + (int64_t)slot * R : cb, ok);
     }
     cp_async_commit();
   };
-
-  float o[NT][4];
+  const int key_group = warp & 3, k_half = warp >> 2;  // (half of a row is RP bytes, a whole number of groups of eight pieces)
+  uint32_t off_q[4], off_c[4], off_v[4];               // lane addresses of piece 2 i + b, i mod 4
 #pragma unroll
-  for (int i = 0; i < NT; ++i) o[i][0] = o[i][1] = o[i][2] = o[i][3] = 0.f;
-  float m_run[2] = {-INFINITY, -INFINITY}, l_run[2] = {0.f, 0.f};  // heads g8 and g8 + 8
+  for (int i = 0; i < 4; ++i) {
+    off_q[i] = sq + swz<ROW>(lane & 15, i * 2 + (lane >> 4)) + k_half * RP;
+    off_c[i] = swz<ROW>(key_group * 8 + (lane & 7), i * 2 + ((lane >> 3) & 1)) + k_half * RP;
+    off_v[i] = swz<ROW>((lane & 7) + ((lane >> 3) & 1) * 8, (warp * NT + i * 2 + (lane >> 4)) & 7) + (uint32_t)((warp * NT / 8) * 128);
+  }
+  constexpr int V_WRAP = NT >= 8 ? 4 : NT / 2;  // pairs of output tiles before a warp's pieces enter the next group of eight
+
+  float o[HT][NT][4];
+#pragma unroll
+  for (int ht = 0; ht < HT; ++ht)
+#pragma unroll
+    for (int i = 0; i < NT; ++i) o[ht][i][0] = o[ht][i][1] = o[ht][i][2] = o[ht][i][3] = 0.f;
+  constexpr int HPW = HEADS / WARPS;  // heads whose softmax this warp keeps
+  float m_run[HPW], l_run[HPW];
+#pragma unroll
+  for (int i = 0; i < HPW; ++i) m_run[i] = -INFINITY, l_run[i] = 0.f;
   if (tile0 < tile1) load(tile0, 0);
   int stage = 0;
   for (int tile = tile0; tile < tile1; ++tile, stage ^= 1) {
-    __syncthreads();  // the other stage and the weights of the tile before are no longer read
-    if (tile + 1 < tile1) {
-      load(tile + 1, stage ^ 1);
-      cp_async_wait<1>();
-    } else {
-      cp_async_wait<0>();
-    }
-    __syncthreads();
+    cp_async_wait<0>();
+    __syncthreads();  // the tile has landed; the other stage and the weights of the tile before are no longer read
+    if (tile + 1 < tile1) load(tile + 1, stage ^ 1);
     const uint32_t sc = base + stage * M::C_BYTES;
-    // scores of 16 heads x this warp's 8 keys
-    float s[4] = {0.f, 0.f, 0.f, 0.f}, s1[4] = {0.f, 0.f, 0.f, 0.f};
-#pragma unroll 8
-    for (int ks = 0; ks < RP / 16; ++ks) {
-      uint32_t qf[4], cf[2];
-      ldsm4(qf, sq + swz<ROW>(lane & 15, ks * 2 + (lane >> 4)));
-      ldsm2(cf, sc + swz<ROW>(warp * 8 + (lane & 7), ks * 2 + ((lane >> 3) & 1)));
-      mma_bf16(ks & 1 ? s1 : s, qf, cf[0], cf[1]);
-    }
+    {
+      float s[HT][4], s1[HT][4];
 #pragma unroll
-    for (int i = 0; i < 4; ++i) s[i] += s1[i];
-    const int key = tile * kKeys + warp * 8 + t4 * 2;
-    float bm[2];
+      for (int ht = 0; ht < HT; ++ht)
 #pragma unroll
-    for (int r = 0; r < 2; ++r) {
-      s[2 * r] = key < n_keys ? s[2 * r] * scale_log2e : -INFINITY;
-      s[2 * r + 1] = key + 1 < n_keys ? s[2 * r + 1] * scale_log2e : -INFINITY;
-      bm[r] = fmaxf(s[2 * r], s[2 * r + 1]);
-      bm[r] = fmaxf(bm[r], __shfl_xor_sync(0xffffffffu, bm[r], 1));
-      bm[r] = fmaxf(bm[r], __shfl_xor_sync(0xffffffffu, bm[r], 2));
-      if (t4 == 0) s_max[warp][g8 + r * 8] = bm[r];
-    }
-    __syncthreads();
-    float mult[2];
+        for (int i = 0; i < 4; ++i) s[ht][i] = s1[ht][i] = 0.f;
 #pragma unroll
-    for (int r = 0; r < 2; ++r) {
-      float m_new = m_run[r];
+      for (int ks = 0; ks < RP / 32; ++ks) {
+        uint32_t cf[2];
+        ldsm2(cf, sc + off_c[ks & 3] + (ks >> 2) * 128);
 #pragma unroll
-      for (int w2 = 0; w2 < WARPS; ++w2) m_new = fmaxf(m_new, s_max[w2][g8 + r * 8]);  // finite: a tile has at least one key
-      mult[r] = exp2f(m_run[r] - m_new);
-      m_run[r] = m_new;
-      const float p0 = exp2f(s[2 * r] - m_new), p1 = exp2f(s[2 * r + 1] - m_new);
-      uint32_t hi, lo;
-      split_pair(p0, p1, hi, lo);
-      const uint32_t at = swz<128>(g8 + r * 8, warp) + t4 * 4;
-      asm volatile("st.shared.b32 [%0], %1;" ::"r"(p_hi + at), "r"(hi) : "memory");
-      asm volatile("st.shared.b32 [%0], %1;" ::"r"(p_lo + at), "r"(lo) : "memory");
-      float ps = p0 + p1;
-      ps += __shfl_xor_sync(0xffffffffu, ps, 1);
-      ps += __shfl_xor_sync(0xffffffffu, ps, 2);
-      if (t4 == 0) s_sum[warp][g8 + r * 8] = ps;
+        for (int ht = 0; ht < HT; ++ht) {
+          uint32_t qf[4];
+          ldsm4(qf, off_q[ks & 3] + (ks >> 2) * 128 + ht * 16 * ROW);
+          mma_bf16(ks & 1 ? s1[ht] : s[ht], qf, cf[0], cf[1]);
+        }
+      }
+#pragma unroll
+      for (int ht = 0; ht < HT; ++ht)
+#pragma unroll
+        for (int r = 0; r < 2; ++r)
+          *reinterpret_cast<float2*>(s_part + (k_half * HEADS + ht * 16 + g8 + r * 8) * kKeys + key_group * 8 + t4 * 2) =
+              make_float2(s[ht][2 * r] + s1[ht][2 * r], s[ht][2 * r + 1] + s1[ht][2 * r + 1]);
     }
     __syncthreads();
+    const bool key_ok = tile * kKeys + lane < n_keys;
 #pragma unroll
-    for (int r = 0; r < 2; ++r) {
-      float ps = 0.f;
+    for (int i = 0; i < HPW; ++i) {
+      const int row = warp * HPW + i;
+      const float v = key_ok ? (s_part[row * kKeys + lane] + s_part[(HEADS + row) * kKeys + lane]) * scale_log2e : -INFINITY;
+      float m_new = v;
 #pragma unroll
-      for (int w2 = 0; w2 < WARPS; ++w2) ps += s_sum[w2][g8 + r * 8];
-      l_run[r] = l_run[r] * mult[r] + ps;
+      for (int off = 16; off > 0; off >>= 1) m_new = fmaxf(m_new, __shfl_xor_sync(0xffffffffu, m_new, off));
+      m_new = fmaxf(m_run[i], m_new);  // finite: a tile has at least one key
+      const float mult = exp2f(m_run[i] - m_new), p = exp2f(v - m_new);
+      m_run[i] = m_new;
+      l_run[i] = l_run[i] * mult + warp_sum(p);
+      const __nv_bfloat16 hi = __float2bfloat16_rn(p), lo = __float2bfloat16_rn(p - __bfloat162float(hi));
+      const uint32_t at = swz<128>(row, lane >> 3) + (lane & 7) * 2;
+      asm volatile("st.shared.b16 [%0], %1;" ::"r"(p_hi + at), "h"(*reinterpret_cast<const uint16_t*>(&hi)) : "memory");
+      asm volatile("st.shared.b16 [%0], %1;" ::"r"(p_lo + at), "h"(*reinterpret_cast<const uint16_t*>(&lo)) : "memory");
+      if (lane == 0) s_mult[row] = mult;
     }
+    __syncthreads();
+    float mult[HT][2];
+    bool moved = false;
 #pragma unroll
-    for (int i = 0; i < NT; ++i) o[i][0] *= mult[0], o[i][1] *= mult[0], o[i][2] *= mult[1], o[i][3] *= mult[1];
+    for (int ht = 0; ht < HT; ++ht)
+#pragma unroll
+      for (int r = 0; r < 2; ++r) mult[ht][r] = s_mult[ht * 16 + g8 + r * 8], moved |= mult[ht][r] != 1.0f;
+    if (__any_sync(0xffffffffu, moved)) {
+#pragma unroll
+      for (int ht = 0; ht < HT; ++ht)
+#pragma unroll
+        for (int i = 0; i < NT; ++i)
+          o[ht][i][0] *= mult[ht][0], o[ht][i][1] *= mult[ht][0], o[ht][i][2] *= mult[ht][1], o[ht][i][3] *= mult[ht][1];
+    }
     // o~ += P c for this warp's RP / WARPS columns
 #pragma unroll
     for (int kk = 0; kk < kKeys / 16; ++kk) {
-      uint32_t ph[4], pl[4];
-      const uint32_t at = swz<128>(lane & 15, kk * 2 + (lane >> 4));
-      ldsm4(ph, p_hi + at);
-      ldsm4(pl, p_lo + at);
+      uint32_t ph[HT][4], pl[HT][4];
+#pragma unroll
+      for (int ht = 0; ht < HT; ++ht) {
+        const uint32_t at = swz<128>(ht * 16 + (lane & 15), kk * 2 + (lane >> 4));
+        ldsm4(ph[ht], p_hi + at);
+        ldsm4(pl[ht], p_lo + at);
+      }
 #pragma unroll
       for (int np = 0; np < NT / 2; ++np) {
         uint32_t cf[4];
-        ldsm4_trans(cf, sc + swz<ROW>(kk * 16 + (lane & 7) + ((lane >> 3) & 1) * 8, warp * NT + np * 2 + (lane >> 4)));
-        mma_bf16(o[2 * np], ph, cf[0], cf[1]);
-        mma_bf16(o[2 * np + 1], ph, cf[2], cf[3]);
-        mma_bf16(o[2 * np], pl, cf[0], cf[1]);
-        mma_bf16(o[2 * np + 1], pl, cf[2], cf[3]);
+        ldsm4_trans(cf, sc + off_v[np % V_WRAP] + (np / V_WRAP) * 128 + kk * 16 * ROW);
+#pragma unroll
+        for (int ht = 0; ht < HT; ++ht) {
+          mma_bf16(o[ht][2 * np], ph[ht], cf[0], cf[1]);
+          mma_bf16(o[ht][2 * np + 1], ph[ht], cf[2], cf[3]);
+          mma_bf16(o[ht][2 * np], pl[ht], cf[0], cf[1]);
+          mma_bf16(o[ht][2 * np + 1], pl[ht], cf[2], cf[3]);
+        }
       }
     }
   }
   cp_async_commit();
   cp_async_wait<0>();  // (a block without tiles still has its queries in flight)
 #pragma unroll
-  for (int r = 0; r < 2; ++r) {
-    const int h = h0 + g8 + r * 8;
-    if (h >= heads) continue;
-    const int64_t item = (b * heads + h) * n_split + split;
-    if (warp == 0 && t4 == 0) part_ml[item] = make_float2(m_run[r], l_run[r]);
-#pragma unroll
-    for (int i = 0; i < NT; ++i) {
-      const int c = (warp * NT + i) * 8 + t4 * 2;
-      if (c < R) *reinterpret_cast<float2*>(part_o + item * R + c) = make_float2(o[i][2 * r], o[i][2 * r + 1]);
-    }
+  for (int i = 0; i < HPW; ++i) {
+    const int h = h0 + warp * HPW + i;
+    if (lane == 0 && h < heads) part_ml[(b * heads + h) * n_split + split] = make_float2(m_run[i], l_run[i]);
   }
+#pragma unroll
+  for (int ht = 0; ht < HT; ++ht)
+#pragma unroll
+    for (int r = 0; r < 2; ++r) {
+      const int h = h0 + ht * 16 + g8 + r * 8;
+      if (h >= heads) continue;
+      const int64_t item = (b * heads + h) * n_split + split;
+#pragma unroll
+      for (int i = 0; i < NT; ++i) {
+        const int c = (warp * NT + i) * 8 + t4 * 2;
+        if (c < R) *reinterpret_cast<float2*>(part_o + item * R + c) = make_float2(o[ht][i][2 * r], o[ht][i][2 * r + 1]);
+      }
+    }
 }
 
 // One block per (sequence, head).
@@ -289,7 +330,7 @@ struct Plan {
 };
 Plan make_plan(int64_t B, int64_t heads, int64_t R, int64_t window) {
   Plan p;
-  const int64_t groups = B * ((heads + kHeads - 1) / kHeads), tiles = (window + kKeys - 1) / kKeys;
+  const int64_t per_block = heads > 16 ? 32 : 16, groups = B * ((heads + per_block - 1) / per_block), tiles = (window + kKeys - 1) / kKeys;
   // ranges per sequence: the fewest rounds of blocks, counted in tiles (a block's start-up and its share of the merge are
   // worth about three)
   const int64_t slots = (int64_t)sm_count() * kStreamCtasPerSm;
@@ -307,29 +348,36 @@ Plan make_plan(int64_t B, int64_t heads, int64_t R, int64_t window) {
   return p;
 }
 
-template <int RP>
+template <int RP, int HT>
 int launch_stream(const __nv_bfloat16* qt, const void* cache, float* po, float2* ml, int64_t B, int64_t heads, int64_t R, int64_t ring, int64_t window,
                   float scale, int n_split, const int* pos_dev, cudaStream_t stream) {
-  constexpr int smem = StreamSmem<RP>::BYTES;
+  constexpr int smem = StreamSmem<RP, HT>::BYTES;
   static std::atomic<bool> attr_set[kMaxDevices];
   const int slot = device_slot();
   if (slot < 0) return B200_ERR_CUDA;
   if (!attr_set[slot].load(std::memory_order_acquire)) {
-    if (cudaFuncSetAttribute(latent_stream_kernel<RP>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return B200_ERR_CUDA;
+    if (cudaFuncSetAttribute(latent_stream_kernel<RP, HT>, cudaFuncAttributeMaxDynamicSharedMemorySize, smem) != cudaSuccess) return B200_ERR_CUDA;
     attr_set[slot].store(true, std::memory_order_release);
   }
-  latent_stream_kernel<RP><<<dim3((unsigned)B, (unsigned)((heads + kHeads - 1) / kHeads), (unsigned)n_split), kStreamThreads, smem, stream>>>(
+  latent_stream_kernel<RP, HT><<<dim3((unsigned)B, (unsigned)((heads + 16 * HT - 1) / (16 * HT)), (unsigned)n_split), kStreamThreads, smem, stream>>>(
       qt, static_cast<const __nv_bfloat16*>(cache), po, ml, (int)heads, (int)R, ring, window, scale * 1.4426950408889634f, pos_dev);
   note_launches(1);
   return status_from_cuda(cudaGetLastError());
+}
+
+template <int RP>
+int launch_stream_heads(const __nv_bfloat16* qt, const void* cache, float* po, float2* ml, int64_t B, int64_t heads, int64_t R, int64_t ring,
+                        int64_t window, float scale, int n_split, const int* pos_dev, cudaStream_t stream) {
+  return heads > 16 ? launch_stream<RP, 2>(qt, cache, po, ml, B, heads, R, ring, window, scale, n_split, pos_dev, stream)
+                    : launch_stream<RP, 1>(qt, cache, po, ml, B, heads, R, ring, window, scale, n_split, pos_dev, stream);
 }
 
 template <bool K_MAJOR>
 void head_product(const __nv_bfloat16* a, int64_t lda, int64_t a_head, const __nv_bfloat16* w, int64_t w_head, int64_t ldw, __nv_bfloat16* out, int64_t ld_out,
                   int64_t out_head, int64_t B, int64_t heads, int64_t N, int64_t K, cudaStream_t stream) {
   const unsigned nb = (unsigned)((N + 63) / 64);
-  if (B <= 16)
-    head_product_kernel<K_MAJOR, 1><<<dim3(nb, (unsigned)heads, 1), 128, 0, stream>>>(a, lda, a_head, w, w_head, ldw, out, ld_out, out_head, (int)B, (int)N, (int)K);
+  if (B <= 128)
+    head_product_kernel<K_MAJOR, 1><<<dim3(nb, (unsigned)heads, (unsigned)((B + 15) / 16)), 128, 0, stream>>>(a, lda, a_head, w, w_head, ldw, out, ld_out, out_head, (int)B, (int)N, (int)K);
   else
     head_product_kernel<K_MAJOR, 4><<<dim3(nb, (unsigned)heads, (unsigned)((B + 63) / 64)), 128, 0, stream>>>(a, lda, a_head, w, w_head, ldw, out, ld_out,
                                                                                                                     out_head, (int)B, (int)N, (int)K);
@@ -348,7 +396,7 @@ int launch_latent_decode_mma(const void* q, int64_t ld_q, const void* w_uk, cons
                              int64_t heads, int64_t dim, int64_t vdim, int64_t R, int64_t ring, int64_t window, float scale, const float* sink,
                              const int* pos_dev, void* workspace, cudaStream_t stream) {
   if (R > 512 || R % 8 || dim % 8 || vdim % 8 || ld_q % 8 || ld_out % 2 || (reinterpret_cast<uintptr_t>(out) & 3) || !aligned16_all(q, w_uk, w_uv, cache)) return B200_ERR_UNSUPPORTED;
-  if (B > 65535 || heads > 65535 || window > (1 << 30)) return B200_ERR_UNSUPPORTED;
+  if (B > 65535 || heads > 65535 || ring > (1 << 30)) return B200_ERR_UNSUPPORTED;
   const Plan p = make_plan(B, heads, R, window);
   uint8_t* ws = static_cast<uint8_t*>(workspace);
   __nv_bfloat16* qt = reinterpret_cast<__nv_bfloat16*>(ws);
@@ -356,9 +404,9 @@ int launch_latent_decode_mma(const void* q, int64_t ld_q, const void* w_uk, cons
   float2* ml = reinterpret_cast<float2*>(ws + p.off_ml);
   __nv_bfloat16* ot = reinterpret_cast<__nv_bfloat16*>(ws + p.off_ot);
   head_product<false>((const __nv_bfloat16*)q, ld_q, dim, (const __nv_bfloat16*)w_uk, dim * R, R, qt, heads * R, R, B, heads, R, dim, stream);
-  int st = R <= 128   ? launch_stream<128>(qt, cache, po, ml, B, heads, R, ring, window, scale, p.n_split, pos_dev, stream)
-           : R <= 256 ? launch_stream<256>(qt, cache, po, ml, B, heads, R, ring, window, scale, p.n_split, pos_dev, stream)
-                      : launch_stream<512>(qt, cache, po, ml, B, heads, R, ring, window, scale, p.n_split, pos_dev, stream);
+  int st = R <= 128   ? launch_stream_heads<128>(qt, cache, po, ml, B, heads, R, ring, window, scale, p.n_split, pos_dev, stream)
+           : R <= 256 ? launch_stream_heads<256>(qt, cache, po, ml, B, heads, R, ring, window, scale, p.n_split, pos_dev, stream)
+                      : launch_stream_heads<512>(qt, cache, po, ml, B, heads, R, ring, window, scale, p.n_split, pos_dev, stream);
   if (st != B200_OK) return st;
   latent_merge_kernel<<<(unsigned)(B * heads), 128, 0, stream>>>(po, ml, ot, (int)heads, (int)R, p.n_split, sink);
   note_launches(1);
