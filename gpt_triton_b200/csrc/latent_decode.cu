@@ -85,28 +85,32 @@ head_product_kernel(const __nv_bfloat16* __restrict__ a, int64_t lda, int64_t a_
 }
 
 // ------------------------------------------------------------------ streaming the latents
-constexpr int kKeys = 32, kStreamThreads = 256, kStreamCtasPerSm = 2;
-static_assert(2 * kKeys == 8 * kStreamThreads / 32, "a warp scores eight keys of a tile over half of the latent");
+constexpr int kKeys = 32, kStreamThreads = 256;
+constexpr int kPartRow = kKeys + 8;  // floats per row of partial scores (the padding spreads eight rows over the banks)
 
 template <int RP, int HT>  // latent size, padded to 128, 256 or 512; 16-head tiles per block
 struct StreamSmem {
   static constexpr int HEADS = 16 * HT;
   static constexpr int ROW = RP * 2;
   static constexpr int C_BYTES = kKeys * ROW;
-  static constexpr int Q_BYTES = HEADS * ROW;
   static constexpr int P_BYTES = HEADS * 128;  // one bf16 part of the weights; rows of 128 bytes, kKeys * 2 of them used
-  static constexpr int S_BYTES = 2 * HEADS * kKeys * 4;  // scores, one partial sum per half of the latent
-  static constexpr int BYTES = 2 * C_BYTES + Q_BYTES + 2 * P_BYTES + S_BYTES;
+  static constexpr int S_BYTES = kStreamThreads / 32 * HEADS * kPartRow * 4;  // scores, one partial sum per eighth of the latent
+  static constexpr int CTAS_PER_SM = HT == 1 ? 2 : 1;  // (the output of 32 heads takes too many registers for two)
+  static constexpr int FIT = (220 * 1024 / CTAS_PER_SM - 2 * P_BYTES - S_BYTES) / C_BYTES;
+  static constexpr int STAGES = FIT < 8 ? FIT : 8;  // tiles in the ring
+  static constexpr int BYTES = STAGES * C_BYTES + 2 * P_BYTES + S_BYTES;
+  static_assert(STAGES >= 2, "shared memory budget");
 };
 
-// Per tile of 32 latents: scores (a warp takes 8 keys and half of the latent), softmax (a warp takes whole heads, one key
-// per lane), weighted sum (a warp takes an eighth of the latent), with a barrier in front of each.
+// Per tile of 32 latents: partial scores (a warp takes all keys over an eighth of the latent; its part of q~ stays in
+// registers), softmax (a warp takes whole heads, one key per lane), weighted sum (a warp takes an eighth of the latent),
+// with a barrier in front of each.
 // blockIdx.x = sequence, y = group of 16 * HT heads, z = range of the window.  Partial results per (sequence, head, range):
 // part_ml = (maximum in log2 units, denominator), part_o = unnormalised sum of latents.
-// Shared-memory addresses: a row's 16-byte pieces are permuted inside groups of eight by the row's low three bits, so a
+// Shared-memory addresses of the weighted sum: a row's 16-byte pieces are permuted inside groups of eight by the row's low three bits, so a
 // lane's address of piece 2 i + b is one of four precomputed offsets (i mod 4) plus 128 bytes for every further four.
 template <int RP, int HT>
-__global__ void __launch_bounds__(kStreamThreads, kStreamCtasPerSm)
+__global__ void __launch_bounds__(kStreamThreads, StreamSmem<RP, HT>::CTAS_PER_SM)
 latent_stream_kernel(const __nv_bfloat16* __restrict__ qt, const __nv_bfloat16* __restrict__ cache, float* __restrict__ part_o, float2* __restrict__ part_ml,
                      int heads, int R, int64_t ring, int64_t window, float scale_log2e, const int* __restrict__ pos_dev) {
   using M = StreamSmem<RP, HT>;
@@ -120,19 +124,13 @@ latent_stream_kernel(const __nv_bfloat16* __restrict__ qt, const __nv_bfloat16* 
   const int64_t b = blockIdx.x;
   const int h0 = blockIdx.y * HEADS, split = blockIdx.z, n_split = gridDim.z;
   const uint32_t base = (uint32_t)__cvta_generic_to_shared(smem);
-  const uint32_t sq = base + 2 * M::C_BYTES, p_hi = sq + M::Q_BYTES, p_lo = p_hi + M::P_BYTES;
-  float* s_part = reinterpret_cast<float*>(smem + 2 * M::C_BYTES + M::Q_BYTES + 2 * M::P_BYTES);  // [2][HEADS][kKeys]
+  const uint32_t p_hi = base + M::STAGES * M::C_BYTES, p_lo = p_hi + M::P_BYTES;
+  float* s_part = reinterpret_cast<float*>(smem + M::STAGES * M::C_BYTES + 2 * M::P_BYTES);  // [WARPS][HEADS][kPartRow]
   const int64_t pos = pos_dev[0], first = pos + 1 > window ? pos + 1 - window : 0;
   const int n_keys = pos < 0 ? 0 : (int)(pos - first + 1);
   const int tiles = (n_keys + kKeys - 1) / kKeys, per = (tiles + n_split - 1) / n_split;
   const int tile0 = split * per, tile1 = min(tiles, tile0 + per);
 
-  // (lands together with the first tile of latents)
-  for (int i = threadIdx.x; i < HEADS * PIECES; i += kStreamThreads) {
-    const int r = i / PIECES, c = i % PIECES;
-    const bool ok = h0 + r < heads && c * 8 < R;
-    cp_async16(sq + swz<ROW>(r, c), ok ? qt + (b * heads + h0 + r) * R + c * 8 : qt, ok);
-  }
   const __nv_bfloat16* cb = cache + b * ring * R;
   const int slot0 = (int)(first % ring), n_ring = (int)ring;
   // this thread's 16-byte pieces of a tile: always column ld_c, rows ld_r, ld_r + ROWS_PER_PASS, ...
@@ -152,14 +150,24 @@ latent_stream_kernel(const __nv_bfloat16* __restrict__ qt, const __nv_bfloat16* 
     }
     cp_async_commit();
   };
-  const int key_group = warp & 3, k_half = warp >> 2;  // (half of a row is RP bytes, a whole number of groups of eight pieces)
-  uint32_t off_q[4], off_c[4], off_v[4];               // lane addresses of piece 2 i + b, i mod 4
+  // this warp's eighth of the queries as A fragments (rows g8, g8 + 8; columns t4 * 2 + {0, 1} and + 8 of each 16)
+  constexpr int KS = RP / 8 / WARPS / 2;  // 16-wide k-steps per warp
+  uint32_t qf[HT][KS][4];
 #pragma unroll
-  for (int i = 0; i < 4; ++i) {
-    off_q[i] = sq + swz<ROW>(lane & 15, i * 2 + (lane >> 4)) + k_half * RP;
-    off_c[i] = swz<ROW>(key_group * 8 + (lane & 7), i * 2 + ((lane >> 3) & 1)) + k_half * RP;
+  for (int ht = 0; ht < HT; ++ht)
+#pragma unroll
+    for (int ks = 0; ks < KS; ++ks)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) {
+        const int h = h0 + ht * 16 + g8 + (e & 1) * 8, c = (warp * KS + ks) * 16 + t4 * 2 + (e >> 1) * 8;
+        qf[ht][ks][e] = h < heads && c < R ? *reinterpret_cast<const uint32_t*>(qt + (b * heads + h) * R + c) : 0u;
+      }
+  uint32_t off_c[KS], off_v[4];  // lane addresses: scores, by k-step; weighted sum, of piece 2 i + b, i mod 4
+#pragma unroll
+  for (int i = 0; i < KS; ++i) off_c[i] = swz<ROW>((lane & 7) + ((lane >> 4) << 3), (warp * KS + i) * 2 + ((lane >> 3) & 1));
+#pragma unroll
+  for (int i = 0; i < 4; ++i)
     off_v[i] = swz<ROW>((lane & 7) + ((lane >> 3) & 1) * 8, (warp * NT + i * 2 + (lane >> 4)) & 7) + (uint32_t)((warp * NT / 8) * 128);
-  }
   constexpr int V_WRAP = NT >= 8 ? 4 : NT / 2;  // pairs of output tiles before a warp's pieces enter the next group of eight
 
   float o[HT][NT][4];
@@ -171,43 +179,54 @@ latent_stream_kernel(const __nv_bfloat16* __restrict__ qt, const __nv_bfloat16* 
   float m_run[HPW], l_run[HPW];
 #pragma unroll
   for (int i = 0; i < HPW; ++i) m_run[i] = -INFINITY, l_run[i] = 0.f;
-  if (tile0 < tile1) load(tile0, 0);
+#pragma unroll
+  for (int i = 0; i < M::STAGES - 1; ++i) {
+    if (tile0 + i < tile1) load(tile0 + i, i);
+    else cp_async_commit();  // (one group per tile, so that the wait below can count them)
+  }
   int stage = 0;
-  for (int tile = tile0; tile < tile1; ++tile, stage ^= 1) {
-    cp_async_wait<0>();
-    __syncthreads();  // the tile has landed; the other stage and the weights of the tile before are no longer read
-    if (tile + 1 < tile1) load(tile + 1, stage ^ 1);
+  for (int tile = tile0; tile < tile1; ++tile, stage = stage + 1 == M::STAGES ? 0 : stage + 1) {
+    cp_async_wait<M::STAGES - 2>();
+    __syncthreads();  // the tile has landed; the stage before it and the weights of the tile before are no longer read
+    if (tile + M::STAGES - 1 < tile1) load(tile + M::STAGES - 1, stage == 0 ? M::STAGES - 1 : stage - 1);
+    else cp_async_commit();
     const uint32_t sc = base + stage * M::C_BYTES;
     {
-      float s[HT][4], s1[HT][4];
+      float s[HT][kKeys / 8][4];
 #pragma unroll
       for (int ht = 0; ht < HT; ++ht)
 #pragma unroll
-        for (int i = 0; i < 4; ++i) s[ht][i] = s1[ht][i] = 0.f;
+        for (int nt = 0; nt < kKeys / 8; ++nt) s[ht][nt][0] = s[ht][nt][1] = s[ht][nt][2] = s[ht][nt][3] = 0.f;
 #pragma unroll
-      for (int ks = 0; ks < RP / 32; ++ks) {
-        uint32_t cf[2];
-        ldsm2(cf, sc + off_c[ks & 3] + (ks >> 2) * 128);
+      for (int ks = 0; ks < KS; ++ks)
 #pragma unroll
-        for (int ht = 0; ht < HT; ++ht) {
-          uint32_t qf[4];
-          ldsm4(qf, off_q[ks & 3] + (ks >> 2) * 128 + ht * 16 * ROW);
-          mma_bf16(ks & 1 ? s1[ht] : s[ht], qf, cf[0], cf[1]);
+        for (int np = 0; np < kKeys / 16; ++np) {
+          uint32_t cf[4];
+          ldsm4(cf, sc + off_c[ks] + np * 16 * ROW);
+#pragma unroll
+          for (int ht = 0; ht < HT; ++ht) {
+            mma_bf16(s[ht][2 * np], qf[ht][ks], cf[0], cf[1]);
+            mma_bf16(s[ht][2 * np + 1], qf[ht][ks], cf[2], cf[3]);
+          }
         }
-      }
 #pragma unroll
       for (int ht = 0; ht < HT; ++ht)
 #pragma unroll
-        for (int r = 0; r < 2; ++r)
-          *reinterpret_cast<float2*>(s_part + (k_half * HEADS + ht * 16 + g8 + r * 8) * kKeys + key_group * 8 + t4 * 2) =
-              make_float2(s[ht][2 * r] + s1[ht][2 * r], s[ht][2 * r + 1] + s1[ht][2 * r + 1]);
+        for (int nt = 0; nt < kKeys / 8; ++nt)
+#pragma unroll
+          for (int r = 0; r < 2; ++r)
+            *reinterpret_cast<float2*>(s_part + (warp * HEADS + ht * 16 + g8 + r * 8) * kPartRow + nt * 8 + t4 * 2) =
+                make_float2(s[ht][nt][2 * r], s[ht][nt][2 * r + 1]);
     }
     __syncthreads();
     const bool key_ok = tile * kKeys + lane < n_keys;
 #pragma unroll
     for (int i = 0; i < HPW; ++i) {
       const int row = warp * HPW + i;
-      const float v = key_ok ? (s_part[row * kKeys + lane] + s_part[(HEADS + row) * kKeys + lane]) * scale_log2e : -INFINITY;
+      float v = 0.f;
+#pragma unroll
+      for (int w2 = 0; w2 < WARPS; ++w2) v += s_part[(w2 * HEADS + row) * kPartRow + lane];
+      v = key_ok ? v * scale_log2e : -INFINITY;
       float m_new = v;
 #pragma unroll
       for (int off = 16; off > 0; off >>= 1) m_new = fmaxf(m_new, __shfl_xor_sync(0xffffffffu, m_new, off));
@@ -259,8 +278,6 @@ latent_stream_kernel(const __nv_bfloat16* __restrict__ qt, const __nv_bfloat16* 
       }
     }
   }
-  cp_async_commit();
-  cp_async_wait<0>();  // (a block without tiles still has its queries in flight)
 #pragma unroll
   for (int i = 0; i < HPW; ++i) {
     const int h = h0 + warp * HPW + i;
@@ -333,7 +350,7 @@ Plan make_plan(int64_t B, int64_t heads, int64_t R, int64_t window) {
   const int64_t per_block = heads > 16 ? 32 : 16, groups = B * ((heads + per_block - 1) / per_block), tiles = (window + kKeys - 1) / kKeys;
   // ranges per sequence: the fewest rounds of blocks, counted in tiles (a block's start-up and its share of the merge are
   // worth about three)
-  const int64_t slots = (int64_t)sm_count() * kStreamCtasPerSm;
+  const int64_t slots = (int64_t)sm_count() * (heads > 16 ? 1 : 2);
   int64_t n = 1, best = -1;
   for (int64_t k = 1; k <= tiles && k <= kMaxSplit; ++k) {
     const int64_t cost = ((groups * k + slots - 1) / slots) * ((tiles + k - 1) / k + 3);
