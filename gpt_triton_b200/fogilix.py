@@ -12,9 +12,9 @@ import torch
 from torch import nn
 
 from . import kernels as K
-from .generation import GeneratesTokens
-from .mixers import DenseFeedForward, LatentAttention, LightningAttention, PromptContext, StepContext, _weight
-from .module_base import _EvalOnly, _OperandCache
+from .decoder import StreamDecoder
+from .mixers import DenseFeedForward, LatentAttention, LightningAttention, _weight
+from .module_base import _OperandCache
 
 
 @dataclass(frozen=True)
@@ -89,8 +89,8 @@ class FogilixLayer(nn.Module):
             self.mlp = DenseFeedForward(w, spec.ff)
 
 
-class Fogilix(GeneratesTokens, _EvalOnly):
-    exact_float32 = True  # float32 models run in true 32-bit
+class Fogilix(StreamDecoder):
+    TENSOR_NAMES = (("final.norm", "final_norm"), ("dkv.norm", "dkv_norm"))
 
     def __init__(self, config):
         super().__init__()
@@ -105,25 +105,10 @@ class Fogilix(GeneratesTokens, _EvalOnly):
         self.head = _weight(config.vocab, config.width)
         self._operand = _OperandCache()
 
-    # ---- weights
-    @staticmethod
-    def _parameter_name(tensor):
-        """Name in the checkpoint -> name of the parameter."""
-        name = tensor.replace("final.norm", "final_norm").replace("dkv.norm", "dkv_norm")
-        return "layers." + name[1:] if name[:1] == "l" and name[1:2].isdigit() else name
-
-    @staticmethod
-    def tensor_name(parameter):
-        """The other way round."""
-        name = parameter.replace("final_norm", "final.norm").replace("dkv_norm", "dkv.norm")
-        return "l" + name.removeprefix("layers.") if name.startswith("layers.") else name
-
     @classmethod
     def from_checkpoint(cls, config, tensors):
         """config: the parsed config.json; tensors: name -> tensor of model.safetensors."""
-        model = cls(FogilixConfig.from_dict(config))
-        model.load_state_dict({cls._parameter_name(k): v for k, v in tensors.items()})
-        return model
+        return cls._load(FogilixConfig.from_dict(config), tensors)
 
     def _gain(self, param):
         """Norm weights are stored around zero."""
@@ -140,7 +125,10 @@ class Fogilix(GeneratesTokens, _EvalOnly):
                 gains.append(layer.norm2)
         return gains[0] if gains else self.final_norm, list(zip(subs, gains[1:] + [self.final_norm]))
 
-    # ---- the step function
+    def new_cache(self, batch, capacity):
+        dev, dtype = self.embed.device, self.embed.dtype
+        return [layer.mix.new_cache(batch, capacity, dev, dtype) for layer in self.layers]
+
     def _run(self, ids, ctx, phase, tap=None):
         """ids (rows,) -> NormedRows behind the final norm.  `tap` (for tests) is called with the stream after every layer."""
         self._check_eval()
@@ -153,54 +141,6 @@ class Fogilix(GeneratesTokens, _EvalOnly):
                 tap(x)
         return rows
 
-    # ---- what GenerationSession drives (generation.py)
-    def vocab_size(self):
-        return self.config.vocab
-
-    def check_capacity(self, capacity):
-        pass  # no position table: any length
-
-    def new_cache(self, batch, capacity):
-        dev, dtype = self.embed.device, self.embed.dtype
-        return [layer.mix.new_cache(batch, capacity, dev, dtype) for layer in self.layers]
-
-    def prompt_pass(self, ids, cache, start, pos=None, want=None, tap=None):
-        B, n = ids.shape
-        rows = self._run(ids.reshape(-1).contiguous(), PromptContext(B, n, start, cache), "prompt", tap)
-        if want is None:
-            want = torch.tensor([n - 1], device=ids.device)
-        index = (torch.arange(B, device=ids.device)[:, None] * n + want[None, :]).reshape(-1)
-        return rows if index.numel() == B * n and n == 1 else rows.select(index)
-
-    def decode_pass(self, ids, cache, pos):
-        return self._run(ids, StepContext(ids.shape[0], pos, cache), "step")
-
     def head_logits(self, rows):
         """Final rows -> float32 logits (rows, vocab)."""
-        w = self._operand.derived(("head",), (self.head,), lambda: K.operand_rows(self.head.data)[0])
-        return K.linear(rows, w, out_scale=self.config.logit_scale, out_dtype=torch.float32)
-
-    def pick(self, rows, temperature, top_k, seed, pos):
-        logits = self.head_logits(rows)
-        if temperature == 0.0:
-            return logits.argmax(dim=-1)
-        return K.sample_logits(logits, temperature=temperature, top_k=top_k, seed=seed, step=pos)
-
-    # ---- whole sequences
-    @torch.no_grad()
-    def logits(self, ids):
-        """ids (batch, n) -> float32 logits (batch, n, vocab)."""
-        B, n = ids.shape
-        rows = self._run(ids.reshape(-1).contiguous(), PromptContext(B, n, 0, None), "prompt")
-        return self.head_logits(rows).view(B, n, -1)
-
-    forward = logits
-
-    @torch.no_grad()
-    def logits_and_next_ids(self, ids):
-        logits = self.logits(ids)
-        return logits, logits.argmax(dim=-1)
-
-    @torch.no_grad()
-    def next_ids(self, ids):
-        return self.logits(ids).argmax(dim=-1)
+        return K.linear(rows, self._head_operand(), out_scale=self.config.logit_scale, out_dtype=torch.float32)

@@ -629,9 +629,15 @@ class NormedRows:
 
     def select(self, index):
         """The rows `index` (int64 tensor) of this matrix."""
-        out = _rows_empty(index.numel(), self.data.shape[1], self.data.dtype, self.data.device)
-        out.copy_(self.data.index_select(0, index))
-        return NormedRows(out, self.sumsq.index_select(1, index), self.norm_cols, self.eps)
+        return NormedRows(select_rows(self.data, index), self.sumsq.index_select(1, index), self.norm_cols, self.eps)
+
+
+def select_rows(rows, index):
+    """The rows `index` (int64 tensor) of a NormedRows or a plain matrix."""
+    if isinstance(rows, NormedRows):
+        return rows.select(index)
+    out = _rows_empty(index.numel(), rows.shape[1], rows.dtype, rows.device)
+    return out.copy_(rows.index_select(0, index))
 
 
 def operand_rows(*weights):
