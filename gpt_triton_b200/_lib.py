@@ -13,6 +13,7 @@ from .build import LIB_PATH
 
 F32, F16, BF16 = 0, 1, 2
 _TORCH_TO_CODE = {torch.float32: F32, torch.float16: F16, torch.bfloat16: BF16}
+CODE_TO_TORCH = {code: dtype for dtype, code in _TORCH_TO_CODE.items()}
 
 c_i64, c_int, c_float, c_void_p, c_size_t = ctypes.c_int64, ctypes.c_int, ctypes.c_float, ctypes.c_void_p, ctypes.c_size_t
 _p_i64 = ctypes.POINTER(ctypes.c_int64)
@@ -26,7 +27,40 @@ class LinearArgs(ctypes.Structure):
                 ("row_sumsq", c_void_p), ("row_sumsq_ld", c_i64), ("row_sumsq_cols", c_i64), ("out", c_void_p), ("ld_out", c_i64),
                 ("act_split", c_i64), ("x", c_void_p), ("ld_x", c_i64), ("gain", c_void_p), ("gx", c_void_p), ("ld_gx", c_i64),
                 ("sumsq_out", c_void_p), ("sumsq_out_ld", c_i64), ("status_word", c_void_p), ("op_dtype", c_int), ("out_dtype", c_int),
-                ("row_sumsq_slices", c_int), ("act_lo", c_int), ("act_hi", c_int), ("eps", c_float), ("out_scale", c_float)]
+                ("row_sumsq_slices", c_int), ("act_lo", c_int), ("act_hi", c_int), ("eps", c_float), ("out_scale", c_float), ("bias", c_void_p), ("act_param", c_float)]
+
+
+def _fields(text):
+    """"type name name; type name" -> ctypes fields; ptr, i64, int and float."""
+    kinds = {"ptr": c_void_p, "i64": c_i64, "int": c_int, "float": c_float}
+    out = []
+    for part in text.split(";"):
+        kind, *names = part.split()
+        out += [(n, kinds[kind]) for n in names]
+    return out
+
+
+class StreamArgs(ctypes.Structure):
+    """b200_stream_args, field for field (as the classes below)."""
+
+    _fields_ = _fields("ptr x y; i64 ld_y; ptr y_gain ids table; i64 V; ptr shift gain h; i64 ld_h T W; float table_scale eps; int keep dtype")
+
+
+class RotaryArgs(ctypes.Structure):
+    _fields_ = _fields("ptr rows; i64 ld off_k off_v; ptr q_weight k_weight freq k_rows; i64 ld_k; ptr v_rows; i64 ld_v; ptr k_cache v_cache pos_dev; "
+                       "i64 B n q_heads kv_heads maps dim vdim rot_dims hist ring start; float eps; int dtype v_rows_dtype")
+
+
+class PairAttentionArgs(ctypes.Structure):
+    _fields_ = _fields("ptr q; i64 ld_q; ptr k; i64 k_batch k_head k_row; ptr v; i64 v_batch v_head v_row; ptr gate; i64 ld_gate; ptr lambda_ out; i64 ld_out; "
+                       "ptr pos_dev; i64 B n hist ring heads kv_heads dim vdim window; float scale softcap eps out_scale; int dtype v_dtype; ptr workspace; "
+                       "i64 workspace_bytes; ptr status_word")
+
+
+class DeltaArgs(ctypes.Structure):
+    _fields_ = _fields("ptr rows; i64 ld off_k off_v off_a off_b off_g; ptr conv_w conv_state; i64 conv_cols taps; ptr mixed; i64 ld_mixed; "
+                       "ptr norms gates a_log dt_bias norm_w state y; i64 ld_y; ptr pos_dev; i64 B n start heads kv_heads dim vdim; "
+                       "float eps unit_eps q_scale; int fresh dtype; ptr workspace; i64 workspace_bytes")
 
 
 # name -> (restype, argtypes); must list every function include/b200_gpt.h declares
@@ -71,6 +105,14 @@ SIGNATURES = {
     "b200_decayed_attention_workspace_bytes": (c_size_t, [c_i64] * 5 + [c_int]),
     "b200_decayed_attention": (c_int, [c_void_p] + [c_i64] * 4 + [c_void_p] * 3 + [c_int, c_void_p, c_i64, c_void_p] + [c_i64] * 6
                                + [c_int, c_void_p, c_size_t, c_void_p, c_void_p]),
+    "b200_stream_update": (c_int, [ctypes.POINTER(StreamArgs), c_void_p]),
+    "b200_gated_pairs": (c_int, [c_void_p, c_i64, c_void_p, c_i64, c_i64, c_i64, c_float, c_float, c_int, c_void_p]),
+    "b200_rotary_append": (c_int, [ctypes.POINTER(RotaryArgs), c_void_p]),
+    "b200_pair_attention_v_dtype": (c_int, [c_i64, c_i64, c_int]),
+    "b200_pair_attention_workspace_bytes": (c_i64, [ctypes.POINTER(PairAttentionArgs)]),
+    "b200_pair_attention": (c_int, [ctypes.POINTER(PairAttentionArgs), c_void_p]),
+    "b200_delta_workspace_bytes": (c_i64, [ctypes.POINTER(DeltaArgs)]),
+    "b200_delta": (c_int, [ctypes.POINTER(DeltaArgs), c_void_p]),
     "b200_selftest_bounded_wait": (c_int, [c_void_p, c_i64, c_void_p]),
 }
 

@@ -36,7 +36,7 @@ const char* b200_status_string(int status) {
 
 const char* b200_last_cuda_error(void) { return cudaGetErrorString(g_last_cuda); }
 
-int b200_abi_version(void) { return 7; }
+int b200_abi_version(void) { return 8; }
 
 uint64_t b200_launch_count(void) { return b200::launches_so_far(); }
 
@@ -247,7 +247,8 @@ int b200_linear(const b200_linear_args* args, void* stream) {
   if (p.out && p.ld_out < p.N) return B200_ERR_BAD_ARGUMENT;
   if (p.x && (p.ld_x < p.N || (p.gain && (!p.gx || p.ld_gx < p.N || !p.sumsq_out || p.sumsq_out_ld < p.M)))) return B200_ERR_BAD_ARGUMENT;
   if (p.row_sumsq && (p.row_sumsq_slices < 1 || p.row_sumsq_cols < 1 || p.row_sumsq_ld < p.M)) return B200_ERR_BAD_ARGUMENT;
-  if (p.act_lo < 0 || p.act_lo > B200_ACT_GELU_TANH || p.act_hi < 0 || p.act_hi > B200_ACT_GELU_TANH) return B200_ERR_BAD_ARGUMENT;
+  if (p.act_lo < 0 || p.act_lo > B200_ACT_SOFTCAP || p.act_hi < 0 || p.act_hi > B200_ACT_SOFTCAP) return B200_ERR_BAD_ARGUMENT;
+  if ((p.act_lo == B200_ACT_SOFTCAP || p.act_hi == B200_ACT_SOFTCAP) && !(p.act_param > 0.f)) return B200_ERR_BAD_ARGUMENT;
   return note(p.op_dtype == B200_F32 ? b200::launch_linear_f32(p, (cudaStream_t)stream) : b200::launch_linear_sm100(p, (cudaStream_t)stream));
 }
 
@@ -324,6 +325,87 @@ int b200_decayed_attention(const void* qkvg, int64_t ld, int64_t off_k, int64_t 
   if (need && (!workspace || workspace_bytes < need || (reinterpret_cast<uintptr_t>(workspace) & 255))) return B200_ERR_WORKSPACE;
   return note(b200::launch_decayed_attention(qkvg, ld, off_k, off_v, off_g, decay, weight, state, fresh, y, ld_y, sumsq, ld_sumsq, B, T, heads, dim, vdim,
                                              dtype, workspace, status_word, (cudaStream_t)stream));
+}
+
+// ------------------------------------------------------------------ decoders with a norm in front of and behind every sublayer
+int b200_stream_update(const b200_stream_args* args, void* stream) {
+  if (!args) return B200_ERR_BAD_ARGUMENT;
+  const b200_stream_args& p = *args;
+  if (p.T < 0 || p.T > kMaxExtent || p.W < 1 || !model_dtype(p.dtype) || (p.y && (!p.y_gain || p.ld_y < p.W)) || (p.gain && (!p.h || p.ld_h < p.W)))
+    return B200_ERR_BAD_ARGUMENT;
+  if (p.ids && (!p.table || p.V < 1)) return B200_ERR_BAD_ARGUMENT;
+  if (p.T == 0) return B200_OK;
+  if (!p.x) return B200_ERR_BAD_ARGUMENT;
+  return note(b200::launch_stream_update(p, (cudaStream_t)stream));
+}
+
+int b200_gated_pairs(const void* z, int64_t ld_z, void* out, int64_t ld_out, int64_t T, int64_t F, float limit, float alpha, int dtype, void* stream) {
+  if (T < 0 || F < 1 || ld_z < (F + 31) / 32 * 64 || ld_out < F || !model_dtype(dtype)) return B200_ERR_BAD_ARGUMENT;
+  if (T == 0) return B200_OK;
+  if (!z || !out) return B200_ERR_BAD_ARGUMENT;
+  return note(b200::launch_gated_pairs(z, ld_z, out, ld_out, T, F, limit, alpha, dtype, (cudaStream_t)stream));
+}
+
+int b200_rotary_append(const b200_rotary_args* args, void* stream) {
+  if (!args) return B200_ERR_BAD_ARGUMENT;
+  const b200_rotary_args& p = *args;
+  if (p.B < 0 || p.n < 0 || p.q_heads < 1 || p.kv_heads < 1 || p.maps < 1 || p.dim < 1 || p.vdim < 1 || p.hist < 0 || p.start < 0 || !model_dtype(p.dtype))
+    return B200_ERR_BAD_ARGUMENT;
+  if (p.rot_dims < 0 || p.rot_dims > p.dim || p.rot_dims % 2 || (p.rot_dims && !p.freq)) return B200_ERR_BAD_ARGUMENT;
+  if (p.off_k < p.q_heads * p.dim || p.off_v < p.off_k + p.kv_heads * p.maps * p.dim || p.ld < p.off_v + p.kv_heads * p.vdim) return B200_ERR_BAD_ARGUMENT;
+  if ((p.k_rows == nullptr) != (p.v_rows == nullptr) || (p.k_cache == nullptr) != (p.v_cache == nullptr)) return B200_ERR_BAD_ARGUMENT;
+  if (p.k_rows && (p.ld_k < p.kv_heads * p.maps * p.dim || p.ld_v < p.kv_heads * p.vdim)) return B200_ERR_BAD_ARGUMENT;
+  if (p.v_rows_dtype != p.dtype && !(p.v_rows_dtype == B200_F16 && p.dtype == B200_BF16)) return B200_ERR_BAD_ARGUMENT;
+  if (p.k_cache && p.ring < 1) return B200_ERR_BAD_ARGUMENT;
+  if (p.hist && (!p.k_rows || !p.k_cache || p.hist > p.ring || p.start < p.hist || p.pos_dev)) return B200_ERR_BAD_ARGUMENT;
+  if (p.B == 0 || p.n == 0) return B200_OK;
+  if (!p.rows || !p.q_weight || !p.k_weight || p.B * (p.hist + p.n) > kMaxExtent) return B200_ERR_BAD_ARGUMENT;
+  return note(b200::launch_rotary_append(p, (cudaStream_t)stream));
+}
+
+int b200_pair_attention_v_dtype(int64_t dim, int64_t vdim, int dtype) { return b200::pair_attention_v_dtype(dim, vdim, dtype); }
+
+int64_t b200_pair_attention_workspace_bytes(const b200_pair_attention_args* args) {
+  return args && args->B > 0 && args->kv_heads > 0 && args->heads > 0 ? b200::pair_attention_workspace_bytes(*args) : 0;
+}
+
+int b200_pair_attention(const b200_pair_attention_args* args, void* stream) {
+  if (!args) return B200_ERR_BAD_ARGUMENT;
+  const b200_pair_attention_args& p = *args;
+  if (p.B < 0 || p.n < 0 || p.hist < 0 || p.kv_heads < 1 || p.heads < p.kv_heads || p.heads % p.kv_heads || p.dim < 1 || p.vdim < 1 || p.window < 1 ||
+      !model_dtype(p.dtype))
+    return B200_ERR_BAD_ARGUMENT;
+  if (p.v_dtype != p.dtype && !(p.v_dtype == B200_F16 && p.dtype == B200_BF16)) return B200_ERR_BAD_ARGUMENT;
+  if (p.ld_q < 2 * p.heads * p.dim || p.ld_out < p.heads * p.vdim || p.ld_gate < p.heads || p.hist + p.n > kMaxExtent) return B200_ERR_BAD_ARGUMENT;
+  if (p.pos_dev ? (p.n != 1 || p.ring < 1 || p.window > p.ring) : p.ring != 0) return B200_ERR_BAD_ARGUMENT;
+  if (p.B == 0 || p.n == 0) return B200_OK;
+  if (!p.q || !p.k || !p.v || !p.gate || !p.lambda || !p.out) return B200_ERR_BAD_ARGUMENT;
+  const int64_t need = b200::pair_attention_workspace_bytes(p);
+  if (need && (!p.workspace || p.workspace_bytes < need || (reinterpret_cast<uintptr_t>(p.workspace) & 255))) return B200_ERR_WORKSPACE;
+  return note(b200::launch_pair_attention(p, (cudaStream_t)stream));
+}
+
+int64_t b200_delta_workspace_bytes(const b200_delta_args* args) {
+  return args && args->B > 0 && args->n > 0 && args->heads > 0 ? b200::delta_workspace_bytes(*args) : 0;
+}
+
+int b200_delta(const b200_delta_args* args, void* stream) {
+  if (!args) return B200_ERR_BAD_ARGUMENT;
+  const b200_delta_args& p = *args;
+  if (p.B < 0 || p.n < 0 || p.kv_heads < 1 || p.heads < p.kv_heads || p.heads % p.kv_heads || p.dim < 1 || p.vdim < 1 || p.taps < 1 || p.start < 0 ||
+      !model_dtype(p.dtype))
+    return B200_ERR_BAD_ARGUMENT;
+  const int64_t kd = p.kv_heads * p.dim, hv = p.heads * p.vdim;
+  if (p.off_k < kd || p.off_v < p.off_k + kd || p.conv_cols < p.off_v + hv || p.ld_mixed < p.conv_cols || p.ld_y < hv) return B200_ERR_BAD_ARGUMENT;
+  if (p.off_a < p.conv_cols || p.off_b < p.conv_cols || p.off_g < p.conv_cols || p.ld < p.off_a + p.heads || p.ld < p.off_b + p.heads || p.ld < p.off_g + hv)
+    return B200_ERR_BAD_ARGUMENT;
+  if (!p.fresh && !p.conv_state && p.taps > 1) return B200_ERR_BAD_ARGUMENT;
+  if (p.B == 0 || p.n == 0) return B200_OK;
+  if (!p.rows || !p.conv_w || !p.mixed || !p.norms || !p.gates || !p.a_log || !p.dt_bias || !p.norm_w || !p.state || !p.y || p.B * p.n > kMaxExtent)
+    return B200_ERR_BAD_ARGUMENT;
+  const int64_t need = b200::delta_workspace_bytes(p);
+  if (need && (!p.workspace || p.workspace_bytes < need || (reinterpret_cast<uintptr_t>(p.workspace) & 255))) return B200_ERR_WORKSPACE;
+  return note(b200::launch_delta(p, (cudaStream_t)stream));
 }
 
 int b200_selftest_bounded_wait(int* status_word, int64_t limit_cycles, void* stream) {

@@ -284,6 +284,15 @@ int launch_decayed_attention(const void* qkvg, int64_t ld, int64_t off_k, int64_
                              float* state, int fresh, void* y, int64_t ld_y, float* sumsq, int64_t ld_sumsq, int64_t B, int64_t T, int64_t heads,
                              int64_t dim, int64_t vdim, int dtype, void* workspace, int* status_word, cudaStream_t stream);
 
+int launch_stream_update(const b200_stream_args& p, cudaStream_t stream);
+int launch_gated_pairs(const void* z, int64_t ld_z, void* out, int64_t ld_out, int64_t T, int64_t F, float limit, float alpha, int dtype, cudaStream_t stream);
+int launch_rotary_append(const b200_rotary_args& p, cudaStream_t stream);
+int launch_pair_attention(const b200_pair_attention_args& p, cudaStream_t stream);
+int pair_attention_v_dtype(int64_t dim, int64_t vdim, int dtype);
+int64_t pair_attention_workspace_bytes(const b200_pair_attention_args& p);
+int64_t delta_workspace_bytes(const b200_delta_args& p);
+int launch_delta(const b200_delta_args& p, cudaStream_t stream);
+
 // One warp waiting (bounded) on a barrier that nothing completes: reports B200_ERR_DEVICE_WAIT through status_word.
 int launch_bounded_wait_selftest(int* status_word, int64_t limit_cycles, cudaStream_t stream);
 // tcgen05/TMA attention (head size 64, fp16); B200_ERR_UNSUPPORTED means "use the generic kernel".

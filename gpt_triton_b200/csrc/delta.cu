@@ -1,0 +1,163 @@
+// Gated delta rule.  Per head with an fp32 state S [dim, vdim], one decay g and one step size beta per token:
+//     S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
+// q, k, v pass a short causal convolution per channel and silu; q and k become unit vectors.
+//
+//   delta_inputs_kernel    convolution and silu (stored in the operand type), 1 / |q|, 1 / |k| of what is stored, log decays and
+//                          step sizes in fp32
+//   conv_store_kernel      the last inputs of the convolution into the ring that remembers them
+//   delta_any_kernel       the recurrence token by token, any sizes, both storage types, state in global memory
+#include "common.cuh"
+
+namespace b200 {
+namespace {
+
+__device__ __forceinline__ float silu_exact(float v) { return v / (1.0f + expf(-v)); }
+__device__ __forceinline__ float softplus_exact(float v) { return fmaxf(v, 0.f) + log1pf(expf(-fabsf(v))); }
+
+// ------------------------------------------------------------------ convolution, unit norms, gates
+constexpr int kInputWarps = 8, kInputTokens = 16;
+
+// One input of the convolution at position `pos` of sequence b: a row of this call, the ring's memory, or zero.
+template <typename T>
+__device__ __forceinline__ float conv_input(const b200_delta_args& p, int64_t b, int64_t t, int64_t pos, int64_t c) {
+  if (t >= 0) return to_float(static_cast<const T*>(p.rows)[(b * p.n + t) * p.ld + c]);
+  if (pos < 0) return 0.f;
+  return to_float(static_cast<const T*>(p.conv_state)[(b * p.taps + pos % p.taps) * p.conv_cols + c]);
+}
+
+template <typename T>
+__global__ void __launch_bounds__(32 * kInputWarps)
+delta_inputs_kernel(b200_delta_args p, int64_t tiles) {
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int64_t b = blockIdx.x / tiles, t0 = (blockIdx.x % tiles) * kInputTokens;
+  const int64_t start = p.pos_dev ? (int64_t)p.pos_dev[0] : p.start;
+  const int nt = (int)(p.n - t0 < kInputTokens ? p.n - t0 : kInputTokens);
+  const int64_t M = p.B * p.n;
+  const int taps = (int)p.taps;
+  const int sections = (int)(2 * p.kv_heads + p.heads);
+  for (int s = warp; s < sections; s += kInputWarps) {
+    const bool is_v = s >= 2 * p.kv_heads, is_k = !is_v && s >= p.kv_heads;
+    const int width = (int)(is_v ? p.vdim : p.dim);
+    const int64_t c0 = is_v ? p.off_v + (s - 2 * p.kv_heads) * p.vdim : is_k ? p.off_k + (s - p.kv_heads) * p.dim : s * p.dim;
+    for (int i = 0; i < nt; ++i) {
+      const int64_t t = t0 + i, row = b * p.n + t;
+      float sq = 0.f;
+      for (int c = lane; c < width; c += 32) {
+        float a = 0.f;
+        for (int k = 0; k < taps; ++k) {
+          const int64_t back = taps - 1 - k;
+          a = fmaf(p.conv_w[(c0 + c) * taps + k], conv_input<T>(p, b, t - back, start + t - back, c0 + c), a);
+        }
+        const T o = from_float<T>(silu_exact(a));
+        static_cast<T*>(p.mixed)[row * p.ld_mixed + c0 + c] = o;
+        const float f = to_float(o);
+        sq = fmaf(f, f, sq);
+      }
+      if (!is_v) {
+        sq = warp_sum(sq);
+        if (lane == 0) p.norms[(int64_t)s * M + row] = (is_k ? 1.0f : p.q_scale) / sqrtf(sq + p.unit_eps);
+      }
+    }
+  }
+  for (int64_t i = threadIdx.x; i < nt * p.heads; i += 32 * kInputWarps) {
+    const int64_t h = i / nt, row = b * p.n + t0 + i % nt;
+    const T* src = static_cast<const T*>(p.rows) + row * p.ld;
+    p.gates[h * M + row] = -expf(p.a_log[h]) * softplus_exact(to_float(src[p.off_a + h]) + p.dt_bias[h]);
+    p.gates[(p.heads + h) * M + row] = 1.0f / (1.0f + expf(-to_float(src[p.off_b + h])));
+  }
+}
+
+// Positions [end - (taps - 1), end) of this call's inputs into slot position % taps (a slot is read for at most taps - 1
+// positions, so the oldest one may be overwritten by the newest).
+template <typename T>
+__global__ void __launch_bounds__(256)
+conv_store_kernel(b200_delta_args p) {
+  const int64_t b = blockIdx.x;
+  const int64_t start = p.pos_dev ? (int64_t)p.pos_dev[0] : p.start;
+  const int64_t first = p.n > p.taps - 1 ? p.n - (p.taps - 1) : 0;
+  for (int64_t t = first; t < p.n; ++t) {
+    const T* src = static_cast<const T*>(p.rows) + (b * p.n + t) * p.ld;
+    T* dst = static_cast<T*>(p.conv_state) + (b * p.taps + (start + t) % p.taps) * p.conv_cols;
+    for (int64_t c = (int64_t)blockIdx.y * 256 + threadIdx.x; c < p.conv_cols; c += (int64_t)gridDim.y * 256) dst[c] = src[c];
+  }
+}
+
+// ------------------------------------------------------------------ token by token, any sizes
+constexpr int kAnyThreads = 128;
+template <typename T>
+__global__ void __launch_bounds__(kAnyThreads)
+delta_any_kernel(b200_delta_args p) {
+  extern __shared__ float smem_f[];
+  __shared__ float part[kAnyThreads / 32];
+  const int dim = (int)p.dim, vdim = (int)p.vdim;
+  float *qs = smem_f, *ks = qs + dim, *os = ks + dim;
+  const int64_t h = blockIdx.x % p.heads, b = blockIdx.x / p.heads, kv = h / (p.heads / p.kv_heads), M = p.B * p.n;
+  float* S = p.state + (b * p.heads + h) * (int64_t)dim * vdim;
+  const T* mixed = static_cast<const T*>(p.mixed);
+  for (int64_t t = 0; t < p.n; ++t) {
+    const int64_t row = b * p.n + t;
+    const T* src = mixed + row * p.ld_mixed;
+    const float rq = p.norms[kv * M + row], rk = p.norms[(p.kv_heads + kv) * M + row];
+    const float g = expf(p.gates[h * M + row]), beta = p.gates[(p.heads + h) * M + row];
+    for (int i = threadIdx.x; i < dim; i += kAnyThreads) qs[i] = to_float(src[kv * dim + i]) * rq, ks[i] = to_float(src[p.off_k + kv * dim + i]) * rk;
+    __syncthreads();
+    const bool zero = p.fresh && t == 0;
+    float sq = 0.f;
+    for (int c = threadIdx.x; c < vdim; c += kAnyThreads) {
+      float seen = 0.f;
+      if (!zero)
+        for (int i = 0; i < dim; ++i) seen = fmaf(S[(int64_t)i * vdim + c] * g, ks[i], seen);
+      const float u = beta * (to_float(src[p.off_v + h * vdim + c]) - seen);
+      float o = 0.f;
+      for (int i = 0; i < dim; ++i) {
+        const float s = fmaf(ks[i], u, zero ? 0.f : S[(int64_t)i * vdim + c] * g);
+        S[(int64_t)i * vdim + c] = s;
+        o = fmaf(s, qs[i], o);
+      }
+      os[c] = o;
+      sq = fmaf(o, o, sq);
+    }
+    sq = warp_sum(sq);
+    if ((threadIdx.x & 31) == 0) part[threadIdx.x >> 5] = sq;
+    __syncthreads();
+    sq = 0.f;
+    for (int i = 0; i < kAnyThreads / 32; ++i) sq += part[i];
+    const float inv = 1.0f / sqrtf(sq / (float)vdim + p.eps);
+    const T* gate = static_cast<const T*>(p.rows) + row * p.ld + p.off_g + h * vdim;
+    T* y = static_cast<T*>(p.y) + row * p.ld_y + h * vdim;
+    for (int c = threadIdx.x; c < vdim; c += kAnyThreads) y[c] = from_float<T>(os[c] * inv * p.norm_w[c] * to_float(gate[c]));
+    __syncthreads();
+  }
+}
+
+template <typename T>
+int launch_typed(const b200_delta_args& p, cudaStream_t stream) {
+  const int64_t tiles = (p.n + kInputTokens - 1) / kInputTokens;
+  if (p.B * tiles > 0x7fffffffLL || p.B * p.heads > 0x7fffffffLL) return B200_ERR_BAD_ARGUMENT;
+  delta_inputs_kernel<T><<<(unsigned)(p.B * tiles), 32 * kInputWarps, 0, stream>>>(p, tiles);
+  note_launches(1);
+  if (p.conv_state && p.taps > 1) {
+    int64_t cols = (p.conv_cols + 255) / 256;
+    if (cols > 64) cols = 64;
+    conv_store_kernel<T><<<dim3((unsigned)p.B, (unsigned)cols), 256, 0, stream>>>(p);
+    note_launches(1);
+  }
+  const size_t smem = (size_t)(2 * p.dim + p.vdim) * 4;
+  if (smem > 47 * 1024) return B200_ERR_UNSUPPORTED;
+  delta_any_kernel<T><<<(unsigned)(p.B * p.heads), kAnyThreads, smem, stream>>>(p);
+  note_launches(1);
+  return status_from_cuda(cudaGetLastError());
+}
+
+}  // namespace
+
+int64_t delta_workspace_bytes(const b200_delta_args& p) {
+  (void)p;
+  return 0;
+}
+
+int launch_delta(const b200_delta_args& p, cudaStream_t stream) {
+  return p.dtype == B200_BF16 ? launch_typed<__nv_bfloat16>(p, stream) : launch_typed<float>(p, stream);
+}
+
+}  // namespace b200

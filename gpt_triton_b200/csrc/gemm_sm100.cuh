@@ -173,6 +173,8 @@ struct EpilogueArgs {
   float sq_cols, eps, out_scale;
   int act_lo, act_hi;
   int64_t act_split;
+  float act_param;     // the activation's constant, for those that have one
+  const float* fbias;  // LN == 3, optional: added to row_scale * acc (fp32 [N], 16-byte aligned)
   float* x;
   int64_t ld_x;
   const float* gain;
@@ -271,8 +273,16 @@ __device__ __forceinline__ float sigmoid_fast(float x) {
   asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + e));
   return r;
 }
-__device__ __forceinline__ float activate(float v, int act) {
+// cap * tanh(v / cap) as cap - 2 cap / (1 + exp(2 v / cap)): exact to a few ulps of cap.
+__device__ __forceinline__ float softcap_fast(float v, float cap, float two_log2e_over_cap) {
+  float e, r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(v * two_log2e_over_cap));
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + e));
+  return fmaf(-2.0f * cap, r, cap);
+}
+__device__ __forceinline__ float activate(float v, int act, float param) {
   switch (act) {
+    case B200_ACT_SOFTCAP: return softcap_fast(v, param, 2.8853900817779268f / param);
     case B200_ACT_SILU: return v * sigmoid_fast(v);
     case B200_ACT_SIGMOID: return sigmoid_fast(v);
     case B200_ACT_GELU_TANH: return gelu_fast(v);
@@ -280,7 +290,7 @@ __device__ __forceinline__ float activate(float v, int act) {
   return v;
 }
 // The activation of 32 consecutive columns; which one is (almost always) uniform over the chunk.
-__device__ __forceinline__ void activate_chunk(float (&f)[32], int col0, int act_lo, int act_hi, int64_t split) {
+__device__ __forceinline__ void activate_chunk(float (&f)[32], int col0, int act_lo, int act_hi, int64_t split, float param) {
   const bool low = col0 + 32 <= split;
   if (low || col0 >= split) {
     switch (low ? act_lo : act_hi) {
@@ -296,10 +306,31 @@ __device__ __forceinline__ void activate_chunk(float (&f)[32], int col0, int act
 #pragma unroll
         for (int j = 0; j < 32; ++j) f[j] = gelu_fast(f[j]);
         break;
+      case B200_ACT_SOFTCAP: {
+        const float k = 2.8853900817779268f / param;
+#pragma unroll
+        for (int j = 0; j < 32; ++j) f[j] = softcap_fast(f[j], param, k);
+        break;
+      }
     }
   } else {
 #pragma unroll
-    for (int j = 0; j < 32; ++j) f[j] = activate(f[j], col0 + j < split ? act_lo : act_hi);
+    for (int j = 0; j < 32; ++j) f[j] = activate(f[j], col0 + j < split ? act_lo : act_hi, param);
+  }
+}
+
+// f += the fp32 bias of columns col0 .. col0 + 31 (the same addresses for the whole warp).
+__device__ __forceinline__ void add_bias_chunk(float (&f)[32], const float* bias, int col0, int64_t N) {
+  if (col0 + 32 <= N) {
+#pragma unroll
+    for (int j = 0; j < 32; j += 4) {
+      const float4 b = __ldg(reinterpret_cast<const float4*>(bias + col0 + j));
+      f[j] += b.x, f[j + 1] += b.y, f[j + 2] += b.z, f[j + 3] += b.w;
+    }
+  } else {
+#pragma unroll
+    for (int j = 0; j < 32; ++j)
+      if (col0 + j < N) f[j] += __ldg(bias + col0 + j);
   }
 }
 
@@ -455,7 +486,10 @@ __device__ __forceinline__ void epilogue_chunk(const uint32_t (&acc)[32], const 
       const float2 v2 = __fmul2_rn(make_float2(__uint_as_float(acc[j]), __uint_as_float(acc[j + 1])), r2);
       f[j] = v2.x, f[j + 1] = v2.y;
     }
-    if constexpr (LN == 3) activate_chunk(f, col0, e.act_lo, e.act_hi, e.act_split);
+    if constexpr (LN == 3) {
+      if (e.fbias) add_bias_chunk(f, e.fbias, col0, N);
+      activate_chunk(f, col0, e.act_lo, e.act_hi, e.act_split, e.act_param);
+    }
   } else if (e.bias) {
 #pragma unroll
     for (int j = 0; j < 32; j += 4) {

@@ -8,11 +8,12 @@ namespace {
 
 constexpr int TM = 64, TN = 64, TK = 16, PAD = 4;
 
-__device__ __forceinline__ float activate_exact(float v, int act) {
+__device__ __forceinline__ float activate_exact(float v, int act, float param) {
   switch (act) {
     case B200_ACT_SILU: return v / (1.0f + expf(-v));
     case B200_ACT_SIGMOID: return 1.0f / (1.0f + expf(-v));
     case B200_ACT_GELU_TANH: return 0.5f * v * (1.0f + tanhf(0.7978845608028654f * (v + 0.044715f * v * v * v)));
+    case B200_ACT_SOFTCAP: return param * tanhf(v / param);
   }
   return v;
 }
@@ -73,7 +74,8 @@ __global__ void __launch_bounds__(256) linear_f32_kernel(b200_linear_args p) {
         sq = fmaf(v, v, sq);
         if (p.gain) static_cast<float*>(p.gx)[row * p.ld_gx + col] = v * p.gain[col];
       } else {
-        static_cast<float*>(p.out)[row * p.ld_out + col] = activate_exact(v, col < p.act_split ? p.act_lo : p.act_hi);
+        static_cast<float*>(p.out)[row * p.ld_out + col] =
+            activate_exact(p.bias ? v + p.bias[col] : v, col < p.act_split ? p.act_lo : p.act_hi, p.act_param);
       }
     }
     if (p.x && p.gain) {  // (block-uniform) the 16 threads of a row are consecutive lanes

@@ -608,7 +608,7 @@ def sample_logits(logits, temperature=1.0, top_k=0, seed=0, step=None, out=None)
 
 # ----------------------------------------------------------------------------- RMS-normed decoders, fp32 residual stream
 # No counterpart in the reference.  bf16 runs on the tensor cores with fp32 accumulation; fp32 is true 32-bit.
-ACTIVATIONS = {None: 0, "silu": 1, "sigmoid": 2, "gelu_tanh": 3}
+ACTIVATIONS = {None: 0, "silu": 1, "sigmoid": 2, "gelu_tanh": 3, "softcap": 4}
 
 
 def _rows_empty(M, cols, dtype, device):
@@ -706,10 +706,15 @@ def embedding_rms(ids, table, gain, eps):
 
 
 @torch.no_grad()
-def linear(rows, weight, *, act=None, act_split=None, act_after=None, out_scale=1.0, out_dtype=None):
-    """act(norm(rows) @ weight^T * out_scale): rows a NormedRows or a plain (M, K) matrix, weight (N, K).  `act` applies to
-    the output columns below `act_split` (default: all), `act_after` to the rest."""
+def linear(rows, weight, *, bias=None, act=None, act_split=None, act_after=None, act_param=0.0, out_scale=1.0, out_dtype=None):
+    """act(norm(rows) @ weight^T * out_scale + bias): rows a NormedRows or a plain (M, K) matrix, weight (N, K), bias float32
+    (N,).  `act` applies to the output columns below `act_split` (default: all), `act_after` to the rest; `act_param`: the
+    constant of "softcap"."""
     p, a, dev = _linear_args(rows, weight)
+    if bias is not None:
+        assert bias.dtype == torch.float32 and bias.shape == (p.N,) and bias.is_contiguous() and bias.device == dev
+        p.bias = bias.data_ptr()
+    p.act_param = act_param
     out = _rows_empty(p.M, p.N, out_dtype or a.dtype, dev)
     p.out, p.ld_out, p.out_dtype = out.data_ptr(), max(out.stride(0), p.N), dtype_code(out.dtype)
     p.act_lo, p.act_hi = ACTIVATIONS[act], ACTIVATIONS[act_after]
@@ -840,3 +845,190 @@ def decayed_attention(qkvg, offsets, decay, weight, state, batch, heads, dim, vd
                                         _ptr(ws), need, _status_ptr(dev), stream_ptr(dev))
     check(st, "decayed_attention")
     return NormedRows(y, sumsq, heads * vdim, eps)
+
+
+# ----------------------------------------------------------------------------- decoders with a norm in front of and behind every sublayer
+def _pitch(t):
+    return max(t.stride(0), t.shape[1])
+
+
+@torch.no_grad()
+def stream_update(x, eps, *, y=None, y_gain=None, ids=None, table=None, table_scale=1.0, shift=None, gain=None, out_dtype=None):
+    """One pass over an fp32 stream between two sublayers: x += norm(y) * y_gain + table[ids] * table_scale + shift, each
+    optional, in place; with `gain` returns norm(x) * gain in `out_dtype`, the rows of the next product.  `x` an int: a new
+    stream of that many rows, starting from zero.  Returns (x, rows or None)."""
+    require_cuda(y, y_gain, ids, table, shift, gain)
+    p = _lib.StreamArgs()
+    if isinstance(x, int):
+        x = torch.empty((x, table.shape[1]), device=table.device, dtype=torch.float32)
+    else:
+        p.keep = 1
+    dev = _same_device(x, y, y_gain, ids, table, shift, gain)
+    p.T, p.W = x.shape
+    assert x.dtype == torch.float32 and x.is_contiguous()
+    p.x, p.eps, p.table_scale = x.data_ptr(), eps, table_scale
+    dtype = out_dtype or (y.dtype if y is not None else table.dtype)
+    for vec in (y_gain, shift, gain):
+        assert vec is None or (vec.dtype == torch.float32 and vec.shape == (p.W,) and vec.is_contiguous())
+    if y is not None:
+        assert y.shape == x.shape and y.stride(1) == 1 and y.dtype == dtype
+        p.y, p.ld_y, p.y_gain = y.data_ptr(), _pitch(y), y_gain.data_ptr()
+    if ids is not None:
+        assert ids.dtype == torch.int64 and ids.is_contiguous() and ids.numel() == p.T and table.is_contiguous() and table.dtype == dtype
+        p.ids, p.table, p.V = ids.data_ptr(), table.data_ptr(), table.shape[0]
+    p.shift, p.gain, p.dtype = _ptr(shift), _ptr(gain), dtype_code(dtype)
+    rows = None
+    if gain is not None:
+        rows = _rows_empty(p.T, p.W, dtype, dev)
+        p.h, p.ld_h = rows.data_ptr(), _pitch(rows)
+    with torch.cuda.device(dev):
+        check(_lib.load().b200_stream_update(ctypes.byref(p), stream_ptr(dev)), "stream_update")
+    return x, rows
+
+
+GATED_BLOCK = 32  # gate columns, then as many up columns
+
+
+def interleave_gated(gate, up):
+    """Weights (F, k) or biases (F,) of a gated feed-forward's two products as those of one, in the column order that
+    `gated_linear` reads: blocks of 32 gate rows and their 32 up rows, zero rows behind the last."""
+    F = gate.shape[0]
+    blocks = (F + GATED_BLOCK - 1) // GATED_BLOCK
+    pad = lambda t: torch.cat([t, t.new_zeros((blocks * GATED_BLOCK - F, *t.shape[1:]))]).view(blocks, 1, GATED_BLOCK, *t.shape[1:])
+    return torch.cat([pad(gate), pad(up)], dim=1).reshape(2 * blocks * GATED_BLOCK, *gate.shape[1:]).contiguous()
+
+
+@torch.no_grad()
+def gated_linear(rows, weight, bias, ff, *, limit, alpha):
+    """gate * sigmoid(alpha * gate) * (up + 1), gate = min(., limit) and up = clamp(., -limit, limit) being the two halves of
+    rows @ weight^T + bias, weight and bias from `interleave_gated`; (M, ff)."""
+    z = linear(rows, weight, bias=bias)
+    out = _rows_empty(z.shape[0], ff, z.dtype, z.device)
+    with torch.cuda.device(z.device):
+        st = _lib.load().b200_gated_pairs(z.data_ptr(), _pitch(z), out.data_ptr(), _pitch(out), z.shape[0], ff, limit, alpha, dtype_code(z.dtype), stream_ptr(z.device))
+    check(st, "gated_linear")
+    return out
+
+
+def rotary_frequencies(base, dims, device):
+    """base^(-2i / dims) for i < dims / 2 as (dims / 2, 2) float32: high and low part."""
+    f = torch.tensor([float(base) ** (-2.0 * i / dims) for i in range(dims // 2)], dtype=torch.float64)
+    hi = f.float()
+    return torch.stack([hi, (f - hi.double()).float()], dim=1).contiguous().to(device)
+
+
+@torch.no_grad()
+def rotary_append(qkv, offsets, q_weight, k_weight, freq, eps, batch, *, q_heads, kv_heads, maps, dim, vdim, cache=None, hist=0, start=0, pos=None,
+                  keep_rows=True, v_dtype=None):
+    """RMS norm per head and rotation by position of the queries (in place) and keys of qkv (batch * n, .), whose keys and
+    values start at the columns `offsets`.  They join `cache` = (keys (batch, kv_heads, ring, maps * dim), values (batch,
+    kv_heads, ring, vdim)) at the slots position % ring, the first position being `start`, or pos[0] on the device.  With
+    `keep_rows` returns (keys (batch * (hist + n), .), values): those of the `hist` tokens before them, then the new ones."""
+    require_cuda(qkv, q_weight, k_weight, freq, pos)
+    assert qkv.stride(1) == 1 and q_weight.dtype == k_weight.dtype == freq.dtype == torch.float32 and q_weight.shape == k_weight.shape == (dim,)
+    M = qkv.shape[0]
+    dev = _same_device(qkv, q_weight, k_weight, freq, pos)
+    p = _lib.RotaryArgs()
+    p.rows, p.ld, p.off_k, p.off_v = qkv.data_ptr(), _pitch(qkv), offsets[0], offsets[1]
+    p.q_weight, p.k_weight, p.freq, p.rot_dims = q_weight.data_ptr(), k_weight.data_ptr(), freq.data_ptr(), 2 * freq.shape[0]
+    p.B, p.n, p.q_heads, p.kv_heads, p.maps, p.dim, p.vdim = batch, M // batch, q_heads, kv_heads, maps, dim, vdim
+    p.hist, p.start, p.eps, p.dtype, p.pos_dev = hist, start, eps, dtype_code(qkv.dtype), _ptr(pos)
+    p.v_rows_dtype = dtype_code(v_dtype or qkv.dtype)
+    if cache is not None:
+        k_cache, v_cache = cache
+        assert k_cache.is_contiguous() and v_cache.is_contiguous() and k_cache.dtype == v_cache.dtype == qkv.dtype
+        assert k_cache.shape[:2] == v_cache.shape[:2] == (batch, kv_heads) and k_cache.shape[2] == v_cache.shape[2]
+        assert k_cache.shape[3] == maps * dim and v_cache.shape[3] == vdim
+        p.k_cache, p.v_cache, p.ring = k_cache.data_ptr(), v_cache.data_ptr(), k_cache.shape[2]
+    k = v = None
+    if keep_rows:
+        k = _rows_empty(batch * (hist + p.n), kv_heads * maps * dim, qkv.dtype, dev)
+        v = _rows_empty(batch * (hist + p.n), kv_heads * vdim, v_dtype or qkv.dtype, dev)
+        p.k_rows, p.ld_k, p.v_rows, p.ld_v = k.data_ptr(), _pitch(k), v.data_ptr(), _pitch(v)
+    with torch.cuda.device(dev):
+        check(_lib.load().b200_rotary_append(ctypes.byref(p), stream_ptr(dev)), "rotary_append")
+    return k, v
+
+
+def pair_attention_v_dtype(dim, vdim, dtype):
+    """The type in which `pair_attention` wants a prompt's values."""
+    return _lib.CODE_TO_TORCH[_lib.load().b200_pair_attention_v_dtype(dim, vdim, dtype_code(dtype))]
+
+
+@torch.no_grad()
+def pair_attention(q, k, v, gate, lam, batch, *, heads, kv_heads, dim, vdim, window, scale, softcap, eps, out_scale, pos=None):
+    """Differential attention with a sliding window: per head two softmax maps over the same values, a1 - lam * a2, RMS-normed
+    over vdim, times out_scale and the head's gate (batch * n, heads).  A prompt: q (batch * n, .) are the last n positions
+    of k, v (batch * m, .).  With `pos`: one token per sequence at position pos[0], k and v the caches of `rotary_append`."""
+    require_cuda(q, k, v, gate, lam, pos)
+    dev = _same_device(q, k, v, gate, lam, pos)
+    M = q.shape[0]
+    assert q.stride(1) == gate.stride(1) == 1 and q.dtype == k.dtype == gate.dtype and gate.shape == (M, heads) and lam.dtype == torch.float32
+    p = _lib.PairAttentionArgs()
+    p.q, p.ld_q, p.gate, p.ld_gate, p.lambda_ = q.data_ptr(), max(q.stride(0), 2 * heads * dim), gate.data_ptr(), max(gate.stride(0), heads), lam.data_ptr()
+    p.B, p.n, p.heads, p.kv_heads, p.dim, p.vdim = batch, M // batch, heads, kv_heads, dim, vdim
+    p.k, p.v = k.data_ptr(), v.data_ptr()
+    if pos is None:
+        m = k.shape[0] // batch
+        assert k.stride(1) == v.stride(1) == 1 and v.shape[0] == k.shape[0] and m >= p.n
+        p.hist, p.window = m - p.n, min(window, m)
+        p.k_row, p.v_row = _pitch(k), _pitch(v)
+        p.k_batch, p.k_head, p.v_batch, p.v_head = m * p.k_row, 2 * dim, m * p.v_row, vdim
+    else:
+        assert k.is_contiguous() and v.is_contiguous() and k.shape == (batch, kv_heads, k.shape[2], 2 * dim) and v.shape == (batch, kv_heads, k.shape[2], vdim)
+        p.ring = k.shape[2]
+        p.window, p.pos_dev = min(window, p.ring), pos.data_ptr()
+        p.k_row, p.v_row = 2 * dim, vdim
+        p.k_head, p.v_head = p.ring * p.k_row, p.ring * p.v_row
+        p.k_batch, p.v_batch = kv_heads * p.k_head, kv_heads * p.v_head
+    p.scale, p.softcap, p.eps, p.out_scale = scale, softcap, eps, out_scale
+    p.dtype, p.v_dtype, p.status_word = dtype_code(q.dtype), dtype_code(v.dtype), _status_ptr(dev)
+    out = _rows_empty(M, heads * vdim, q.dtype, dev)
+    p.out, p.ld_out = out.data_ptr(), _pitch(out)
+    lib = _lib.load()
+    p.workspace_bytes = lib.b200_pair_attention_workspace_bytes(ctypes.byref(p))
+    ws = torch.empty((p.workspace_bytes,), device=dev, dtype=torch.uint8) if p.workspace_bytes else None
+    p.workspace = _ptr(ws)
+    with torch.cuda.device(dev):
+        check(lib.b200_pair_attention(ctypes.byref(p), stream_ptr(dev)), "pair_attention")
+    return out
+
+
+# ----------------------------------------------------------------------------- gated delta rule
+UNIT_EPS = 1e-6
+
+
+@torch.no_grad()
+def gated_delta(rows, offsets, conv_w, a_log, dt_bias, norm_w, state, conv_state, batch, *, heads, kv_heads, dim, vdim, eps, q_scale, start=0, pos=None):
+    """Short convolutions, unit norms and the gated delta rule over the n tokens of each sequence, the output normed per head
+    and gated; (batch * n, heads * vdim).  rows (batch * n, .) holds q | k | v | a | b | gate from the columns 0 and `offsets`
+    on.  state (batch, heads, dim, vdim) float32 and conv_state (batch, taps, conv_cols) are updated in place (start 0 without
+    `pos`: both taken as zero); conv_state None: nothing is remembered."""
+    require_cuda(rows, conv_w, a_log, dt_bias, norm_w, state, conv_state, pos)
+    dev = _same_device(rows, conv_w, a_log, dt_bias, norm_w, state, conv_state, pos)
+    M = rows.shape[0]
+    assert rows.stride(1) == 1 and conv_w.is_contiguous() and state.is_contiguous() and state.shape == (batch, heads, dim, vdim)
+    assert all(t.dtype == torch.float32 for t in (conv_w, a_log, dt_bias, norm_w, state)) and norm_w.shape == (vdim,) and a_log.shape == dt_bias.shape == (heads,)
+    p = _lib.DeltaArgs()
+    p.rows, p.ld = rows.data_ptr(), _pitch(rows)
+    p.off_k, p.off_v, p.off_a, p.off_b, p.off_g = offsets
+    p.conv_w, (p.conv_cols, p.taps) = conv_w.data_ptr(), conv_w.shape
+    if conv_state is not None:
+        assert conv_state.is_contiguous() and conv_state.shape == (batch, p.taps, p.conv_cols) and conv_state.dtype == rows.dtype
+        p.conv_state = conv_state.data_ptr()
+    mixed = _rows_empty(M, p.conv_cols, rows.dtype, dev)
+    norms = torch.empty((2 * kv_heads, M), device=dev, dtype=torch.float32)
+    gates = torch.empty((2 * heads, M), device=dev, dtype=torch.float32)
+    y = _rows_empty(M, heads * vdim, rows.dtype, dev)
+    p.mixed, p.ld_mixed, p.norms, p.gates, p.y, p.ld_y = mixed.data_ptr(), _pitch(mixed), norms.data_ptr(), gates.data_ptr(), y.data_ptr(), _pitch(y)
+    p.a_log, p.dt_bias, p.norm_w, p.state, p.pos_dev = a_log.data_ptr(), dt_bias.data_ptr(), norm_w.data_ptr(), state.data_ptr(), _ptr(pos)
+    p.B, p.n, p.start, p.heads, p.kv_heads, p.dim, p.vdim = batch, M // batch, start, heads, kv_heads, dim, vdim
+    p.eps, p.unit_eps, p.q_scale, p.dtype = eps, UNIT_EPS, q_scale, dtype_code(rows.dtype)
+    p.fresh = int(pos is None and start == 0)
+    lib = _lib.load()
+    p.workspace_bytes = lib.b200_delta_workspace_bytes(ctypes.byref(p))
+    ws = torch.empty((p.workspace_bytes,), device=dev, dtype=torch.uint8) if p.workspace_bytes else None
+    p.workspace = _ptr(ws)
+    with torch.cuda.device(dev):
+        check(lib.b200_delta(ctypes.byref(p), stream_ptr(dev)), "gated_delta")
+    return y

@@ -44,6 +44,13 @@ def _fogilix(config, tensors):
     return Fogilix.from_checkpoint(config, tensors)
 
 
+@register("Nufasun")
+def _nufasun(config, tensors):
+    from .nufasun import Nufasun
+
+    return Nufasun.from_checkpoint(config, tensors)
+
+
 @register("GPT2Model", "GPT2LMHeadModel", "gpt2")
 def _gpt2(config, tensors):
     from .gpt import FusedGPT, convert_huggingface_to_triton

@@ -306,12 +306,13 @@ int b200_sample_logits(const void* logits, int64_t ld, int64_t B, int64_t V, int
  * sums of squares of x; the product that consumes the normed rows multiplies gx and applies 1 / sqrt(sum / cols + eps)
  * to the accumulator.  The rounding of gx is relative to each element, so this is as exact as rounding the normed row.
  */
-enum { B200_ACT_NONE = 0, B200_ACT_SILU = 1, B200_ACT_SIGMOID = 2, B200_ACT_GELU_TANH = 3 };
+enum { B200_ACT_NONE = 0, B200_ACT_SILU = 1, B200_ACT_SIGMOID = 2, B200_ACT_GELU_TANH = 3, B200_ACT_SOFTCAP = 4 };
 
 /*
  * acc = A [M,K] . B [N,K]^T (both K-major, op_dtype B200_BF16 on the tensor cores or B200_F32 in true 32-bit), then
  *   s[row] = out_scale / sqrt(sum_i row_sumsq[i * row_sumsq_ld + row] / row_sumsq_cols + eps)   (row_sumsq NULL: out_scale)
- *   x == NULL:  out[row, col] = act(s[row] * acc), act = act_lo for col < act_split, act_hi from there on;
+ *   x == NULL:  out[row, col] = act(s[row] * acc + bias[col]), act = act_lo for col < act_split, act_hi from there on (bias
+ *               fp32 [N], 16-byte aligned, NULL: none; B200_ACT_SOFTCAP: act_param * tanh(v / act_param));
  *   x != NULL:  x[row, col] += s[row] * acc (fp32, in place) and, if gain (fp32 [N]) is given, gx = op_dtype(gain[col] *
  *               new x) and sumsq_out[slice * sumsq_out_ld + row] = sum of (new x)^2 over slice's columns.  A slice is
  *               b200_linear_slice_cols(M, op_dtype) columns; the slices are added in order, so results are reproducible.
@@ -336,6 +337,8 @@ typedef struct {
   int* status_word;
   int op_dtype, out_dtype, row_sumsq_slices, act_lo, act_hi;
   float eps, out_scale;
+  const float* bias;
+  float act_param;
 } b200_linear_args;
 int64_t b200_linear_slice_cols(int64_t M, int op_dtype);
 int b200_linear(const b200_linear_args* args, void* stream);
@@ -400,6 +403,142 @@ size_t b200_decayed_attention_workspace_bytes(int64_t B, int64_t T, int64_t head
 int b200_decayed_attention(const void* qkvg, int64_t ld, int64_t off_k, int64_t off_v, int64_t off_g, const double* decay, const float* weight,
                            float* state, int fresh, void* y, int64_t ld_y, float* sumsq, int64_t ld_sumsq, int64_t B, int64_t T, int64_t heads,
                            int64_t dim, int64_t vdim, int dtype, void* workspace, size_t workspace_bytes, int* status_word, void* stream);
+
+/*
+ * ------------------------------------------------------------------------------------------------------------------
+ * Decoders with a norm in front of and behind every sublayer (no counterpart in the reference).
+ *
+ * One pass over the T rows of the fp32 stream x [T,W] (contiguous) between two sublayers:
+ *   x <- (keep ? x : 0) + norm(y) * y_gain + table[ids] * table_scale + shift
+ *   h <- dtype(norm(x) * gain)
+ * norm(r) = r / sqrt(mean(r^2) + eps); y, ids / table [V,W], shift [W] and gain are optional (NULL).  An id outside [0,V)
+ * adds nothing.  Gains and shift fp32 [W]; y, table and h of `dtype` (B200_BF16 or B200_F32).
+ */
+typedef struct {
+  float* x;
+  const void* y;
+  int64_t ld_y;
+  const float* y_gain;
+  const int64_t* ids;
+  const void* table;
+  int64_t V;
+  const float* shift;
+  const float* gain;
+  void* h;
+  int64_t ld_h, T, W;
+  float table_scale, eps;
+  int keep, dtype;
+} b200_stream_args;
+int b200_stream_update(const b200_stream_args* args, void* stream);
+
+/*
+ * out[row, j] = gate * sigmoid(alpha * gate) * (up + 1) with gate = min(z_gate, limit), up = clamp(z_up, -limit, limit).  The
+ * columns of z come in blocks of 64: the gates of 32 outputs, then their ups.  z [T, 64 * ceil(F / 32)], out [T, F].
+ */
+int b200_gated_pairs(const void* z, int64_t ld_z, void* out, int64_t ld_out, int64_t T, int64_t F, float limit, float alpha, int dtype, void* stream);
+
+/*
+ * Queries and keys behind their products.  Row b*n + t of rows (pitch ld) holds q_heads heads of dim columns from column 0,
+ * kv_heads * maps key heads from off_k and kv_heads value heads of vdim columns from off_v.  Every query and key head is
+ * RMS-normed (weights fp32 [dim]) and its column pairs (2i, 2i + 1), i < rot_dims / 2, are turned by position * f_i, f_i =
+ * freq[2i] + freq[2i + 1] (a frequency in two fp32 parts).  The first new token of a sequence has position start, or
+ * *pos_dev if pos_dev is not NULL.
+ *   queries  in place
+ *   keys and values  to the rows [hist, hist + n) of k_rows [B, hist + n, .] (pitch ld_k) and v_rows (pitch ld_v, dtype or
+ *            B200_F16), both NULL: nowhere; and, for the last min(n, ring) tokens, to the slots position % ring of
+ *            k_cache [B, kv_heads, ring, maps * dim] and v_cache [B, kv_heads, ring, vdim] (NULL: nowhere)
+ * hist > 0: the rows [0, hist) are filled from the caches first (positions [start - hist, start)).
+ */
+typedef struct {
+  void* rows;
+  int64_t ld, off_k, off_v;
+  const float* q_weight;
+  const float* k_weight;
+  const float* freq;
+  void* k_rows;
+  int64_t ld_k;
+  void* v_rows;
+  int64_t ld_v;
+  void* k_cache;
+  void* v_cache;
+  const int32_t* pos_dev;
+  int64_t B, n, q_heads, kv_heads, maps, dim, vdim, rot_dims, hist, ring, start;
+  float eps;
+  int dtype, v_rows_dtype;
+} b200_rotary_args;
+int b200_rotary_append(const b200_rotary_args* args, void* stream);
+
+/*
+ * Differential attention: head h has two query maps of dim columns (q columns 2*h*dim and (2*h + 1)*dim) and reads key/value
+ * head h / (heads / kv_heads), whose keys are two maps of dim columns and whose values of vdim columns serve both.
+ *   score = scale * q.k, then softcap * tanh(score / softcap) (softcap <= 0: as it is); softmax over the visible keys
+ *   o = a1 - *lambda * a2;  out = o / sqrt(mean(o^2) + eps) * out_scale * gate[row * ld_gate + h]
+ * Keys and values of sequence b, key/value head g, key j: k + b*k_batch + g*k_head + j*k_row (v alike; elements).
+ *   a prompt (pos_dev NULL): n queries per sequence, query t at key index hist + t, keys 0 .. hist + n - 1, ring 0
+ *   one token (n = 1): it stands at position *pos_dev and key j sits at j % ring
+ * A query sees itself and the window - 1 keys before it.  v of v_dtype: dtype, or B200_F16 beside B200_BF16 (what the
+ * tensor-core kernel for prompts reads; b200_pair_attention_v_dtype says which one is wanted).
+ */
+typedef struct {
+  const void* q;
+  int64_t ld_q;
+  const void* k;
+  int64_t k_batch, k_head, k_row;
+  const void* v;
+  int64_t v_batch, v_head, v_row;
+  const void* gate;
+  int64_t ld_gate;
+  const float* lambda;
+  void* out;
+  int64_t ld_out;
+  const int32_t* pos_dev;
+  int64_t B, n, hist, ring, heads, kv_heads, dim, vdim, window;
+  float scale, softcap, eps, out_scale;
+  int dtype, v_dtype;
+  void* workspace;
+  int64_t workspace_bytes;
+  int* status_word;
+} b200_pair_attention_args;
+int b200_pair_attention_v_dtype(int64_t dim, int64_t vdim, int dtype);
+int64_t b200_pair_attention_workspace_bytes(const b200_pair_attention_args* args);
+int b200_pair_attention(const b200_pair_attention_args* args, void* stream);
+
+/*
+ * Gated delta rule over n tokens per sequence.  Row b*n + t of rows (pitch ld) holds the raw projections: q, k (kv_heads *
+ * dim columns from 0 and off_k), v (heads * vdim, off_v), decay and step-size inputs a, b (heads each, off_a, off_b) and the
+ * output gate (heads * vdim, off_g).  q, k, v pass a causal convolution per channel (conv_w fp32 [conv_cols, taps], the last
+ * tap the current token's, channel = column) and silu; with unit(x) = x / sqrt(sum(x^2) + unit_eps), q <- q_scale * unit(q),
+ * k <- unit(k), per head, g = exp(-exp(a_log) softplus(a + dt_bias)), beta = sigmoid(b):
+ *   S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q;  y = o / sqrt(mean(o^2) + eps) * norm_w * gate
+ * head h reading q and k of head h / (heads / kv_heads).  state [B, heads, dim, vdim] fp32 and conv_state [B, taps, conv_cols]
+ * (inputs of the convolution, position % taps) are read (fresh != 0: taken as zero) and updated; conv_state NULL: not kept.
+ * mixed [B*n, .] (pitch ld_mixed >= conv_cols), norms fp32 [2 * kv_heads, B*n] and gates fp32 [2 * heads, B*n] are scratch.
+ */
+typedef struct {
+  const void* rows;
+  int64_t ld, off_k, off_v, off_a, off_b, off_g;
+  const float* conv_w;
+  void* conv_state;
+  int64_t conv_cols, taps;
+  void* mixed;
+  int64_t ld_mixed;
+  float* norms;
+  float* gates;
+  const float* a_log;
+  const float* dt_bias;
+  const float* norm_w;
+  float* state;
+  void* y;
+  int64_t ld_y;
+  const int32_t* pos_dev;
+  int64_t B, n, start, heads, kv_heads, dim, vdim;
+  float eps, unit_eps, q_scale;
+  int fresh, dtype;
+  void* workspace;
+  int64_t workspace_bytes;
+} b200_delta_args;
+int64_t b200_delta_workspace_bytes(const b200_delta_args* args);
+int b200_delta(const b200_delta_args* args, void* stream);
 
 /*
  * Self-test of the bounded waits every tensor-core kernel of this library uses (no reference counterpart): launches
