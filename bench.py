@@ -802,7 +802,7 @@ def fogilix_config(width, layers, vocab, kv_rank, window):
     return {"architecture": "Fogilix", "vocab": vocab, "width": width, "layers": out, "norm": {"eps": 1e-5}, "logit_scale": 1.0}
 
 
-def _random_parameters(model):
+def _random_parameters(model, plain_norms=False):
     with torch.no_grad():
         for name, prm in model.named_parameters():
             if prm.dim() == 2:
@@ -810,6 +810,8 @@ def _random_parameters(model):
             else:
                 prm.zero_()
                 if name.endswith("layer_norm_weight") or name.endswith("mix.norm") or name.endswith("dkv_norm"):
+                    prm.fill_(1.0)
+                elif plain_norms and "norm" in name:
                     prm.fill_(1.0)
     return model
 
@@ -865,7 +867,9 @@ def gpt_work(c, batch, n, cached, decode):
 
 _FAMILY = (("gemm_", "gemm"), ("argmax_reduce", "gemm"), ("ln_stats_from", "gemm"), ("attention_sm100", "attention"), ("attention_decode", "attention"),
            ("attention_kernel", "attention"), ("latent_append", "latents"), ("latent_gather", "latents"), ("latent_", "attention"),
-           ("head_product", "attention"), ("chunked_kernel", "lightning"), ("segment_scan", "lightning"), ("recurrent_kernel", "lightning"))
+           ("head_product", "attention"), ("chunked_kernel", "lightning"), ("segment_scan", "lightning"), ("recurrent_kernel", "lightning"),
+           ("stream_update", "stream"), ("embedding_rms", "stream"), ("gated_pairs", "gemm"), ("rotary", "rotary"), ("ring_gather", "rotary"),
+           ("pair_", "attention"), ("delta_", "delta"), ("conv_store", "delta"))
 
 
 def family_table(trace, work, peaks):
@@ -888,14 +892,74 @@ def family_table(trace, work, peaks):
     return out
 
 
-def run_fogilix(args):
-    """Prefill and decode throughput of the Fogilix decoder at a few sizes (random weights, bf16), beside a FusedGPT of the
-    same width, depth, feed-forward and vocabulary: one JSON line per size, with the time of each kernel family against its
+# Nufasun beside a Fogilix of the same width, depth and vocabulary (and the same number of feed-forward weights): attention and
+# delta layers in turn; heads of 2 x 64 query/key and 128 value columns, four per key/value head; delta heads of 128 x 128, two
+# per key head.
+NUFASUN_SIZES = {
+    "w1024": {"width": 1024, "layers": 8, "vocab": 32768, "window": 512},
+    "w2048": {"width": 2048, "layers": 8, "vocab": 32768, "window": 1024},
+    "w4096": {"width": 4096, "layers": 4, "vocab": 32768, "window": 1024},
+}
+
+
+def nufasun_config(width, layers, vocab, window):
+    heads, out = width // 128, []
+    for i in range(layers):
+        mlp = {"kind": "dense", "ff": round(8 * width / 3 / 64) * 64, "limit": 7.0}
+        if i % 2 == 0:
+            out.append({"type": "delta", "mixer": {"heads": heads, "kv_heads": heads // 2, "dim": 128, "vdim": 128, "conv": 4}, "mlp": mlp})
+        else:
+            mixer = {"heads": heads, "kv_heads": heads // 4, "dim": 64, "vdim": 128, "mask": {"size": window}, "diff": 0.6, "softcap": 30.0, "scale": 0.125,
+                     "rot": {"base": 1e5, "dims": 64}}
+            out.append({"type": "attention", "mixer": mixer, "mlp": mlp})
+    return {"architecture": "Nufasun", "vocab": vocab, "width": width, "layers": out, "norm": {"eps": 1e-6}, "embedding": {"scale": 1.0}, "logit_softcap": 15.0,
+            "loop": {"start": 0, "stop": layers, "times": 1}}
+
+
+def nufasun_work(cfg, batch, n, cached, decode):
+    """Algorithmic flop and bytes of one pass, by kernel family."""
+    T, w = batch * n, cfg["width"]
+    work = {k: [0.0, 0.0] for k in ("gemm", "attention", "delta", "stream", "rotary")}
+
+    def add(key, flop, nbytes):
+        work[key][0] += flop
+        work[key][1] += nbytes
+
+    product = lambda m, nn, k, out: add("gemm", 2.0 * m * nn * k, 2.0 * (m * k + nn * k + m * out))
+    for layer in cfg["layers"]:
+        m = layer["mixer"]
+        H, G, d, dv = m["heads"], m["kv_heads"], m["dim"], m["vdim"]
+        if layer["type"] == "delta":
+            cols = 2 * G * d + 2 * H * dv + 2 * H
+            product(T, cols, w, cols)
+            # the recurrence itself: S^T k, k u^T and S^T q per token; q, k, v, gate in, y out, the state once in and out
+            add("delta", 6.0 * T * H * d * dv, 2.0 * T * (2 * G * d + 3 * H * dv) + 8.0 * batch * H * d * dv)
+        else:
+            cols = 2 * H * d + G * (2 * d + dv) + H
+            product(T, cols, w, cols)
+            win = m["mask"]["size"]
+            keys = batch * (min(cached + 1, win) if decode else sum(min(i + 1, win) for i in range(n)))
+            kv = 2.0 * G * (2 * d + dv) * (keys if decode else T)
+            add("attention", 4.0 * keys * H * (d + dv), kv + 2.0 * T * (2 * H * d + H * dv))
+            add("rotary", 0.0, 4.0 * T * (2 * H * d + G * (2 * d + dv)))
+        product(T, w, H * dv, w)
+        ff = layer["mlp"]["ff"]
+        product(T, 2 * ff, w, ff)
+        product(T, w, ff, w)
+        add("stream", 0.0, 2 * T * w * 12.0)
+    product(batch, cfg["vocab"], w, 2 * cfg["vocab"])
+    return {k: tuple(v) for k, v in work.items()}
+
+
+def run_decoders(args, sizes, chosen, kinds):
+    """Prefill and decode throughput of a decoder at a few sizes (random weights, bf16), beside another model of the same
+    width, depth, feed-forward weights and vocabulary: one JSON line per size, with the time of each kernel family against its
     roofline.  Prefill: the prompt pass of a session (cache filled, first logits); decode: replays of the captured step."""
     from gpt_triton_b200 import kernels as K
     from gpt_triton_b200.fogilix import Fogilix, FogilixConfig
     from gpt_triton_b200.generation import GenerationSession
     from gpt_triton_b200.gpt import FusedGPT, GPTConfig
+    from gpt_triton_b200.nufasun import Nufasun, NufasunConfig
 
     dev = torch.device("cuda", 0)
     torch.cuda.set_device(dev)
@@ -913,20 +977,23 @@ def run_fogilix(args):
         torch.cuda.synchronize()
         return s.elapsed_time(e) / reps
 
-    for size in (args.fogilix_size.split(",") if args.fogilix_size else list(FOGILIX_SIZES)):
-        z = FOGILIX_SIZES[size]
-        line = {"model": f"fogilix_{size}", **z, "dtype": "bf16", "data": "synthetic", "peak_source": peak_src, "runs": []}
-        for kind in ("fogilix", "gpt"):
+    for size in (chosen.split(",") if chosen else list(sizes)):
+        z = sizes[size]
+        line = {"model": f"{kinds[0]}_{size}", **z, "dtype": "bf16", "data": "synthetic", "peak_source": peak_src, "runs": []}
+        for kind in kinds:
             torch.manual_seed(0)
             with torch.device(dev):
                 if kind == "fogilix":
-                    cfg = fogilix_config(**z)
+                    cfg = fogilix_config(**{"kv_rank": 256 if z["width"] <= 1024 else 512, **z})
                     model = Fogilix(FogilixConfig.from_dict(cfg))
+                elif kind == "nufasun":
+                    cfg = nufasun_config(**z)
+                    model = Nufasun(NufasunConfig.from_dict(cfg))
                 else:
                     cfg = GPTConfig(vocab_size=z["vocab"], block_size=4096, n_layer=z["layers"], n_head=z["width"] // 64, n_embd=z["width"])
                     model = FusedGPT(cfg)
-            model = _random_parameters(model).to(torch.bfloat16).eval()
-            count = lambda b, n, cached, dec: (fogilix_work if kind == "fogilix" else gpt_work)(cfg, b, n, cached, dec)
+            model = _random_parameters(model, plain_norms=kind == "nufasun").to(torch.bfloat16).eval()
+            count = lambda b, n, cached, dec: {"fogilix": fogilix_work, "nufasun": nufasun_work, "gpt": gpt_work}[kind](cfg, b, n, cached, dec)
             for batch, n in ((16, 2048), (1, 4096)):
                 ids = torch.randint(0, z["vocab"], (batch, n), device=dev)
                 sess = GenerationSession(model, batch, n)
@@ -997,9 +1064,14 @@ def main():
     ap.add_argument("--new-tokens", type=int, default=64, help="--decode: tokens generated per sequence")
     ap.add_argument("--fogilix", action="store_true", help="prefill and decode throughput of the Fogilix decoder beside a FusedGPT of equal size")
     ap.add_argument("--fogilix-size", default="", help=f"--fogilix: sizes to run, with commas between them (of {', '.join(FOGILIX_SIZES)}; default all)")
+    ap.add_argument("--nufasun", action="store_true", help="prefill and decode throughput of the Nufasun decoder beside a Fogilix of equal size")
+    ap.add_argument("--nufasun-size", default="", help=f"--nufasun: sizes to run, with commas between them (of {', '.join(NUFASUN_SIZES)}; default all)")
+    ap.add_argument("--alone", action="store_true", help="--fogilix, --nufasun: without the model beside it")
     args = ap.parse_args()
-    if args.fogilix:
-        run_fogilix(args)
+    if args.fogilix or args.nufasun:
+        kinds = ("fogilix", "gpt") if args.fogilix else ("nufasun", "fogilix")
+        sizes, chosen = (FOGILIX_SIZES, args.fogilix_size) if args.fogilix else (NUFASUN_SIZES, args.nufasun_size)
+        run_decoders(args, sizes, chosen, kinds[:1] if args.alone else kinds)
         return
     if args.decode:  # (with --gap-table: the per-kernel trace of one decode step instead of the timing line)
         run_decode(args)

@@ -94,8 +94,7 @@ int launch_any(const b200_pair_attention_args& p, cudaStream_t stream) {
 }  // namespace
 
 int pair_attention_v_dtype(int64_t dim, int64_t vdim, int dtype) {
-  (void)dim, (void)vdim;
-  return dtype;
+  return pair_attention_sm100_takes(dim, vdim, dtype) ? B200_F16 : dtype;
 }
 
 int64_t pair_attention_workspace_bytes(const b200_pair_attention_args& p) {
@@ -104,6 +103,10 @@ int64_t pair_attention_workspace_bytes(const b200_pair_attention_args& p) {
 }
 
 int launch_pair_attention(const b200_pair_attention_args& p, cudaStream_t stream) {
+  if (!p.pos_dev) {
+    const int st = launch_pair_attention_sm100(p, stream);
+    if (st != B200_ERR_UNSUPPORTED) return st;
+  }
   if (p.dtype == B200_F32) return launch_any<float, float>(p, stream);
   if (p.v_dtype == B200_F16) return launch_any<__nv_bfloat16, __half>(p, stream);
   return launch_any<__nv_bfloat16, __nv_bfloat16>(p, stream);

@@ -16,7 +16,9 @@ __device__ __forceinline__ float2 position_angle(float pos, float f_hi, float f_
   const float rest = fmaf(pos, f_hi, -a) + pos * f_lo;
   float s, c;
   sincosf(a, &s, &c);
-  return make_float2(fmaf(-s, rest, c), fmaf(c, rest, s));  // (cos, sin)
+  const float r2 = rest * rest;  // (|rest| is at most half a unit in the last place of a)
+  const float cr = fmaf(r2, fmaf(r2, 1.0f / 24.0f, -0.5f), 1.0f), sr = rest * fmaf(r2, -1.0f / 6.0f, 1.0f);
+  return make_float2(c * cr - s * sr, s * cr + c * sr);  // (cos, sin)
 }
 
 template <typename T>
