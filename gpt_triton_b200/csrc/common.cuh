@@ -295,6 +295,10 @@ int pair_attention_v_dtype(int64_t dim, int64_t vdim, int dtype);
 int64_t pair_attention_workspace_bytes(const b200_pair_attention_args& p);
 int64_t delta_workspace_bytes(const b200_delta_args& p);
 int launch_delta(const b200_delta_args& p, cudaStream_t stream);
+// Chunked version on tensor cores (delta_chunk.cu; bf16, enough tokens, heads up to 128 in multiples of 8).
+bool delta_chunk_takes(const b200_delta_args& p);
+int64_t delta_chunk_workspace_bytes(const b200_delta_args& p);
+int launch_delta_chunk(const b200_delta_args& p, cudaStream_t stream);
 
 // One warp waiting (bounded) on a barrier that nothing completes: reports B200_ERR_DEVICE_WAIT through status_word.
 int launch_bounded_wait_selftest(int* status_word, int64_t limit_cycles, cudaStream_t stream);

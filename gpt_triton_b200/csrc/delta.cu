@@ -2,10 +2,14 @@
 //     S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
 // q, k, v pass a short causal convolution per channel and silu; q and k become unit vectors.
 //
+// One token, a few tokens, or fp32 (heads up to 128 x 256):
+//   delta_step_kernel      everything in one kernel, token by token; the state of a head in the registers of one block
+// Many tokens, bf16 (delta_chunk.cu): 64 tokens at a time on the tensor cores.
+// Any other size:
 //   delta_inputs_kernel    convolution and silu (stored in the operand type), 1 / |q|, 1 / |k| of what is stored, log decays and
 //                          step sizes in fp32
-//   conv_store_kernel      the last inputs of the convolution into the ring that remembers them
-//   delta_any_kernel       the recurrence token by token, any sizes, both storage types, state in global memory
+//   delta_any_kernel       the recurrence token by token, state in global memory
+// conv_store_kernel puts the last inputs of the convolutions into the ring that remembers them.
 #include "common.cuh"
 
 namespace b200 {
@@ -130,31 +134,156 @@ delta_any_kernel(b200_delta_args p) {
   }
 }
 
-template <typename T>
-int launch_typed(const b200_delta_args& p, cudaStream_t stream) {
-  const int64_t tiles = (p.n + kInputTokens - 1) / kInputTokens;
-  if (p.B * tiles > 0x7fffffffLL || p.B * p.heads > 0x7fffffffLL) return B200_ERR_BAD_ARGUMENT;
-  delta_inputs_kernel<T><<<(unsigned)(p.B * tiles), 32 * kInputWarps, 0, stream>>>(p, tiles);
-  note_launches(1);
-  if (p.conv_state && p.taps > 1) {
-    int64_t cols = (p.conv_cols + 255) / 256;
-    if (cols > 64) cols = 64;
-    conv_store_kernel<T><<<dim3((unsigned)p.B, (unsigned)cols), 256, 0, stream>>>(p);
-    note_launches(1);
+// ------------------------------------------------------------------ token by token, the state in registers
+// One block per (sequence, head): four row groups of warps (ROWS = 16 or 32 state rows each) x one group per 32 columns.
+constexpr int kStepRowWarps = 4, kStepMaxCols = 256;
+
+template <typename T, int ROWS, int THREADS>
+__global__ void __launch_bounds__(THREADS, 1)
+delta_step_kernel(b200_delta_args p) {
+  constexpr int DIM = kStepRowWarps * ROWS;
+  __shared__ __align__(16) float qs[DIM], ks[DIM];
+  __shared__ float vs[kStepMaxCols], part[kStepRowWarps][kStepMaxCols], red[3][32];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, n_warps = blockDim.x >> 5;
+  const int rw = warp % kStepRowWarps, col = (warp / kStepRowWarps) * 32 + lane, row0 = rw * ROWS;
+  const int dim = (int)p.dim, vdim = (int)p.vdim, taps = (int)p.taps;
+  const int64_t h = blockIdx.x % p.heads, b = blockIdx.x / p.heads, group = p.heads / p.kv_heads, kv = h / group;
+  const int64_t start = p.pos_dev ? (int64_t)p.pos_dev[0] : p.start;
+  const bool col_ok = col < vdim;
+  float* st = p.state + (b * p.heads + h) * (int64_t)dim * vdim + col;
+  float s[ROWS];
+#pragma unroll
+  for (int i = 0; i < ROWS; ++i) s[i] = (!p.fresh && col_ok && row0 + i < dim) ? st[(int64_t)(row0 + i) * vdim] : 0.f;
+  const float decay_rate = -expf(p.a_log[h]), dt_bias = p.dt_bias[h];
+  const int channels = 2 * dim + vdim;
+  for (int64_t t = 0; t < p.n; ++t) {
+    const int64_t row = b * p.n + t;
+    const T* src = static_cast<const T*>(p.rows) + row * p.ld;
+    // convolutions and silu: q, then k, then v channels
+    float sq_q = 0.f, sq_k = 0.f;
+    for (int c = threadIdx.x; c < channels; c += blockDim.x) {
+      const int64_t col_in = c < dim ? kv * dim + c : c < 2 * dim ? p.off_k + kv * dim + (c - dim) : p.off_v + h * vdim + (c - 2 * dim);
+      float a = 0.f;
+      for (int k = 0; k < taps; ++k) {
+        const int64_t back = taps - 1 - k;
+        a = fmaf(p.conv_w[col_in * taps + k], conv_input<T>(p, b, t - back, start + t - back, col_in), a);
+      }
+      const float o = to_float(from_float<T>(silu_exact(a)));
+      if (c < dim) qs[c] = o, sq_q = fmaf(o, o, sq_q);
+      else if (c < 2 * dim) ks[c - dim] = o, sq_k = fmaf(o, o, sq_k);
+      else vs[c - 2 * dim] = o;
+    }
+    // (rows of the state beyond dim see a key and a query of zero)
+    for (int c = dim + threadIdx.x; c < DIM; c += blockDim.x) qs[c] = 0.f, ks[c] = 0.f;
+    sq_q = warp_sum(sq_q), sq_k = warp_sum(sq_k);
+    if (lane == 0) red[0][warp] = sq_q, red[1][warp] = sq_k;
+    const float g = expf(decay_rate * softplus_exact(to_float(src[p.off_a + h]) + dt_bias));
+    const float beta = 1.0f / (1.0f + expf(-to_float(src[p.off_b + h])));
+    __syncthreads();
+    float rq = 0.f, rk = 0.f;
+    for (int i = 0; i < n_warps; ++i) rq += red[0][i], rk += red[1][i];
+    rq = p.q_scale / sqrtf(rq + p.unit_eps), rk = 1.0f / sqrtf(rk + p.unit_eps);
+    float seen = 0.f;
+#pragma unroll
+    for (int i = 0; i < ROWS; i += 4) {
+      const float4 k4 = *reinterpret_cast<const float4*>(&ks[row0 + i]);
+      s[i] *= g, s[i + 1] *= g, s[i + 2] *= g, s[i + 3] *= g;
+      seen = fmaf(s[i], k4.x, fmaf(s[i + 1], k4.y, fmaf(s[i + 2], k4.z, fmaf(s[i + 3], k4.w, seen))));
+    }
+    part[rw][col] = seen;
+    __syncthreads();
+    seen = (part[0][col] + part[1][col]) + (part[2][col] + part[3][col]);
+    const float u = col_ok ? beta * (vs[col] - seen * rk) * rk : 0.f;
+    float o = 0.f;
+#pragma unroll
+    for (int i = 0; i < ROWS; i += 4) {
+      const float4 k4 = *reinterpret_cast<const float4*>(&ks[row0 + i]);
+      const float4 q4 = *reinterpret_cast<const float4*>(&qs[row0 + i]);
+      s[i] = fmaf(k4.x, u, s[i]), o = fmaf(s[i], q4.x, o);
+      s[i + 1] = fmaf(k4.y, u, s[i + 1]), o = fmaf(s[i + 1], q4.y, o);
+      s[i + 2] = fmaf(k4.z, u, s[i + 2]), o = fmaf(s[i + 2], q4.z, o);
+      s[i + 3] = fmaf(k4.w, u, s[i + 3]), o = fmaf(s[i + 3], q4.w, o);
+    }
+    __syncthreads();  // everyone has read the first partial sums
+    part[rw][col] = o;
+    __syncthreads();
+    o = ((part[0][col] + part[1][col]) + (part[2][col] + part[3][col])) * rq;
+    // norm over the head: the first row group's warps hold every column once
+    const float sq = warp_sum(rw == 0 && col_ok ? o * o : 0.f);
+    if (lane == 0) red[2][warp] = sq;
+    __syncthreads();
+    if (rw == 0 && col_ok) {
+      float total = 0.f;
+      for (int i = 0; i < n_warps; i += kStepRowWarps) total += red[2][i];
+      const float inv = 1.0f / sqrtf(total / (float)vdim + p.eps);
+      static_cast<T*>(p.y)[row * p.ld_y + h * vdim + col] = from_float<T>(o * inv * p.norm_w[col] * to_float(src[p.off_g + h * vdim + col]));
+    }
+    // (qs, ks, vs are written again only after everyone has passed the last barrier; red[2] behind the next token's first)
   }
-  const size_t smem = (size_t)(2 * p.dim + p.vdim) * 4;
-  if (smem > 47 * 1024) return B200_ERR_UNSUPPORTED;
-  delta_any_kernel<T><<<(unsigned)(p.B * p.heads), kAnyThreads, smem, stream>>>(p);
+#pragma unroll
+  for (int i = 0; i < ROWS; ++i)
+    if (col_ok && row0 + i < dim) st[(int64_t)(row0 + i) * vdim] = s[i];
+  if (p.n == 1 && p.conv_state && taps > 1) {
+    // this token's inputs take a slot that no block reads in this step; a key head's channels are its first value head's to store
+    const T* src = static_cast<const T*>(p.rows) + b * p.ld;
+    T* dst = static_cast<T*>(p.conv_state) + (b * taps + start % taps) * p.conv_cols;
+    for (int c = threadIdx.x; c < channels; c += blockDim.x) {
+      if (c < 2 * dim && h % group) continue;
+      const int64_t col_in = c < dim ? kv * dim + c : c < 2 * dim ? p.off_k + kv * dim + (c - dim) : p.off_v + h * vdim + (c - 2 * dim);
+      dst[col_in] = src[col_in];
+    }
+  }
+}
+
+bool takes_step(const b200_delta_args& p) {
+  return p.dim <= 128 && p.vdim <= kStepMaxCols;
+}
+
+template <typename T>
+int launch_step(const b200_delta_args& p, cudaStream_t stream) {
+  const unsigned threads = 32 * kStepRowWarps * (unsigned)((p.vdim + 31) / 32), blocks = (unsigned)(p.B * p.heads);
+  if (p.dim <= 64 && threads <= 512) delta_step_kernel<T, 16, 512><<<blocks, threads, 0, stream>>>(p);
+  else if (p.dim <= 64) delta_step_kernel<T, 16, 1024><<<blocks, threads, 0, stream>>>(p);
+  else if (threads <= 512) delta_step_kernel<T, 32, 512><<<blocks, threads, 0, stream>>>(p);
+  else delta_step_kernel<T, 32, 1024><<<blocks, threads, 0, stream>>>(p);
   note_launches(1);
   return status_from_cuda(cudaGetLastError());
 }
 
+template <typename T>
+int launch_store(const b200_delta_args& p, cudaStream_t stream) {
+  if (!p.conv_state || p.taps < 2) return B200_OK;
+  int64_t cols = (p.conv_cols + 255) / 256;
+  if (cols > 64) cols = 64;
+  conv_store_kernel<T><<<dim3((unsigned)p.B, (unsigned)cols), 256, 0, stream>>>(p);
+  note_launches(1);
+  return status_from_cuda(cudaGetLastError());
+}
+
+template <typename T>
+int launch_typed(const b200_delta_args& p, cudaStream_t stream) {
+  const int64_t tiles = (p.n + kInputTokens - 1) / kInputTokens;
+  if (p.B > 65535 || p.B * tiles > 0x7fffffffLL || p.B * p.heads > 0x7fffffffLL) return B200_ERR_BAD_ARGUMENT;
+  int st = B200_OK;
+  if (delta_chunk_takes(p)) {
+    st = launch_delta_chunk(p, stream);
+  } else if (takes_step(p)) {
+    st = launch_step<T>(p, stream);
+    if (p.n == 1) return st;
+  } else {
+    const size_t smem = (size_t)(2 * p.dim + p.vdim) * 4;
+    if (smem > 47 * 1024) return B200_ERR_UNSUPPORTED;
+    delta_inputs_kernel<T><<<(unsigned)(p.B * tiles), 32 * kInputWarps, 0, stream>>>(p, tiles);
+    delta_any_kernel<T><<<(unsigned)(p.B * p.heads), kAnyThreads, smem, stream>>>(p);
+    note_launches(2);
+    st = status_from_cuda(cudaGetLastError());
+  }
+  return st == B200_OK ? launch_store<T>(p, stream) : st;
+}
+
 }  // namespace
 
-int64_t delta_workspace_bytes(const b200_delta_args& p) {
-  (void)p;
-  return 0;
-}
+int64_t delta_workspace_bytes(const b200_delta_args& p) { return delta_chunk_takes(p) ? delta_chunk_workspace_bytes(p) : 0; }
 
 int launch_delta(const b200_delta_args& p, cudaStream_t stream) {
   return p.dtype == B200_BF16 ? launch_typed<__nv_bfloat16>(p, stream) : launch_typed<float>(p, stream);
