@@ -18,7 +18,7 @@ CSRC = os.path.join(PKG_DIR, "csrc")
 OBJ_DIR = os.path.join(PKG_DIR, "_obj")
 LIB_PATH = os.path.join(PKG_DIR, "libb200gpt.so")
 SOURCES = ["api.cu", "elementwise.cu", "gemm_sm100.cu", "linear_sm100.cu", "linear_f32.cu", "attention.cu", "attention_sm100.cu", "latent.cu",
-           "latent_decode.cu", "lightning.cu", "stream.cu", "rotary.cu", "pair_attention.cu", "pair_attention_sm100.cu", "delta.cu", "delta_chunk.cu", "decode.cu", "ffn_static_scratch.cu", "selftest.cu"]
+           "latent_decode.cu", "lightning.cu", "stream.cu", "rotary.cu", "pair_attention.cu", "pair_attention_sm100.cu", "pair_decode.cu", "delta.cu", "delta_chunk.cu", "decode.cu", "ffn_static_scratch.cu", "selftest.cu"]
 HEADERS = [os.path.join(CSRC, "common.cuh"), os.path.join(CSRC, "sm100_primitives.cuh"), os.path.join(CSRC, "gemm_sm100.cuh"),
            os.path.join(CSRC, "mma_sync.cuh"), os.path.join(CSRC, "attention_sm100.cuh"),
            os.path.join(os.path.dirname(PKG_DIR), "include", "b200_gpt.h")]

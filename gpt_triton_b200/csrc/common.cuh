@@ -291,6 +291,8 @@ int launch_pair_attention(const b200_pair_attention_args& p, cudaStream_t stream
 // tcgen05/TMA version for prompts (bf16, head sizes up to 128 in multiples of 8); B200_ERR_UNSUPPORTED: the any-size kernel.
 bool pair_attention_sm100_takes(int64_t dim, int64_t vdim, int dtype);
 int launch_pair_attention_sm100(const b200_pair_attention_args& p, cudaStream_t stream);
+// One token per sequence on tensor cores, same sizes.
+int launch_pair_decode(const b200_pair_attention_args& p, cudaStream_t stream);
 int pair_attention_v_dtype(int64_t dim, int64_t vdim, int dtype);
 int64_t pair_attention_workspace_bytes(const b200_pair_attention_args& p);
 int64_t delta_workspace_bytes(const b200_delta_args& p);

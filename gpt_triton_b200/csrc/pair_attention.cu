@@ -1,5 +1,6 @@
 // Differential attention: per head two softmax maps over the same values, subtracted, normed and gated; sliding window,
-// grouped key/value heads, soft-capped scores.  The kernel of this file takes any sizes, both storage types, prompts and
+// grouped key/value heads, soft-capped scores.  Prompts run pair_attention_sm100.cu and single tokens pair_decode.cu where they
+// fit; the kernel of this file takes any sizes, both storage types, prompts and
 // single tokens; fp32 storage is computed in true 32-bit throughout.
 #include "common.cuh"
 
@@ -103,10 +104,8 @@ int64_t pair_attention_workspace_bytes(const b200_pair_attention_args& p) {
 }
 
 int launch_pair_attention(const b200_pair_attention_args& p, cudaStream_t stream) {
-  if (!p.pos_dev) {
-    const int st = launch_pair_attention_sm100(p, stream);
-    if (st != B200_ERR_UNSUPPORTED) return st;
-  }
+  const int st = p.pos_dev ? launch_pair_decode(p, stream) : launch_pair_attention_sm100(p, stream);
+  if (st != B200_ERR_UNSUPPORTED) return st;
   if (p.dtype == B200_F32) return launch_any<float, float>(p, stream);
   if (p.v_dtype == B200_F16) return launch_any<__nv_bfloat16, __half>(p, stream);
   return launch_any<__nv_bfloat16, __nv_bfloat16>(p, stream);
