@@ -27,7 +27,8 @@ class LinearArgs(ctypes.Structure):
                 ("row_sumsq", c_void_p), ("row_sumsq_ld", c_i64), ("row_sumsq_cols", c_i64), ("out", c_void_p), ("ld_out", c_i64),
                 ("act_split", c_i64), ("x", c_void_p), ("ld_x", c_i64), ("gain", c_void_p), ("gx", c_void_p), ("ld_gx", c_i64),
                 ("sumsq_out", c_void_p), ("sumsq_out_ld", c_i64), ("status_word", c_void_p), ("op_dtype", c_int), ("out_dtype", c_int),
-                ("row_sumsq_slices", c_int), ("act_lo", c_int), ("act_hi", c_int), ("eps", c_float), ("out_scale", c_float), ("bias", c_void_p), ("act_param", c_float)]
+                ("row_sumsq_slices", c_int), ("act_lo", c_int), ("act_hi", c_int), ("eps", c_float), ("out_scale", c_float), ("bias", c_void_p), ("act_param", c_float),
+                ("pair_limit", c_float), ("pair_alpha", c_float), ("pair_cols", c_i64)]
 
 
 def _fields(text):

@@ -244,7 +244,8 @@ int b200_linear(const b200_linear_args* args, void* stream) {
   if (p.M < 0 || p.N < 0 || p.K < 1 || p.M > kMaxExtent || p.N > kMaxExtent || p.K > kMaxExtent || !valid_dtype(p.op_dtype)) return B200_ERR_BAD_ARGUMENT;
   if (p.M == 0 || p.N == 0) return B200_OK;
   if (!p.a || !p.b || p.lda < p.K || p.ldb < p.K || (p.x == nullptr) == (p.out == nullptr)) return B200_ERR_BAD_ARGUMENT;
-  if (p.out && p.ld_out < p.N) return B200_ERR_BAD_ARGUMENT;
+  if (p.pair_cols < 0 || (p.pair_cols && (p.x || p.N != (p.pair_cols + 31) / 32 * 64))) return B200_ERR_BAD_ARGUMENT;
+  if (p.out && p.ld_out < (p.pair_cols ? p.pair_cols : p.N)) return B200_ERR_BAD_ARGUMENT;
   if (p.x && (p.ld_x < p.N || (p.gain && (!p.gx || p.ld_gx < p.N || !p.sumsq_out || p.sumsq_out_ld < p.M)))) return B200_ERR_BAD_ARGUMENT;
   if (p.row_sumsq && (p.row_sumsq_slices < 1 || p.row_sumsq_cols < 1 || p.row_sumsq_ld < p.M)) return B200_ERR_BAD_ARGUMENT;
   if (p.act_lo < 0 || p.act_lo > B200_ACT_SOFTCAP || p.act_hi < 0 || p.act_hi > B200_ACT_SOFTCAP) return B200_ERR_BAD_ARGUMENT;

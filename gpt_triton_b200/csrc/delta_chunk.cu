@@ -26,7 +26,7 @@ using namespace warp_mma;
 constexpr int kC = 64;  // tokens per chunk
 
 // ------------------------------------------------------------------ convolution and silu
-constexpr int kConvTokens = 16;
+constexpr int kConvTokens = 16, kConvBatch = 4;  // tokens per thread, loads in flight
 // One thread: 8 channels of kConvTokens tokens of one sequence; the last TAPS - 1 inputs stay in registers.
 template <int TAPS>
 __global__ void __launch_bounds__(128)
@@ -50,24 +50,31 @@ delta_conv_kernel(b200_delta_args p, int vecs) {
     if (t >= 0) load8(rows + t * p.ld, x[k]);
     else if (pos >= 0) load8(ring + pos % TAPS * p.conv_cols, x[k]);
   }
+  for (int i0 = 0; i0 < kConvTokens; i0 += kConvBatch) {
+    uint4 raw[kConvBatch];
 #pragma unroll
-  for (int i = 0; i < kConvTokens; ++i) {
-    const int64_t t = t0 + i;
-    if (t >= p.n) break;
-    load8(rows + t * p.ld, x[TAPS - 1]);
-    float o[8];
-#pragma unroll
-    for (int e = 0; e < 8; ++e) {
-      float a = 0.f;
-#pragma unroll
-      for (int k = 0; k < TAPS; ++k) a = fmaf(w[k][e], x[k][e], a);
-      o[e] = a / (1.0f + __expf(-a));
+    for (int i = 0; i < kConvBatch; ++i) {
+      const int64_t t = t0 + i0 + i;
+      raw[i] = t < p.n ? __ldg(reinterpret_cast<const uint4*>(rows + t * p.ld)) : make_uint4(0, 0, 0, 0);
     }
-    store8(out + t * p.ld_mixed, o);
 #pragma unroll
-    for (int k = 0; k + 1 < TAPS; ++k)
+    for (int i = 0; i < kConvBatch; ++i) {
+      const int64_t t = t0 + i0 + i;
+      load8(reinterpret_cast<const __nv_bfloat16*>(&raw[i]), x[TAPS - 1]);
+      float o[8];
 #pragma unroll
-      for (int e = 0; e < 8; ++e) x[k][e] = x[k + 1][e];
+      for (int e = 0; e < 8; ++e) {
+        float a = 0.f;
+#pragma unroll
+        for (int k = 0; k < TAPS; ++k) a = fmaf(w[k][e], x[k][e], a);
+        o[e] = __fdividef(a, 1.0f + __expf(-a));
+      }
+      if (t < p.n) store8(out + t * p.ld_mixed, o);
+#pragma unroll
+      for (int k = 0; k + 1 < TAPS; ++k)
+#pragma unroll
+        for (int e = 0; e < 8; ++e) x[k][e] = x[k + 1][e];
+    }
   }
 }
 template <int TAPS>

@@ -173,6 +173,10 @@ struct EpilogueArgs {
   float sq_cols, eps, out_scale;
   int act_lo, act_hi;
   int64_t act_split;
+  // LN == 5: the columns come in blocks of 64, 32 gate columns and their 32 up columns (z = row_scale * acc + fbias); out
+  // [M, pair_cols] = gate * sigmoid(pair_alpha * gate) * (up + 1), gate = min(z, limit), up = clamp(z, -limit, limit)
+  int64_t pair_cols;
+  float pair_limit, pair_alpha;
   float act_param;     // the activation's constant, for those that have one
   const float* fbias;  // LN == 3, optional: added to row_scale * acc (fp32 [N], 16-byte aligned)
   float* x;
@@ -464,6 +468,50 @@ __device__ __forceinline__ bool residual_rows_wide(const EpilogueArgs<OutT>& e) 
   const uintptr_t gal = e.gain ? (reinterpret_cast<uintptr_t>(e.gx) | (uintptr_t)(e.ld_gx * 2)) : 0;
   const uintptr_t nal = e.gain ? (reinterpret_cast<uintptr_t>(e.gain) & 15) : 0;
   return ((al | gal) & 31) == 0 && nal == 0;
+}
+
+// LN == 5, one thread, one row: a block of 32 gate and 32 up accumulators (column col0 of the product on) -> 32 outputs, to this
+// thread's row of a staging box (`stage` != 0, 16-byte slots [4 * half, 4 * half + 4)) or to global memory.
+template <typename OutT>
+__device__ __forceinline__ void gated_pair_chunk(const uint32_t (&za)[32], const uint32_t (&zb)[32], const EpilogueArgs<OutT>& e, int64_t row, int col0,
+                                                 float row_scale, uint32_t stage, int half, int lane, bool vec_ok) {
+  uint32_t w[16];
+#pragma unroll
+  for (int j = 0; j < 32; j += 4) {
+    float4 ba = make_float4(0.f, 0.f, 0.f, 0.f), bb = ba;
+    if (e.fbias) {
+      ba = __ldg(reinterpret_cast<const float4*>(e.fbias + col0 + j));
+      bb = __ldg(reinterpret_cast<const float4*>(e.fbias + col0 + 32 + j));
+    }
+    const float b0[4] = {ba.x, ba.y, ba.z, ba.w}, b1[4] = {bb.x, bb.y, bb.z, bb.w};
+    float f[4];
+#pragma unroll
+    for (int i = 0; i < 4; ++i) {
+      const float g = fminf(fmaf(__uint_as_float(za[j + i]), row_scale, b0[i]), e.pair_limit);
+      const float u = fminf(fmaxf(fmaf(__uint_as_float(zb[j + i]), row_scale, b1[i]), -e.pair_limit), e.pair_limit);
+      f[i] = g * sigmoid_fast(e.pair_alpha * g) * (u + 1.0f);
+    }
+    w[j / 2] = pack2<OutT>(f[0], f[1]), w[j / 2 + 1] = pack2<OutT>(f[2], f[3]);
+  }
+  if (stage != 0) {
+    const uint32_t rowaddr = stage + (uint32_t)lane * 128u, sw = (uint32_t)(lane & 7);
+#pragma unroll
+    for (int g = 0; g < 4; ++g) st_shared_v4(rowaddr + ((((uint32_t)(half * 4 + g)) ^ sw) << 4), w[4 * g], w[4 * g + 1], w[4 * g + 2], w[4 * g + 3]);
+    return;
+  }
+  const int64_t out0 = col0 / 2;
+  OutT* orow = e.out + row * e.ld_out + out0;
+  if (vec_ok && out0 + 32 <= e.pair_cols) {
+#pragma unroll
+    for (int g = 0; g < 4; ++g) *reinterpret_cast<uint4*>(orow + g * 8) = make_uint4(w[4 * g], w[4 * g + 1], w[4 * g + 2], w[4 * g + 3]);
+  } else {
+#pragma unroll
+    for (int j = 0; j < 16; ++j) {
+      const float2 v = unpack2<OutT>(w[j]);
+      if (out0 + 2 * j < e.pair_cols) orow[2 * j] = from_float<OutT>(v.x);
+      if (out0 + 2 * j + 1 < e.pair_cols) orow[2 * j + 1] = from_float<OutT>(v.y);
+    }
+  }
 }
 
 // One thread, one row, 32 consecutive columns starting at col0: acc (+bias) -> GELU -> (+residual) -> out.
@@ -758,7 +806,7 @@ __device__ __forceinline__ void stats_only_chunk(const uint32_t (&acc)[32], cons
 
 // LN: 0 = plain; 1 = a LayerNorm of A's rows is folded into the epilogue (EpilogueArgs::ln_*); 2 = the epilogue also
 // emits per-slice row moments of what it stores (EpilogueArgs::stats_out), which a following LN == 1 GEMM consumes;
-// 3 / 4 = products around a deferred RMS norm (EpilogueArgs::sq_in ...).
+// 3 / 4 = products around a deferred RMS norm (EpilogueArgs::sq_in ...); 5 = gated pairs of columns (EpilogueArgs::pair_cols).
 template <typename OutT, bool GELU, int CTAS, int STATS, int LN>
 __global__ void __launch_bounds__(NUM_THREADS, 1)
 gemm_tn_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant__ CUtensorMap map_b,
@@ -1018,8 +1066,35 @@ gemm_tn_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_constant_
           tgt = (t64 >= col_base && t64 < col_base + EPI_COLS) ? (int)t64 : -1;
         }
       }
+      if constexpr (LN == 5) {
+        // 128 columns of the product are 64 of the output: one staging box per tile, the two of a warp taking turns
+        const uint32_t box = stage_addr + (uint32_t)acc * EPI_BOX_BYTES;
+        if (lane == 0) tma_store_wait_read_but_one();
+        __syncwarp();
+#pragma unroll
+        for (int c = 0; c < EPI_CHUNKS; c += 2) {
+          uint32_t za[32], zb[32];
+          tmem_ld_32x32(taddr + (uint32_t)(c * 32), za);
+          tmem_ld_32x32(taddr + (uint32_t)(c * 32 + 32), zb);
+          tmem_ld_wait();
+          if (c == EPI_CHUNKS - 2) {
+            tc_fence_before();
+            __syncwarp();
+            if (lane == 0) {
+              if constexpr (CTAS == 2) mbar_arrive_cluster(acc_empty_base + 8 * acc); else mbar_arrive(bar_acc_empty + 8 * acc);
+            }
+          }
+          if (col_base + c * 32 < N) gated_pair_chunk(za, zb, epi, row, col_base + c * 32, ln_r, box, c >> 1, lane, true);
+        }
+        fence_proxy_async_smem();
+        __syncwarp();
+        if (lane == 0) {
+          if (col_base / 2 < epi.pair_cols && row_warp < M) tma_store_2d(&map_out, box, col_base / 2, row_warp);
+          tma_store_commit();
+        }
+      }
 #pragma unroll(STATS == 2 ? 1 : EPI_CHUNKS)  // argmax + log-sum-exp + store: rolled, or the unrolled body spills
-      for (int c = 0; c < EPI_CHUNKS; ++c) {
+      for (int c = 0; c < (LN == 5 ? 0 : EPI_CHUNKS); ++c) {
         uint32_t v[32];
         tmem_ld_32x32(taddr + (uint32_t)(c * 32), v);
         tmem_ld_wait();
@@ -1269,8 +1344,17 @@ gemm_narrow_kernel(const __grid_constant__ CUtensorMap map_a, const __grid_const
       tc_fence_after();
       RowStats unused{-INFINITY, 0, 0.f, -1};
       SliceMoments mom{0.f, 0.f, 0.f, 0.f};
+      if constexpr (LN == 5) {
+        static_assert(NARROW_BN == 64, "one block of gate and up columns per tile");
+        uint32_t za[32], zb[32];
+        const uint32_t at = tmem_d + ((uint32_t)(quarter * 32) << 16);
+        tmem_ld_32x32(at, za);
+        tmem_ld_32x32(at + 32u, zb);
+        tmem_ld_wait();
+        if (row_ok) gated_pair_chunk(za, zb, epi, row, n0, ln_r, 0u, 0, lane, mode != STORE_SCALAR);
+      }
 #pragma unroll
-      for (int c = 0; c < NARROW_BN / 32; ++c) {
+      for (int c = 0; c < (LN == 5 ? 0 : NARROW_BN / 32); ++c) {
         const int col0 = n0 + c * 32;
         if (col0 >= N) break;  // (warp-uniform)
         uint32_t v[32];
@@ -1432,10 +1516,10 @@ static int launch_wide(const void* a, const void* b, EpilogueArgs<OutT> epi, int
   // TMA epilogue: 16-bit output (and residual, if any) with 16-byte aligned base and pitch
   if (STATS != 3 && LN != 4 && sizeof(OutT) == 2 && (reinterpret_cast<uintptr_t>(epi.out) & 15) == 0 && epi.ld_out % 8 == 0 &&
       (!epi.residual || ((reinterpret_cast<uintptr_t>(epi.residual) & 15) == 0 && epi.ld_res % 8 == 0)) &&
-      make_out_map(&mo, epi.out, M, N, epi.ld_out, DType<OutT>::code) == B200_OK &&
+      make_out_map(&mo, epi.out, M, LN == 5 ? epi.pair_cols : N, epi.ld_out, DType<OutT>::code) == B200_OK &&
       (!epi.residual || make_out_map(&mr, const_cast<OutT*>(epi.residual), M, N, epi.ld_res, DType<OutT>::code) == B200_OK))
     epi.tma_store = 1;
-  if ((LN == 1 || LN == 2) && !epi.tma_store) return B200_ERR_UNSUPPORTED;  // the LayerNorm-aware epilogues exist on the staged 16-bit path only
+  if ((LN == 1 || LN == 2 || LN == 5) && !epi.tma_store) return B200_ERR_UNSUPPORTED;  // these epilogues exist on the staged 16-bit path only
   epi.stream_out = epi.tma_store && (double)N * (double)K * 2.0 >= 32e6 && (double)M * (double)N * sizeof(OutT) >= 512e6;
   const int64_t n_tiles = (N + BN - 1) / BN;
   const int pairs = M > BM ? max_pairs<OutT, GELU, STATS, LN>() : 0;

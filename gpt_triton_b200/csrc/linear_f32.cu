@@ -91,7 +91,7 @@ __global__ void __launch_bounds__(256) linear_f32_kernel(b200_linear_args p) {
 int64_t linear_f32_slice_cols() { return TN; }
 
 int launch_linear_f32(const b200_linear_args& p, cudaStream_t stream) {
-  if (!p.x && p.out_dtype != B200_F32) return B200_ERR_UNSUPPORTED;
+  if ((!p.x && p.out_dtype != B200_F32) || p.pair_cols) return B200_ERR_UNSUPPORTED;
   const int64_t nb = (p.N + TN - 1) / TN, mb = (p.M + TM - 1) / TM;
   if (mb > 65535) return B200_ERR_BAD_ARGUMENT;
   linear_f32_kernel<<<dim3((unsigned)nb, (unsigned)mb), 256, 0, stream>>>(p);

@@ -1,5 +1,5 @@
 // 16-bit instantiations of the tcgen05 GEMM behind b200_linear: products over rows whose RMS norm is deferred to the
-// epilogue (gemm_sm100.cuh, LN == 3 and 4).
+// epilogue (gemm_sm100.cuh, LN == 3 and 4), and the gated pairs of a feed-forward (LN == 5).
 #include "gemm_sm100.cuh"
 
 namespace b200 {
@@ -22,6 +22,7 @@ int fill_and_launch(const b200_linear_args& p, cudaStream_t stream) {
   e.eps = p.eps, e.out_scale = p.out_scale;
   e.act_lo = p.act_lo, e.act_hi = p.act_hi, e.act_split = p.act_split;
   e.act_param = p.act_param, e.fbias = p.bias;
+  e.pair_cols = p.pair_cols, e.pair_limit = p.pair_limit, e.pair_alpha = p.pair_alpha;
   e.x = p.x, e.ld_x = p.ld_x, e.gain = p.gain, e.gx = static_cast<__nv_bfloat16*>(p.gx), e.ld_gx = p.ld_gx;
   e.sq_out = p.sumsq_out, e.sq_out_ld = p.sumsq_out_ld;
   return launch<OutT, LN>(p, e, stream);
@@ -36,6 +37,7 @@ int launch_linear_sm100(const b200_linear_args& p, cudaStream_t stream) {
   if ((reinterpret_cast<uintptr_t>(p.a) & 15) || (reinterpret_cast<uintptr_t>(p.b) & 15) || p.lda % 8 || p.ldb % 8) return B200_ERR_ALIGNMENT;
   if (reinterpret_cast<uintptr_t>(p.bias) & 15) return B200_ERR_ALIGNMENT;
   if (p.x) return fill_and_launch<float, 4>(p, stream);
+  if (p.pair_cols) return p.out_dtype == B200_BF16 ? fill_and_launch<__nv_bfloat16, 5>(p, stream) : B200_ERR_UNSUPPORTED;
   if (p.out_dtype == B200_BF16) return fill_and_launch<__nv_bfloat16, 3>(p, stream);
   if (p.out_dtype == B200_F32) return fill_and_launch<float, 3>(p, stream);
   return B200_ERR_UNSUPPORTED;

@@ -902,10 +902,19 @@ def interleave_gated(gate, up):
 def gated_linear(rows, weight, bias, ff, *, limit, alpha):
     """gate * sigmoid(alpha * gate) * (up + 1), gate = min(., limit) and up = clamp(., -limit, limit) being the two halves of
     rows @ weight^T + bias, weight and bias from `interleave_gated`; (M, ff)."""
+    p, a, dev = _linear_args(rows, weight)
+    out = _rows_empty(p.M, ff, a.dtype, dev)
+    lib = _lib.load()
+    if a.dtype == torch.bfloat16:  # in the product's epilogue
+        assert bias.dtype == torch.float32 and bias.shape == (p.N,) and bias.is_contiguous() and bias.device == dev
+        p.out, p.ld_out, p.out_dtype, p.act_split = out.data_ptr(), _pitch(out), dtype_code(out.dtype), p.N
+        p.bias, p.pair_cols, p.pair_limit, p.pair_alpha = bias.data_ptr(), ff, limit, alpha
+        with torch.cuda.device(dev):
+            check(lib.b200_linear(ctypes.byref(p), stream_ptr(dev)), "gated_linear")
+        return out
     z = linear(rows, weight, bias=bias)
-    out = _rows_empty(z.shape[0], ff, z.dtype, z.device)
-    with torch.cuda.device(z.device):
-        st = _lib.load().b200_gated_pairs(z.data_ptr(), _pitch(z), out.data_ptr(), _pitch(out), z.shape[0], ff, limit, alpha, dtype_code(z.dtype), stream_ptr(z.device))
+    with torch.cuda.device(dev):
+        st = lib.b200_gated_pairs(z.data_ptr(), _pitch(z), out.data_ptr(), _pitch(out), p.M, ff, limit, alpha, dtype_code(z.dtype), stream_ptr(dev))
     check(st, "gated_linear")
     return out
 

@@ -316,6 +316,8 @@ enum { B200_ACT_NONE = 0, B200_ACT_SILU = 1, B200_ACT_SIGMOID = 2, B200_ACT_GELU
  *   x != NULL:  x[row, col] += s[row] * acc (fp32, in place) and, if gain (fp32 [N]) is given, gx = op_dtype(gain[col] *
  *               new x) and sumsq_out[slice * sumsq_out_ld + row] = sum of (new x)^2 over slice's columns.  A slice is
  *               b200_linear_slice_cols(M, op_dtype) columns; the slices are added in order, so results are reproducible.
+ *   pair_cols > 0 (bf16 in and out, x NULL): N = 64 * ceil(pair_cols / 32), the columns of s[row] * acc + bias in the order that
+ *               b200_gated_pairs reads, and out [M, pair_cols] is what it computes with pair_limit and pair_alpha.
  * bf16: A and B 16-byte aligned, lda and ldb multiples of 8.  out_dtype: op_dtype or B200_F32.
  */
 typedef struct {
@@ -338,7 +340,8 @@ typedef struct {
   int op_dtype, out_dtype, row_sumsq_slices, act_lo, act_hi;
   float eps, out_scale;
   const float* bias;
-  float act_param;
+  float act_param, pair_limit, pair_alpha;
+  int64_t pair_cols;
 } b200_linear_args;
 int64_t b200_linear_slice_cols(int64_t M, int op_dtype);
 int b200_linear(const b200_linear_args* args, void* stream);
