@@ -2,7 +2,9 @@
 //     S <- g S;  u = beta (v - S^T k);  S <- S + k u^T;  o = S^T q
 // q, k, v pass a short causal convolution per channel and silu; q and k become unit vectors.
 //
-// One token, a few tokens, or fp32 (heads up to 128 x 256):
+// One token:
+//   delta_token_kernel     everything in one kernel, the state through shared memory (heads up to 256 columns each)
+// A few tokens, or fp32 (heads up to 128 x 256):
 //   delta_step_kernel      everything in one kernel, token by token; the state of a head in the registers of one block
 // Many tokens, bf16 (delta_chunk.cu): 64 tokens at a time on the tensor cores.
 // Any other size:
@@ -10,6 +12,8 @@
 //                          step sizes in fp32
 //   delta_any_kernel       the recurrence token by token, state in global memory
 // conv_store_kernel puts the last inputs of the convolutions into the ring that remembers them.
+#include <atomic>
+
 #include "common.cuh"
 
 namespace b200 {
@@ -235,6 +239,127 @@ delta_step_kernel(b200_delta_args p) {
   }
 }
 
+// ------------------------------------------------------------------ one token, the state through shared memory
+// One block per (sequence, head).  The state is on its way into shared memory (asynchronous copies: several blocks per SM
+// have theirs in flight) while the convolutions run; a warp takes every eighth row, a lane four columns of 128.
+constexpr int kTokenThreads = 256, kTokenWarps = kTokenThreads / 32, kTokenMaxDim = 256;
+
+template <typename T>
+__global__ void __launch_bounds__(kTokenThreads)
+delta_token_kernel(b200_delta_args p) {
+  extern __shared__ __align__(16) float S[];  // [dim][vdim], then partial sums [warps][128]
+  __shared__ float qs[kTokenMaxDim], ks[kTokenMaxDim], vs[kStepMaxCols], os[kStepMaxCols], red[2][kTokenWarps];
+  const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31;
+  const int dim = (int)p.dim, vdim = (int)p.vdim, taps = (int)p.taps;
+  const int heads = (int)p.heads, h = (int)(blockIdx.x % heads), group = heads / (int)p.kv_heads, kv = h / group;
+  const int64_t b = blockIdx.x / heads;
+  const int start = p.pos_dev ? p.pos_dev[0] : (int)p.start;
+  float* st = p.state + (b * heads + h) * (int64_t)dim * vdim;
+  float* part = S + dim * vdim;
+  for (int i = threadIdx.x; i < dim * vdim / 4; i += kTokenThreads)
+    asm volatile("cp.async.cg.shared.global [%0], [%1], 16;" ::"r"((uint32_t)__cvta_generic_to_shared(S + i * 4)), "l"(st + i * 4) : "memory");
+  asm volatile("cp.async.commit_group;" ::: "memory");
+  const T* src = static_cast<const T*>(p.rows) + b * p.ld;
+  T* ring = static_cast<T*>(p.conv_state) + b * taps * p.conv_cols;
+  const int slot = start % taps;  // this token's; the one before it is one slot down
+  float sq_q = 0.f, sq_k = 0.f;
+  for (int c = threadIdx.x; c < 2 * dim + vdim; c += kTokenThreads) {
+    const int64_t col = c < dim ? (int64_t)kv * dim + c : c < 2 * dim ? p.off_k + kv * dim + (c - dim) : p.off_v + h * vdim + (c - 2 * dim);
+    const float* w = p.conv_w + col * taps;
+    const T now = src[col];
+    float a = w[taps - 1] * to_float(now);
+    for (int back = 1; back < taps; ++back)
+      if (start >= back) a = fmaf(w[taps - 1 - back], to_float(ring[(int64_t)(slot >= back ? slot - back : slot - back + taps) * p.conv_cols + col]), a);
+    // (no block reads this slot in this step; a key head's channels are its first value head's to store)
+    if (taps > 1 && p.conv_state && (c >= 2 * dim || h % group == 0)) ring[(int64_t)slot * p.conv_cols + col] = now;
+    const float o = to_float(from_float<T>(silu_exact(a)));
+    if (c < dim) qs[c] = o, sq_q = fmaf(o, o, sq_q);
+    else if (c < 2 * dim) ks[c - dim] = o, sq_k = fmaf(o, o, sq_k);
+    else vs[c - 2 * dim] = o;
+  }
+  sq_q = warp_sum(sq_q), sq_k = warp_sum(sq_k);
+  if (lane == 0) red[0][warp] = sq_q, red[1][warp] = sq_k;
+  const float g = expf(-expf(p.a_log[h]) * softplus_exact(to_float(src[p.off_a + h]) + p.dt_bias[h]));
+  const float beta = 1.0f / (1.0f + expf(-to_float(src[p.off_b + h])));
+  asm volatile("cp.async.wait_group 0;" ::: "memory");
+  __syncthreads();
+  float rq = 0.f, rk = 0.f;
+#pragma unroll
+  for (int i = 0; i < kTokenWarps; ++i) rq += red[0][i], rk += red[1][i];
+  rq = p.q_scale / sqrtf(rq + p.unit_eps), rk = 1.0f / sqrtf(rk + p.unit_eps);
+  // a lane's four columns, summed over the warps' rows
+  auto meet = [&](float4 x) -> float4 {
+    __syncthreads();
+    *reinterpret_cast<float4*>(part + warp * 128 + lane * 4) = x;
+    __syncthreads();
+    float4 s = make_float4(0.f, 0.f, 0.f, 0.f);
+#pragma unroll
+    for (int i = 0; i < kTokenWarps; ++i) {
+      const float4 y = *reinterpret_cast<const float4*>(part + i * 128 + lane * 4);
+      s.x += y.x, s.y += y.y, s.z += y.z, s.w += y.w;
+    }
+    return s;
+  };
+  float sq = 0.f;
+  for (int c0 = 0; c0 < vdim; c0 += 128) {
+    const int c = c0 + lane * 4;
+    const bool ok = c < vdim;
+    float4 seen = make_float4(0.f, 0.f, 0.f, 0.f);
+    if (ok) {
+#pragma unroll 4
+      for (int r = warp; r < dim; r += kTokenWarps) {
+        const float4 x = *reinterpret_cast<const float4*>(S + r * vdim + c);
+        const float k = ks[r];
+        seen.x = fmaf(x.x, k, seen.x), seen.y = fmaf(x.y, k, seen.y), seen.z = fmaf(x.z, k, seen.z), seen.w = fmaf(x.w, k, seen.w);
+      }
+    }
+    seen = meet(seen);
+    const float f = g * rk, bk = beta * rk;
+    float4 u = make_float4(0.f, 0.f, 0.f, 0.f), o = u;
+    if (ok) {
+      u = make_float4(bk * (vs[c] - f * seen.x), bk * (vs[c + 1] - f * seen.y), bk * (vs[c + 2] - f * seen.z), bk * (vs[c + 3] - f * seen.w));
+#pragma unroll 4
+      for (int r = warp; r < dim; r += kTokenWarps) {
+        float4 x = *reinterpret_cast<const float4*>(S + r * vdim + c);
+        const float k = ks[r], q = qs[r];
+        x = make_float4(fmaf(k, u.x, g * x.x), fmaf(k, u.y, g * x.y), fmaf(k, u.z, g * x.z), fmaf(k, u.w, g * x.w));
+        *reinterpret_cast<float4*>(st + (int64_t)r * vdim + c) = x;
+        o.x = fmaf(x.x, q, o.x), o.y = fmaf(x.y, q, o.y), o.z = fmaf(x.z, q, o.z), o.w = fmaf(x.w, q, o.w);
+      }
+    }
+    o = meet(o);
+    o = make_float4(o.x * rq, o.y * rq, o.z * rq, o.w * rq);
+    if (ok) {
+      sq = fmaf(o.x, o.x, fmaf(o.y, o.y, fmaf(o.z, o.z, fmaf(o.w, o.w, sq))));
+      if (warp == 0) *reinterpret_cast<float4*>(os + c) = o;
+    }
+  }
+  const float inv = 1.0f / sqrtf(warp_sum(sq) / (float)vdim + p.eps);  // (every warp holds all columns)
+  __syncthreads();
+  for (int c = threadIdx.x; c < vdim; c += kTokenThreads)
+    static_cast<T*>(p.y)[b * p.ld_y + h * vdim + c] = from_float<T>(os[c] * inv * p.norm_w[c] * to_float(src[p.off_g + h * vdim + c]));
+}
+
+int token_smem(const b200_delta_args& p) { return (int)(p.dim * p.vdim + kTokenWarps * 128) * 4; }
+bool takes_token(const b200_delta_args& p) {
+  return p.n == 1 && !p.fresh && p.conv_state && p.dim <= kTokenMaxDim && p.vdim <= kStepMaxCols && p.vdim % 4 == 0 && token_smem(p) <= 200 * 1024 &&
+         (reinterpret_cast<uintptr_t>(p.state) & 15) == 0 && p.start < 0x7fffffffLL;
+}
+
+template <typename T>
+int launch_token(const b200_delta_args& p, cudaStream_t stream) {
+  static std::atomic<bool> done[kMaxDevices];
+  const int slot = device_slot();
+  if (slot < 0) return B200_ERR_CUDA;
+  if (!done[slot].load(std::memory_order_acquire)) {
+    if (cudaFuncSetAttribute(delta_token_kernel<T>, cudaFuncAttributeMaxDynamicSharedMemorySize, 200 * 1024) != cudaSuccess) return B200_ERR_CUDA;
+    done[slot].store(true, std::memory_order_release);
+  }
+  delta_token_kernel<T><<<(unsigned)(p.B * p.heads), kTokenThreads, token_smem(p), stream>>>(p);
+  note_launches(1);
+  return status_from_cuda(cudaGetLastError());
+}
+
 bool takes_step(const b200_delta_args& p) {
   return p.dim <= 128 && p.vdim <= kStepMaxCols;
 }
@@ -267,6 +392,8 @@ int launch_typed(const b200_delta_args& p, cudaStream_t stream) {
   int st = B200_OK;
   if (delta_chunk_takes(p)) {
     st = launch_delta_chunk(p, stream);
+  } else if (takes_token(p)) {
+    return launch_token<T>(p, stream);
   } else if (takes_step(p)) {
     st = launch_step<T>(p, stream);
     if (p.n == 1) return st;

@@ -26,7 +26,7 @@ using namespace warp_mma;
 constexpr int kC = 64;  // tokens per chunk
 
 // ------------------------------------------------------------------ convolution and silu
-constexpr int kConvTokens = 16, kConvBatch = 4;  // tokens per thread, loads in flight
+constexpr int kConvTokens = 16, kConvBatch = 8;  // tokens per thread, loads in flight
 // One thread: 8 channels of kConvTokens tokens of one sequence; the last TAPS - 1 inputs stay in registers.
 template <int TAPS>
 __global__ void __launch_bounds__(128)
@@ -39,9 +39,10 @@ delta_conv_kernel(b200_delta_args p, int vecs) {
   const auto* ring = static_cast<const __nv_bfloat16*>(p.conv_state) + b * p.taps * p.conv_cols + c;
   float w[TAPS][8], x[TAPS][8];
 #pragma unroll
-  for (int e = 0; e < 8; ++e)
-#pragma unroll
-    for (int k = 0; k < TAPS; ++k) w[k][e] = __ldg(p.conv_w + (c + e) * TAPS + k);
+  for (int i = 0; i < 8 * TAPS; i += 4) {  // (8 * TAPS consecutive floats from a multiple of 32 bytes on)
+    const float4 f = __ldg(reinterpret_cast<const float4*>(p.conv_w + c * TAPS + i));
+    w[i % TAPS][i / TAPS] = f.x, w[(i + 1) % TAPS][(i + 1) / TAPS] = f.y, w[(i + 2) % TAPS][(i + 2) / TAPS] = f.z, w[(i + 3) % TAPS][(i + 3) / TAPS] = f.w;
+  }
 #pragma unroll
   for (int k = 0; k < TAPS - 1; ++k) {
     const int64_t t = t0 - (TAPS - 1) + k, pos = p.start + t;
@@ -99,7 +100,8 @@ struct PrepareSmem {
   static constexpr int PITCH = DIM * 2 + 16;  // bytes per row of a token tile: ldmatrix rows fall into different banks
   static constexpr int TILE = kC * PITCH;
   static constexpr int A_PITCH = kC + 4;      // floats
-  static constexpr int BYTES = 2 * TILE + 2 * kC * A_PITCH * 4;
+  static constexpr int SQUARE = kC * A_PITCH * 4;  // A and its inverse take the tiles' place
+  static constexpr int BYTES = 2 * (TILE > SQUARE ? TILE : SQUARE);
 };
 
 __device__ __forceinline__ float ex2_ratio(float x) {
@@ -132,8 +134,8 @@ delta_chunk_prepare(b200_delta_args p, int n_chunks) {
   const int n = (int)(p.n - t0 < kC ? p.n - t0 : kC);
   uint8_t* record = static_cast<uint8_t*>(p.workspace) + (int64_t)blockIdx.x * kRecordBytes;
   const uint32_t base = (uint32_t)__cvta_generic_to_shared(smem), sq = base, sk = base + M::TILE;
-  float* A = reinterpret_cast<float*>(smem + 2 * M::TILE);  // [64][68]: A, then T below the diagonal blocks
-  float* X = A + kC * M::A_PITCH;                           // T
+  float* A = reinterpret_cast<float*>(smem);  // [64][68]
+  float* X = A + kC * M::A_PITCH;             // its inverse
   const auto* mixed = static_cast<const __nv_bfloat16*>(p.mixed) + row0 * p.ld_mixed + kv * p.dim;
   load_tile<DIM>(sq, mixed, p.ld_mixed, n, (int)p.dim, 128);
   load_tile<DIM>(sk, mixed + p.off_k, p.ld_mixed, n, (int)p.dim, 128);
@@ -205,6 +207,7 @@ delta_chunk_prepare(b200_delta_args p, int n_chunks) {
       }
     }
   }
+  __syncthreads();  // the tiles are done with
   const int i0 = warp * 16 + g8;
 #pragma unroll
   for (int r = 0; r < 2; ++r) {
@@ -336,7 +339,8 @@ delta_chunk_scan(b200_delta_args p, int n_chunks, int vblocks) {
   constexpr int MT = DIM / 64, NT = CW / 8;  // 16-row state tiles per warp, 8-column tiles per warp
   extern __shared__ __align__(128) uint8_t smem[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g8 = lane >> 2, t4 = lane & 3;
-  const int rg = warp & 3, cg = warp >> 2;  // row group, column group
+  // row group, column group; odd column groups in reverse, so that a scheduler's warps share the triangles' work evenly
+  const int cg = warp >> 2, rg = cg & 1 ? 3 - (warp & 3) : warp & 3;
   const int vb = blockIdx.x % vblocks;
   const int64_t h = (blockIdx.x / vblocks) % p.heads, b = blockIdx.x / ((int64_t)vblocks * p.heads);
   const int64_t kv = h / (p.heads / p.kv_heads);
@@ -566,40 +570,61 @@ delta_chunk_scan(b200_delta_args p, int n_chunks, int vblocks) {
 }
 
 // ------------------------------------------------------------------ norm per head, gate
-// One warp per (row, head), in place on y.
+// In place on y.  `lanes` (a power of two) lanes of 8 columns side by side take a (row, head); heads beyond 256 columns: NV = 2.
+constexpr int kFinishItems = 4;  // per lane group, all loads in flight
+template <int NV>
 __global__ void __launch_bounds__(256)
-delta_finish_kernel(b200_delta_args p, int64_t items) {
-  constexpr int NV = 2;  // vectors of 8 per lane: heads of up to 512 columns
-  const int lane = threadIdx.x & 31;
-  const int64_t item = (int64_t)blockIdx.x * 8 + (threadIdx.x >> 5);
-  if (item >= items) return;
-  const int64_t row = item / p.heads, h = item % p.heads;
-  const int vdim = (int)p.vdim;
-  auto* y = static_cast<__nv_bfloat16*>(p.y) + row * p.ld_y + h * vdim;
-  const auto* gate = static_cast<const __nv_bfloat16*>(p.rows) + row * p.ld + p.off_g + h * vdim;
-  float f[NV][8], g[NV][8], sq = 0.f;
+delta_finish_kernel(b200_delta_args p, int64_t items, int lanes) {
+  const int lane = threadIdx.x & 31, per_warp = 32 / lanes;
+  const int64_t first = ((int64_t)blockIdx.x * 8 + (threadIdx.x >> 5)) * per_warp * kFinishItems + lane / lanes;
+  const int c = (lane % lanes) * 8, vdim = (int)p.vdim, heads = (int)p.heads;
+  uint4 y[kFinishItems][NV], g[kFinishItems][NV];
+  int64_t at[kFinishItems];
 #pragma unroll
-  for (int i = 0; i < NV; ++i) {
-    const int c = (i * 32 + lane) * 8;
-    if (c < vdim) {
-      load8(y + c, f[i]);
-      load8(gate + c, g[i]);
+  for (int i = 0; i < kFinishItems; ++i) {
+    const int64_t item = first + i * per_warp, row = item / heads;
+    const int h = (int)(item - row * heads);
+    at[i] = item < items ? row * p.ld_y + h * vdim + c : -1;
 #pragma unroll
-      for (int e = 0; e < 8; ++e) sq = fmaf(f[i][e], f[i][e], sq);
+    for (int n = 0; n < NV; ++n) {
+      const bool ok = item < items && c + n * 256 < vdim;
+      y[i][n] = ok ? *reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(p.y) + at[i] + n * 256) : make_uint4(0, 0, 0, 0);
+      g[i][n] = ok ? __ldg(reinterpret_cast<const uint4*>(static_cast<const __nv_bfloat16*>(p.rows) + row * p.ld + p.off_g + h * vdim + c + n * 256)) : make_uint4(0, 0, 0, 0);
     }
   }
-  const float inv = 1.0f / sqrtf(warp_sum(sq) / (float)vdim + p.eps);
 #pragma unroll
-  for (int i = 0; i < NV; ++i) {
-    const int c = (i * 32 + lane) * 8;
-    if (c < vdim) {
-      float w[8];
-      load8(p.norm_w + c, w);
+  for (int i = 0; i < kFinishItems; ++i) {
+    float f[NV][8], sq = 0.f;
 #pragma unroll
-      for (int e = 0; e < 8; ++e) w[e] *= f[i][e] * inv * g[i][e];
-      store8(y + c, w);
+    for (int n = 0; n < NV; ++n) {
+      load8(reinterpret_cast<const __nv_bfloat16*>(&y[i][n]), f[n]);
+#pragma unroll
+      for (int e = 0; e < 8; ++e) sq = fmaf(f[n][e], f[n][e], sq);
+    }
+    for (int o = 1; o < lanes; o <<= 1) sq += __shfl_xor_sync(0xffffffffu, sq, o);
+    const float inv = 1.0f / sqrtf(sq / (float)vdim + p.eps);
+#pragma unroll
+    for (int n = 0; n < NV; ++n) {
+      if (at[i] >= 0 && c + n * 256 < vdim) {
+        float w[8], gate[8];
+        load8(p.norm_w + c + n * 256, w);
+        load8(reinterpret_cast<const __nv_bfloat16*>(&g[i][n]), gate);
+#pragma unroll
+        for (int e = 0; e < 8; ++e) w[e] *= f[n][e] * inv * gate[e];
+        store8(static_cast<__nv_bfloat16*>(p.y) + at[i] + n * 256, w);
+      }
     }
   }
+}
+int launch_finish(const b200_delta_args& p, cudaStream_t stream) {
+  int lanes = 1;
+  while (lanes < 32 && lanes * 8 < p.vdim) lanes *= 2;
+  const int64_t items = p.B * p.n * p.heads, per_block = 8LL * (32 / lanes) * kFinishItems;
+  const unsigned grid = (unsigned)((items + per_block - 1) / per_block);
+  if (p.vdim <= 256) delta_finish_kernel<1><<<grid, 256, 0, stream>>>(p, items, lanes);
+  else delta_finish_kernel<2><<<grid, 256, 0, stream>>>(p, items, lanes);
+  note_launches(1);
+  return status_from_cuda(cudaGetLastError());
 }
 
 template <typename K>
@@ -649,10 +674,7 @@ int launch_sized(const b200_delta_args& p, cudaStream_t stream) {
   else if (heads * ((p.vdim + 31) / 32) >= sm_count()) st = launch_scan<DIM, 32, 16>(p, n_chunks, stream);
   else st = launch_scan<DIM, 16, 16>(p, n_chunks, stream);
   if (st != B200_OK) return st;
-  const int64_t items = p.B * p.n * p.heads;
-  delta_finish_kernel<<<(unsigned)((items + 7) / 8), 256, 0, stream>>>(p, items);
-  note_launches(1);
-  return status_from_cuda(cudaGetLastError());
+  return launch_finish(p, stream);
 }
 
 }  // namespace
@@ -661,7 +683,7 @@ bool delta_chunk_takes(const b200_delta_args& p) {
   return p.dtype == B200_BF16 && !p.pos_dev && p.n >= kC / 2 && p.dim <= 128 && p.vdim <= 512 && p.dim % 8 == 0 && p.vdim % 8 == 0 && p.taps <= 8 &&
          p.off_k % 8 == 0 && p.off_v % 8 == 0 && p.off_g % 8 == 0 && p.ld % 8 == 0 && p.ld_mixed % 8 == 0 && p.ld_y % 8 == 0 && p.conv_cols % 8 == 0 &&
          ((reinterpret_cast<uintptr_t>(p.rows) | reinterpret_cast<uintptr_t>(p.mixed) | reinterpret_cast<uintptr_t>(p.y) | reinterpret_cast<uintptr_t>(p.norm_w) |
-           reinterpret_cast<uintptr_t>(p.state) | reinterpret_cast<uintptr_t>(p.conv_state)) & 15) == 0 &&
+           reinterpret_cast<uintptr_t>(p.state) | reinterpret_cast<uintptr_t>(p.conv_state) | reinterpret_cast<uintptr_t>(p.conv_w)) & 15) == 0 &&
          p.B <= 65535 && p.n <= 65535LL * kConvTokens && p.B * p.heads * ((p.n + kC - 1) / kC) <= 0x7fffffffLL;
 }
 
