@@ -321,10 +321,11 @@ delta_chunk_prepare(b200_delta_args p, int n_chunks) {
 }
 
 // ------------------------------------------------------------------ chunk after chunk
-// A block owns VC columns of one head's state; warps = 4 row groups x (VC / CW) column groups of CW columns.
+// A block owns VC columns of one head's state.  Half of its warps run the chain from state to state (C_k S -> R -> U -> S), the
+// other half the outputs beside it; each half is 4 row groups x (VC / CW) column groups of CW columns.
 template <int DIM, int VC, int CW>
 struct ScanSmem {
-  static constexpr int WARPS = 4 * (VC / CW), THREADS = 32 * WARPS;
+  static constexpr int ROLE_WARPS = 4 * (VC / CW), THREADS = 64 * ROLE_WARPS;
   static constexpr int KP = DIM * 2 + 16, VP = VC * 2 + 16;  // bytes per row
   static constexpr int TILE = kC * KP, V_TILE = kC * VP;
   static constexpr int STAGE = 2 * TILE + V_TILE + kFactorBytes + 64;
@@ -339,8 +340,9 @@ delta_chunk_scan(b200_delta_args p, int n_chunks, int vblocks) {
   constexpr int MT = DIM / 64, NT = CW / 8;  // 16-row state tiles per warp, 8-column tiles per warp
   extern __shared__ __align__(128) uint8_t smem[];
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g8 = lane >> 2, t4 = lane & 3;
-  // row group, column group; odd column groups in reverse, so that a scheduler's warps share the triangles' work evenly
-  const int cg = warp >> 2, rg = cg & 1 ? 3 - (warp & 3) : warp & 3;
+  const bool chain = warp < M::ROLE_WARPS;
+  // row group, column group; every other four warps in reverse, so that a scheduler's warps share the triangles' work evenly
+  const int cg = (warp % M::ROLE_WARPS) >> 2, rg = ((warp >> 2) & 1) ? 3 - (warp & 3) : warp & 3;
   const int vb = blockIdx.x % vblocks;
   const int64_t h = (blockIdx.x / vblocks) % p.heads, b = blockIdx.x / ((int64_t)vblocks * p.heads);
   const int64_t kv = h / (p.heads / p.kv_heads);
@@ -351,6 +353,7 @@ delta_chunk_scan(b200_delta_args p, int n_chunks, int vblocks) {
   const auto* mixed = static_cast<const __nv_bfloat16*>(p.mixed) + b * p.n * p.ld_mixed;
   const uint8_t* records = static_cast<const uint8_t*>(p.workspace) + (b * n_chunks * p.heads + h) * (int64_t)kRecordBytes;
   const int64_t record_step = p.heads * (int64_t)kRecordBytes;
+  const int i0 = rg * 16 + g8;  // this thread's tokens of a chunk: i0 and i0 + 8
 
   auto load_chunk = [&](int chunk, int stage) {
     const uint32_t dst = base + stage * M::STAGE;
@@ -381,197 +384,201 @@ delta_chunk_scan(b200_delta_args p, int n_chunks, int vblocks) {
   auto b_at = [&](int row, int np) {
     return (uint32_t)((row + (lane & 7) + ((lane >> 3) & 1) * 8) * M::VP + (cg * CW + np * 16 + (lane >> 4) * 8) * 2);
   };
-
-  // this warp's state: rows (rg * MT + mt) * 16 + {g8, g8 + 8}, columns cg * CW + nt * 8 + t4 * 2 + {0, 1} of the block's
-  float st[MT][NT][4];
-  float* state = p.state + (b * p.heads + h) * (int64_t)dim * vdim;
-#pragma unroll
-  for (int mt = 0; mt < MT; ++mt)
-#pragma unroll
-    for (int nt = 0; nt < NT; ++nt)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) {
-        const int r = (rg * MT + mt) * 16 + g8 + (e >> 1) * 8, c = c0 + cg * CW + nt * 8 + t4 * 2 + (e & 1);
-        st[mt][nt][e] = !p.fresh && r < dim && c < vdim ? state[(int64_t)r * vdim + c] : 0.f;
-      }
-
-  load_chunk(0, 0);
-  for (int chunk = 0; chunk < n_chunks; ++chunk) {
-    const int stage = chunk & 1;
-    const int64_t t0 = (int64_t)chunk * kC;
-    const int n = (int)(p.n - t0 < kC ? p.n - t0 : kC);
-    // T and P of this warp's rows: on their way while the state is written
-    const uint4* frag = reinterpret_cast<const uint4*>(records + chunk * record_step) + block_index(rg, 0) * 64 + lane;
-    uint4 th[4], tl[4];
+  // T (which = 0) or P (1) of this warp's rows
+  auto load_triangle = [&](int chunk, int which, uint4 (&hi)[4], uint4 (&lo)[4]) {
+    const uint4* frag = reinterpret_cast<const uint4*>(records + chunk * record_step + which * kFragBytes) + block_index(rg, 0) * 64 + lane;
 #pragma unroll
     for (int kt = 0; kt < 4; ++kt)
-      if (kt <= rg) th[kt] = __ldg(frag + kt * 64), tl[kt] = __ldg(frag + kt * 64 + 32);
-    __syncthreads();  // everyone is done with the chunk before: the other stage, the state parts, U and U'
-    if (chunk + 1 < n_chunks) {
-      load_chunk(chunk + 1, stage ^ 1);
-      cp_async_wait<1>();
-    } else {
-      cp_async_wait<0>();
-    }
-#pragma unroll
-    for (int mt = 0; mt < MT; ++mt)
-#pragma unroll
-      for (int nt = 0; nt < NT; ++nt) {
-        const int r = (rg * MT + mt) * 16 + g8;
-        put(s_hi, s_lo, r, nt, st[mt][nt][0], st[mt][nt][1]);
-        put(s_hi, s_lo, r + 8, nt, st[mt][nt][2], st[mt][nt][3]);
-      }
-    __syncthreads();  // tiles and state parts are in place
-    const uint32_t sk = base + stage * M::STAGE, sq = sk + M::TILE;
-    const uint8_t* sv = smem + stage * M::STAGE + 2 * M::TILE;
-    const float* factor = reinterpret_cast<const float*>(sv + M::V_TILE);
-
-    // C_k S and C_q S for this warp's 16 tokens
-    float r[NT][4], o[NT][4];
+      if (kt <= rg) hi[kt] = __ldg(frag + kt * 64), lo[kt] = __ldg(frag + kt * 64 + 32);
+  };
+  // acc = 64 token rows (this warp's 16) times the state in two parts
+  auto times_state = [&](uint32_t tile, float (&acc)[NT][4]) {
 #pragma unroll
     for (int i = 0; i < NT; ++i)
 #pragma unroll
-      for (int e = 0; e < 4; ++e) r[i][e] = o[i][e] = 0.f;
+      for (int e = 0; e < 4; ++e) acc[i][e] = 0.f;
 #pragma unroll
     for (int ks = 0; ks < DIM / 16; ++ks) {
-      uint32_t kf[4], qf[4];
-      const uint32_t at = (uint32_t)((rg * 16 + (lane & 15)) * M::KP + (ks * 2 + (lane >> 4)) * 16);
-      ldsm4(kf, sk + at);
-      ldsm4(qf, sq + at);
+      uint32_t af[4];
+      ldsm4(af, tile + (uint32_t)((rg * 16 + (lane & 15)) * M::KP + (ks * 2 + (lane >> 4)) * 16));
 #pragma unroll
       for (int np = 0; np < NT / 2; ++np) {
         uint32_t hi[4], lo[4];
         const uint32_t bt = b_at(ks * 16, np);
         ldsm4_trans(hi, s_hi + bt);
         ldsm4_trans(lo, s_lo + bt);
-        mma_bf16(r[2 * np], kf, hi[0], hi[1]);
-        mma_bf16(r[2 * np + 1], kf, hi[2], hi[3]);
-        mma_bf16(o[2 * np], qf, hi[0], hi[1]);
-        mma_bf16(o[2 * np + 1], qf, hi[2], hi[3]);
-        mma_bf16(r[2 * np], kf, lo[0], lo[1]);
-        mma_bf16(r[2 * np + 1], kf, lo[2], lo[3]);
-        mma_bf16(o[2 * np], qf, lo[0], lo[1]);
-        mma_bf16(o[2 * np + 1], qf, lo[2], lo[3]);
+        mma_bf16(acc[2 * np], af, hi[0], hi[1]);
+        mma_bf16(acc[2 * np + 1], af, hi[2], hi[3]);
+        mma_bf16(acc[2 * np], af, lo[0], lo[1]);
+        mma_bf16(acc[2 * np + 1], af, lo[2], lo[3]);
       }
     }
-    const int i0 = rg * 16 + g8;
-    // R = V - diag(G r_k) C_k S
-    {
-      const float g0 = factor[F_GK * kC + i0], g1 = factor[F_GK * kC + i0 + 8];
+  };
+  // acc += lhs (two parts, lower triangular) times a tile in two parts, for this warp's rows
+  auto triangular = [&](const uint4 (&ah)[4], const uint4 (&al)[4], uint32_t hi_tile, uint32_t lo_tile, float (&acc)[NT][4]) {
 #pragma unroll
-      for (int nt = 0; nt < NT; ++nt) {
-        const int c = cg * CW + nt * 8 + t4 * 2;
-        const float2 v0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sv + i0 * M::VP + c * 2));
-        const float2 v1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sv + (i0 + 8) * M::VP + c * 2));
-        put(r_hi, r_lo, i0, nt, fmaf(-g0, r[nt][0], v0.x), fmaf(-g0, r[nt][1], v0.y));
-        put(r_hi, r_lo, i0 + 8, nt, fmaf(-g1, r[nt][2], v1.x), fmaf(-g1, r[nt][3], v1.y));
-      }
-      const float q0 = factor[F_GQ * kC + i0], q1 = factor[F_GQ * kC + i0 + 8];
+    for (int kt = 0; kt < 4; ++kt) {
+      if (kt <= rg) {
+        const uint32_t fh[4] = {ah[kt].x, ah[kt].y, ah[kt].z, ah[kt].w}, fl[4] = {al[kt].x, al[kt].y, al[kt].z, al[kt].w};
 #pragma unroll
-      for (int nt = 0; nt < NT; ++nt) o[nt][0] *= q0, o[nt][1] *= q0, o[nt][2] *= q1, o[nt][3] *= q1;
-    }
-    __syncthreads();  // R is in place
-    // lhs (two parts, lower triangular) times a tile in two parts, for this warp's rows
-    auto triangular = [&](const uint4 (&ah)[4], const uint4 (&al)[4], uint32_t hi_tile, uint32_t lo_tile, float (&acc)[NT][4]) {
-#pragma unroll
-      for (int kt = 0; kt < 4; ++kt) {
-        if (kt <= rg) {
-          const uint32_t fh[4] = {ah[kt].x, ah[kt].y, ah[kt].z, ah[kt].w}, fl[4] = {al[kt].x, al[kt].y, al[kt].z, al[kt].w};
-#pragma unroll
-          for (int np = 0; np < NT / 2; ++np) {
-            uint32_t hi[4], lo[4];
-            const uint32_t bt = b_at(kt * 16, np);
-            ldsm4_trans(hi, hi_tile + bt);
-            ldsm4_trans(lo, lo_tile + bt);
-            mma_bf16(acc[2 * np], fh, hi[0], hi[1]);
-            mma_bf16(acc[2 * np + 1], fh, hi[2], hi[3]);
-            mma_bf16(acc[2 * np], fl, hi[0], hi[1]);
-            mma_bf16(acc[2 * np + 1], fl, hi[2], hi[3]);
-            mma_bf16(acc[2 * np], fh, lo[0], lo[1]);
-            mma_bf16(acc[2 * np + 1], fh, lo[2], lo[3]);
-          }
+        for (int np = 0; np < NT / 2; ++np) {
+          uint32_t hi[4], lo[4];
+          const uint32_t bt = b_at(kt * 16, np);
+          ldsm4_trans(hi, hi_tile + bt);
+          ldsm4_trans(lo, lo_tile + bt);
+          mma_bf16(acc[2 * np], fh, hi[0], hi[1]);
+          mma_bf16(acc[2 * np + 1], fh, hi[2], hi[3]);
+          mma_bf16(acc[2 * np], fl, hi[0], hi[1]);
+          mma_bf16(acc[2 * np + 1], fl, hi[2], hi[3]);
+          mma_bf16(acc[2 * np], fh, lo[0], lo[1]);
+          mma_bf16(acc[2 * np + 1], fh, lo[2], lo[3]);
         }
       }
-    };
-    // U = T R, as it is for the outputs and times (G_64 / G_j) r_kj for the state
-#pragma unroll
-    for (int i = 0; i < NT; ++i)
-#pragma unroll
-      for (int e = 0; e < 4; ++e) r[i][e] = 0.f;
-    triangular(th, tl, r_hi, r_lo, r);
-    // (P's fragments take the registers of T's)
-#pragma unroll
-    for (int kt = 0; kt < 4; ++kt)
-      if (kt <= rg) th[kt] = __ldg(frag + kFragBytes / 16 + kt * 64), tl[kt] = __ldg(frag + kFragBytes / 16 + kt * 64 + 32);
-    {
-      const float f0 = factor[F_WRITE * kC + i0], f1 = factor[F_WRITE * kC + i0 + 8];
-#pragma unroll
-      for (int nt = 0; nt < NT; ++nt) {
-        put(u_hi, u_lo, i0, nt, r[nt][0], r[nt][1]);
-        put(u_hi, u_lo, i0 + 8, nt, r[nt][2], r[nt][3]);
-        put(w_hi, w_lo, i0, nt, r[nt][0] * f0, r[nt][1] * f0);
-        put(w_hi, w_lo, i0 + 8, nt, r[nt][2] * f1, r[nt][3] * f1);
-      }
     }
-    __syncthreads();  // U and U' are in place
-    // S <- G_64 S + C_k^T U'
-    const float decay = factor[4 * kC];
+  };
+
+  load_chunk(0, 0);
+  if (chain) {
+    // this warp's state: rows (rg * MT + mt) * 16 + {g8, g8 + 8}, columns cg * CW + nt * 8 + t4 * 2 + {0, 1} of the block's
+    float st[MT][NT][4];
+    float* state = p.state + (b * p.heads + h) * (int64_t)dim * vdim;
 #pragma unroll
     for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
       for (int nt = 0; nt < NT; ++nt)
 #pragma unroll
-        for (int e = 0; e < 4; ++e) st[mt][nt][e] *= decay;
-#pragma unroll
-    for (int kk = 0; kk < 4; ++kk) {
-      uint32_t kf[MT][4];
+        for (int e = 0; e < 4; ++e) {
+          const int r = (rg * MT + mt) * 16 + g8 + (e >> 1) * 8, c = c0 + cg * CW + nt * 8 + t4 * 2 + (e & 1);
+          st[mt][nt][e] = !p.fresh && r < dim && c < vdim ? state[(int64_t)r * vdim + c] : 0.f;
+        }
+    for (int chunk = 0; chunk < n_chunks; ++chunk) {
+      const int stage = chunk & 1;
+      uint4 th[4], tl[4];
+      load_triangle(chunk, 0, th, tl);
 #pragma unroll
       for (int mt = 0; mt < MT; ++mt)
-        ldsm4_trans(kf[mt], sk + (uint32_t)((kk * 16 + (lane & 7) + ((lane >> 4) << 3)) * M::KP + ((rg * MT + mt) * 16 + ((lane >> 3) & 1) * 8) * 2));
 #pragma unroll
-      for (int np = 0; np < NT / 2; ++np) {
-        uint32_t hi[4], lo[4];
-        const uint32_t bt = b_at(kk * 16, np);
-        ldsm4_trans(hi, w_hi + bt);
-        ldsm4_trans(lo, w_lo + bt);
-#pragma unroll
-        for (int mt = 0; mt < MT; ++mt) {
-          mma_bf16(st[mt][2 * np], kf[mt], hi[0], hi[1]);
-          mma_bf16(st[mt][2 * np + 1], kf[mt], hi[2], hi[3]);
-          mma_bf16(st[mt][2 * np], kf[mt], lo[0], lo[1]);
-          mma_bf16(st[mt][2 * np + 1], kf[mt], lo[2], lo[3]);
+        for (int nt = 0; nt < NT; ++nt) {
+          const int r = (rg * MT + mt) * 16 + g8;
+          put(s_hi, s_lo, r, nt, st[mt][nt][0], st[mt][nt][1]);
+          put(s_hi, s_lo, r + 8, nt, st[mt][nt][2], st[mt][nt][3]);
         }
-      }
-    }
-    // O = diag(G r_q) C_q S + P U
-    triangular(th, tl, u_hi, u_lo, o);
-#pragma unroll
-    for (int e = 0; e < 2; ++e) {
-      const int i = i0 + e * 8;
-      if (i < n) {
-        auto* y = static_cast<__nv_bfloat16*>(p.y) + (b * p.n + t0 + i) * p.ld_y + h * vdim + c0;
+      cp_async_wait<0>();
+      __syncthreads();  // (1) tiles and state parts are in place; everyone is done with the chunk before
+      if (chunk + 1 < n_chunks) load_chunk(chunk + 1, stage ^ 1);
+      const uint32_t sk = base + stage * M::STAGE;
+      const uint8_t* sv = smem + stage * M::STAGE + 2 * M::TILE;
+      const float* factor = reinterpret_cast<const float*>(sv + M::V_TILE);
+      // R = V - diag(G r_k) C_k S
+      float r[NT][4];
+      times_state(sk, r);
+      {
+        const float g0 = factor[F_GK * kC + i0], g1 = factor[F_GK * kC + i0 + 8];
 #pragma unroll
         for (int nt = 0; nt < NT; ++nt) {
           const int c = cg * CW + nt * 8 + t4 * 2;
-          if (c0 + c < vdim) *reinterpret_cast<__nv_bfloat162*>(y + c) = __floats2bfloat162_rn(o[nt][2 * e], o[nt][2 * e + 1]);
+          const float2 v0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sv + i0 * M::VP + c * 2));
+          const float2 v1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sv + (i0 + 8) * M::VP + c * 2));
+          put(r_hi, r_lo, i0, nt, fmaf(-g0, r[nt][0], v0.x), fmaf(-g0, r[nt][1], v0.y));
+          put(r_hi, r_lo, i0 + 8, nt, fmaf(-g1, r[nt][2], v1.x), fmaf(-g1, r[nt][3], v1.y));
+        }
+      }
+      __syncthreads();  // (2) R is in place
+      // U = T R, as it is for the outputs and times (G_64 / G_j) r_kj for the state
+#pragma unroll
+      for (int i = 0; i < NT; ++i)
+#pragma unroll
+        for (int e = 0; e < 4; ++e) r[i][e] = 0.f;
+      triangular(th, tl, r_hi, r_lo, r);
+      {
+        const float f0 = factor[F_WRITE * kC + i0], f1 = factor[F_WRITE * kC + i0 + 8];
+#pragma unroll
+        for (int nt = 0; nt < NT; ++nt) {
+          put(w_hi, w_lo, i0, nt, r[nt][0] * f0, r[nt][1] * f0);
+          put(w_hi, w_lo, i0 + 8, nt, r[nt][2] * f1, r[nt][3] * f1);
+          put(u_hi, u_lo, i0, nt, r[nt][0], r[nt][1]);
+          put(u_hi, u_lo, i0 + 8, nt, r[nt][2], r[nt][3]);
+        }
+      }
+      __syncthreads();  // (3) U and U' are in place
+      // S <- G_64 S + C_k^T U'
+      const float decay = factor[4 * kC];
+#pragma unroll
+      for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+        for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+          for (int e = 0; e < 4; ++e) st[mt][nt][e] *= decay;
+#pragma unroll
+      for (int kk = 0; kk < 4; ++kk) {
+        uint32_t kf[MT][4];
+#pragma unroll
+        for (int mt = 0; mt < MT; ++mt)
+          ldsm4_trans(kf[mt], sk + (uint32_t)((kk * 16 + (lane & 7) + ((lane >> 4) << 3)) * M::KP + ((rg * MT + mt) * 16 + ((lane >> 3) & 1) * 8) * 2));
+#pragma unroll
+        for (int np = 0; np < NT / 2; ++np) {
+          uint32_t hi[4], lo[4];
+          const uint32_t bt = b_at(kk * 16, np);
+          ldsm4_trans(hi, w_hi + bt);
+          ldsm4_trans(lo, w_lo + bt);
+#pragma unroll
+          for (int mt = 0; mt < MT; ++mt) {
+            mma_bf16(st[mt][2 * np], kf[mt], hi[0], hi[1]);
+            mma_bf16(st[mt][2 * np + 1], kf[mt], hi[2], hi[3]);
+            mma_bf16(st[mt][2 * np], kf[mt], lo[0], lo[1]);
+            mma_bf16(st[mt][2 * np + 1], kf[mt], lo[2], lo[3]);
+          }
+        }
+      }
+    }
+#pragma unroll
+    for (int mt = 0; mt < MT; ++mt)
+#pragma unroll
+      for (int nt = 0; nt < NT; ++nt)
+#pragma unroll
+        for (int e = 0; e < 4; e += 2) {
+          const int r = (rg * MT + mt) * 16 + g8 + (e >> 1) * 8, c = c0 + cg * CW + nt * 8 + t4 * 2;
+          if (r < dim && c < vdim) *reinterpret_cast<float2*>(state + (int64_t)r * vdim + c) = make_float2(st[mt][nt][e], st[mt][nt][e + 1]);
+        }
+  } else {
+    for (int chunk = 0; chunk < n_chunks; ++chunk) {
+      const int stage = chunk & 1;
+      const int64_t t0 = (int64_t)chunk * kC;
+      const int n = (int)(p.n - t0 < kC ? p.n - t0 : kC);
+      cp_async_wait<0>();
+      __syncthreads();  // (1)
+      if (chunk + 1 < n_chunks) load_chunk(chunk + 1, stage ^ 1);
+      uint4 ph[4], pl[4];
+      load_triangle(chunk, 1, ph, pl);
+      const float* factor = reinterpret_cast<const float*>(smem + stage * M::STAGE + 2 * M::TILE + M::V_TILE);
+      // O = diag(G r_q) C_q S + P U
+      float o[NT][4];
+      times_state(base + stage * M::STAGE + M::TILE, o);
+      const float q0 = factor[F_GQ * kC + i0], q1 = factor[F_GQ * kC + i0 + 8];
+#pragma unroll
+      for (int nt = 0; nt < NT; ++nt) o[nt][0] *= q0, o[nt][1] *= q0, o[nt][2] *= q1, o[nt][3] *= q1;
+      __syncthreads();  // (2)
+      __syncthreads();  // (3)
+      triangular(ph, pl, u_hi, u_lo, o);
+#pragma unroll
+      for (int e = 0; e < 2; ++e) {
+        const int i = i0 + e * 8;
+        if (i < n) {
+          auto* y = static_cast<__nv_bfloat16*>(p.y) + (b * p.n + t0 + i) * p.ld_y + h * vdim + c0;
+#pragma unroll
+          for (int nt = 0; nt < NT; ++nt) {
+            const int c = cg * CW + nt * 8 + t4 * 2;
+            if (c0 + c < vdim) *reinterpret_cast<__nv_bfloat162*>(y + c) = __floats2bfloat162_rn(o[nt][2 * e], o[nt][2 * e + 1]);
+          }
         }
       }
     }
   }
-#pragma unroll
-  for (int mt = 0; mt < MT; ++mt)
-#pragma unroll
-    for (int nt = 0; nt < NT; ++nt)
-#pragma unroll
-      for (int e = 0; e < 4; e += 2) {
-        const int r = (rg * MT + mt) * 16 + g8 + (e >> 1) * 8, c = c0 + cg * CW + nt * 8 + t4 * 2;
-        if (r < dim && c < vdim) *reinterpret_cast<float2*>(state + (int64_t)r * vdim + c) = make_float2(st[mt][nt][e], st[mt][nt][e + 1]);
-      }
 }
 
 // ------------------------------------------------------------------ norm per head, gate
 // In place on y.  `lanes` (a power of two) lanes of 8 columns side by side take a (row, head); heads beyond 256 columns: NV = 2.
-constexpr int kFinishItems = 4;  // per lane group, all loads in flight
+constexpr int kFinishItems = 2;  // per lane group, all loads in flight
 template <int NV>
 __global__ void __launch_bounds__(256)
 delta_finish_kernel(b200_delta_args p, int64_t items, int lanes) {
@@ -582,8 +589,10 @@ delta_finish_kernel(b200_delta_args p, int64_t items, int lanes) {
   int64_t at[kFinishItems];
 #pragma unroll
   for (int i = 0; i < kFinishItems; ++i) {
-    const int64_t item = first + i * per_warp, row = item / heads;
-    const int h = (int)(item - row * heads);
+    const int64_t item = first + i * per_warp;
+    const uint32_t r32 = (uint32_t)item / (uint32_t)heads;  // (the host keeps the items below 2^31)
+    const int64_t row = r32;
+    const int h = (int)((uint32_t)item - r32 * (uint32_t)heads);
     at[i] = item < items ? row * p.ld_y + h * vdim + c : -1;
 #pragma unroll
     for (int n = 0; n < NV; ++n) {
@@ -684,7 +693,7 @@ bool delta_chunk_takes(const b200_delta_args& p) {
          p.off_k % 8 == 0 && p.off_v % 8 == 0 && p.off_g % 8 == 0 && p.ld % 8 == 0 && p.ld_mixed % 8 == 0 && p.ld_y % 8 == 0 && p.conv_cols % 8 == 0 &&
          ((reinterpret_cast<uintptr_t>(p.rows) | reinterpret_cast<uintptr_t>(p.mixed) | reinterpret_cast<uintptr_t>(p.y) | reinterpret_cast<uintptr_t>(p.norm_w) |
            reinterpret_cast<uintptr_t>(p.state) | reinterpret_cast<uintptr_t>(p.conv_state) | reinterpret_cast<uintptr_t>(p.conv_w)) & 15) == 0 &&
-         p.B <= 65535 && p.n <= 65535LL * kConvTokens && p.B * p.heads * ((p.n + kC - 1) / kC) <= 0x7fffffffLL;
+         p.B <= 65535 && p.n <= 65535LL * kConvTokens && p.B * p.heads * p.n <= 0x7fffffffLL - 4096;
 }
 
 int64_t delta_chunk_workspace_bytes(const b200_delta_args& p) { return p.B * p.heads * ((p.n + kC - 1) / kC) * kRecordBytes; }
