@@ -112,9 +112,9 @@ __device__ __forceinline__ float ex2_ratio(float x) {
 
 // Rows of 16-byte pieces of one head's columns, zero beyond the last token and column.
 template <int DIM>
-__device__ __forceinline__ void load_tile(uint32_t dst, const __nv_bfloat16* src, int64_t ld, int n, int cols, int threads) {
+__device__ __forceinline__ void load_tile(uint32_t dst, const __nv_bfloat16* src, int64_t ld, int n, int cols, int thread, int threads) {
   constexpr int PITCH = DIM * 2 + 16;
-  for (int i = threadIdx.x; i < kC * (DIM / 8); i += threads) {
+  for (int i = thread; i < kC * (DIM / 8); i += threads) {
     const int r = i / (DIM / 8), c = i % (DIM / 8);
     const bool ok = r < n && c * 8 < cols;
     cp_async16(dst + r * PITCH + c * 16, ok ? src + (int64_t)r * ld + c * 8 : src, ok);
@@ -137,8 +137,8 @@ delta_chunk_prepare(b200_delta_args p, int n_chunks) {
   float* A = reinterpret_cast<float*>(smem);  // [64][68]
   float* X = A + kC * M::A_PITCH;             // its inverse
   const auto* mixed = static_cast<const __nv_bfloat16*>(p.mixed) + row0 * p.ld_mixed + kv * p.dim;
-  load_tile<DIM>(sq, mixed, p.ld_mixed, n, (int)p.dim, 128);
-  load_tile<DIM>(sk, mixed + p.off_k, p.ld_mixed, n, (int)p.dim, 128);
+  load_tile<DIM>(sq, mixed, p.ld_mixed, n, (int)p.dim, threadIdx.x, 128);
+  load_tile<DIM>(sk, mixed + p.off_k, p.ld_mixed, n, (int)p.dim, threadIdx.x, 128);
   cp_async_commit();
   // log2 decays, their running sum in two fp32 parts (differences stay exact however long and strong the decays), step sizes
   if (threadIdx.x < kC) {
@@ -355,21 +355,23 @@ delta_chunk_scan(b200_delta_args p, int n_chunks, int vblocks) {
   const int64_t record_step = p.heads * (int64_t)kRecordBytes;
   const int i0 = rg * 16 + g8;  // this thread's tokens of a chunk: i0 and i0 + 8
 
+  // (by the output warps only: the chain has no cycles to spare)
+  const int loader = (int)threadIdx.x - 32 * M::ROLE_WARPS;
   auto load_chunk = [&](int chunk, int stage) {
     const uint32_t dst = base + stage * M::STAGE;
     const int64_t t0 = (int64_t)chunk * kC;
     const int n = (int)(p.n - t0 < kC ? p.n - t0 : kC);
     const auto* src = mixed + t0 * p.ld_mixed;
-    load_tile<DIM>(dst, src + p.off_k + kv * dim, p.ld_mixed, n, dim, M::THREADS);
-    load_tile<DIM>(dst + M::TILE, src + kv * dim, p.ld_mixed, n, dim, M::THREADS);
-    for (int i = threadIdx.x; i < kC * (VC / 8); i += M::THREADS) {
+    load_tile<DIM>(dst, src + p.off_k + kv * dim, p.ld_mixed, n, dim, loader, 32 * M::ROLE_WARPS);
+    load_tile<DIM>(dst + M::TILE, src + kv * dim, p.ld_mixed, n, dim, loader, 32 * M::ROLE_WARPS);
+    for (int i = loader; i < kC * (VC / 8); i += 32 * M::ROLE_WARPS) {
       const int r = i / (VC / 8), c = i % (VC / 8);
       const bool ok = r < n && c0 + c * 8 < vdim;
       const auto* v = src + p.off_v + h * vdim + c0;
       cp_async16(dst + 2 * M::TILE + r * M::VP + c * 16, ok ? v + (int64_t)r * p.ld_mixed + c * 8 : mixed, ok);
     }
     const uint8_t* f = records + chunk * record_step + 2 * kFragBytes;
-    for (int i = threadIdx.x; i < (kFactorBytes + 64) / 16; i += M::THREADS) cp_async16(dst + 2 * M::TILE + M::V_TILE + i * 16, f + i * 16, true);
+    for (int i = loader; i < (kFactorBytes + 64) / 16; i += 32 * M::ROLE_WARPS) cp_async16(dst + 2 * M::TILE + M::V_TILE + i * 16, f + i * 16, true);
     cp_async_commit();
   };
   // accumulators (rows of 16, this warp's columns) as two bf16 parts into a row-major tile
@@ -437,7 +439,6 @@ delta_chunk_scan(b200_delta_args p, int n_chunks, int vblocks) {
     }
   };
 
-  load_chunk(0, 0);
   if (chain) {
     // this warp's state: rows (rg * MT + mt) * 16 + {g8, g8 + 8}, columns cg * CW + nt * 8 + t4 * 2 + {0, 1} of the block's
     float st[MT][NT][4];
@@ -451,10 +452,10 @@ delta_chunk_scan(b200_delta_args p, int n_chunks, int vblocks) {
           const int r = (rg * MT + mt) * 16 + g8 + (e >> 1) * 8, c = c0 + cg * CW + nt * 8 + t4 * 2 + (e & 1);
           st[mt][nt][e] = !p.fresh && r < dim && c < vdim ? state[(int64_t)r * vdim + c] : 0.f;
         }
+    uint4 th[4], tl[4];
+    load_triangle(0, 0, th, tl);
     for (int chunk = 0; chunk < n_chunks; ++chunk) {
       const int stage = chunk & 1;
-      uint4 th[4], tl[4];
-      load_triangle(chunk, 0, th, tl);
 #pragma unroll
       for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
@@ -463,9 +464,7 @@ delta_chunk_scan(b200_delta_args p, int n_chunks, int vblocks) {
           put(s_hi, s_lo, r, nt, st[mt][nt][0], st[mt][nt][1]);
           put(s_hi, s_lo, r + 8, nt, st[mt][nt][2], st[mt][nt][3]);
         }
-      cp_async_wait<0>();
       __syncthreads();  // (1) tiles and state parts are in place; everyone is done with the chunk before
-      if (chunk + 1 < n_chunks) load_chunk(chunk + 1, stage ^ 1);
       const uint32_t sk = base + stage * M::STAGE;
       const uint8_t* sv = smem + stage * M::STAGE + 2 * M::TILE;
       const float* factor = reinterpret_cast<const float*>(sv + M::V_TILE);
@@ -490,6 +489,7 @@ delta_chunk_scan(b200_delta_args p, int n_chunks, int vblocks) {
 #pragma unroll
         for (int e = 0; e < 4; ++e) r[i][e] = 0.f;
       triangular(th, tl, r_hi, r_lo, r);
+      if (chunk + 1 < n_chunks) load_triangle(chunk + 1, 0, th, tl);
       {
         const float f0 = factor[F_WRITE * kC + i0], f1 = factor[F_WRITE * kC + i0 + 8];
 #pragma unroll
@@ -541,6 +541,7 @@ delta_chunk_scan(b200_delta_args p, int n_chunks, int vblocks) {
           if (r < dim && c < vdim) *reinterpret_cast<float2*>(state + (int64_t)r * vdim + c) = make_float2(st[mt][nt][e], st[mt][nt][e + 1]);
         }
   } else {
+    load_chunk(0, 0);
     for (int chunk = 0; chunk < n_chunks; ++chunk) {
       const int stage = chunk & 1;
       const int64_t t0 = (int64_t)chunk * kC;
