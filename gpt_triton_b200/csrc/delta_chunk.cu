@@ -27,6 +27,13 @@ constexpr int kC = 64;  // tokens per chunk
 
 // ------------------------------------------------------------------ convolution and silu
 constexpr int kConvTokens = 16, kConvBatch = 8;  // tokens per thread, loads in flight
+// a / (1 + exp(-a)) with one ex2 and one reciprocal
+__device__ __forceinline__ float silu_quick(float a) {
+  float e, r;
+  asm("ex2.approx.ftz.f32 %0, %1;" : "=f"(e) : "f"(a * -1.4426950408889634f));
+  asm("rcp.approx.ftz.f32 %0, %1;" : "=f"(r) : "f"(1.0f + e));
+  return a * r;
+}
 // One thread: 8 channels of kConvTokens tokens of one sequence; the last TAPS - 1 inputs stay in registers.
 template <int TAPS>
 __global__ void __launch_bounds__(128)
@@ -37,44 +44,53 @@ delta_conv_kernel(b200_delta_args p, int vecs) {
   const auto* rows = static_cast<const __nv_bfloat16*>(p.rows) + b * p.n * p.ld + c;
   auto* out = static_cast<__nv_bfloat16*>(p.mixed) + b * p.n * p.ld_mixed + c;
   const auto* ring = static_cast<const __nv_bfloat16*>(p.conv_state) + b * p.taps * p.conv_cols + c;
-  float w[TAPS][8], x[TAPS][8];
+  float2 w[TAPS][4], x[TAPS][4];  // pairs of channels: packed multiply-adds
+  {
+    float f[8 * TAPS];  // (8 * TAPS consecutive floats from a multiple of 32 bytes on)
 #pragma unroll
-  for (int i = 0; i < 8 * TAPS; i += 4) {  // (8 * TAPS consecutive floats from a multiple of 32 bytes on)
-    const float4 f = __ldg(reinterpret_cast<const float4*>(p.conv_w + c * TAPS + i));
-    w[i % TAPS][i / TAPS] = f.x, w[(i + 1) % TAPS][(i + 1) / TAPS] = f.y, w[(i + 2) % TAPS][(i + 2) / TAPS] = f.z, w[(i + 3) % TAPS][(i + 3) / TAPS] = f.w;
+    for (int i = 0; i < 8 * TAPS; i += 4) {
+      const float4 v4 = __ldg(reinterpret_cast<const float4*>(p.conv_w + c * TAPS + i));
+      f[i] = v4.x, f[i + 1] = v4.y, f[i + 2] = v4.z, f[i + 3] = v4.w;
+    }
+#pragma unroll
+    for (int k = 0; k < TAPS; ++k)
+#pragma unroll
+      for (int e = 0; e < 4; ++e) w[k][e] = make_float2(f[2 * e * TAPS + k], f[(2 * e + 1) * TAPS + k]);
   }
+  auto unpack = [](const uint4& u, float2 (&f)[4]) {
+    const __nv_bfloat162* h = reinterpret_cast<const __nv_bfloat162*>(&u);
+#pragma unroll
+    for (int e = 0; e < 4; ++e) f[e] = __bfloat1622float2(h[e]);
+  };
+  auto load = [&](const __nv_bfloat16* src, bool ok) { return ok ? __ldg(reinterpret_cast<const uint4*>(src)) : make_uint4(0, 0, 0, 0); };
 #pragma unroll
   for (int k = 0; k < TAPS - 1; ++k) {
     const int64_t t = t0 - (TAPS - 1) + k, pos = p.start + t;
-#pragma unroll
-    for (int e = 0; e < 8; ++e) x[k][e] = 0.f;
-    if (t >= 0) load8(rows + t * p.ld, x[k]);
-    else if (pos >= 0) load8(ring + pos % TAPS * p.conv_cols, x[k]);
+    unpack(t >= 0 ? load(rows + t * p.ld, true) : load(ring + (pos + TAPS) % TAPS * p.conv_cols, pos >= 0), x[k]);
   }
   for (int i0 = 0; i0 < kConvTokens; i0 += kConvBatch) {
     uint4 raw[kConvBatch];
 #pragma unroll
-    for (int i = 0; i < kConvBatch; ++i) {
-      const int64_t t = t0 + i0 + i;
-      raw[i] = t < p.n ? __ldg(reinterpret_cast<const uint4*>(rows + t * p.ld)) : make_uint4(0, 0, 0, 0);
-    }
+    for (int i = 0; i < kConvBatch; ++i) raw[i] = load(rows + (t0 + i0 + i) * p.ld, t0 + i0 + i < p.n);
 #pragma unroll
     for (int i = 0; i < kConvBatch; ++i) {
       const int64_t t = t0 + i0 + i;
-      load8(reinterpret_cast<const __nv_bfloat16*>(&raw[i]), x[TAPS - 1]);
-      float o[8];
+      unpack(raw[i], x[TAPS - 1]);
+      uint4 res;
+      uint32_t* o = reinterpret_cast<uint32_t*>(&res);
 #pragma unroll
-      for (int e = 0; e < 8; ++e) {
-        float a = 0.f;
+      for (int e = 0; e < 4; ++e) {
+        float2 a = __fmul2_rn(w[0][e], x[0][e]);
 #pragma unroll
-        for (int k = 0; k < TAPS; ++k) a = fmaf(w[k][e], x[k][e], a);
-        o[e] = __fdividef(a, 1.0f + __expf(-a));
+        for (int k = 1; k < TAPS; ++k) a = __ffma2_rn(w[k][e], x[k][e], a);
+        const __nv_bfloat162 h = __floats2bfloat162_rn(silu_quick(a.x), silu_quick(a.y));
+        o[e] = *reinterpret_cast<const uint32_t*>(&h);
       }
-      if (t < p.n) store8(out + t * p.ld_mixed, o);
+      if (t < p.n) *reinterpret_cast<uint4*>(out + t * p.ld_mixed) = res;
 #pragma unroll
       for (int k = 0; k + 1 < TAPS; ++k)
 #pragma unroll
-        for (int e = 0; e < 8; ++e) x[k][e] = x[k + 1][e];
+        for (int e = 0; e < 4; ++e) x[k][e] = x[k + 1][e];
     }
   }
 }
@@ -250,11 +266,13 @@ delta_chunk_prepare(b200_delta_args p, int n_chunks) {
     for (int i = 0; i < 32; ++i) {
       float s0 = i == lane ? 1.f : 0.f, s1 = 0.f;
 #pragma unroll
-      for (int j = 0; j + 1 < i; j += 2) {
-        s0 = fmaf(-L[i * M::A_PITCH + j], x[j], s0);
-        s1 = fmaf(-L[i * M::A_PITCH + j + 1], x[j + 1], s1);
+      for (int j = 0; j < i; j += 4) {
+        const float4 l = *reinterpret_cast<const float4*>(L + i * M::A_PITCH + j);
+        s0 = fmaf(-l.x, x[j], s0);
+        if (j + 1 < i) s1 = fmaf(-l.y, x[j + 1], s1);
+        if (j + 2 < i) s0 = fmaf(-l.z, x[j + 2], s0);
+        if (j + 3 < i) s1 = fmaf(-l.w, x[j + 3], s1);
       }
-      if (i & 1) s0 = fmaf(-L[i * M::A_PITCH + i - 1], x[i - 1], s0);
       x[i] = s0 + s1;
       X[(warp * 32 + i) * M::A_PITCH + warp * 32 + lane] = x[i];
     }
@@ -266,12 +284,16 @@ delta_chunk_prepare(b200_delta_args p, int n_chunks) {
     auto product = [&](const float* lhs, const float* rhs, float (&acc)[2][4]) {
 #pragma unroll
       for (int e = 0; e < 4; ++e) acc[0][e] = acc[1][e] = 0.f;
-#pragma unroll 8
-      for (int k = 0; k < 32; ++k) {
-        const float4 v = *reinterpret_cast<const float4*>(rhs + k * M::A_PITCH + c);
-        const float a0 = lhs[r * M::A_PITCH + k], a1 = lhs[(r + 1) * M::A_PITCH + k];
-        acc[0][0] = fmaf(a0, v.x, acc[0][0]), acc[0][1] = fmaf(a0, v.y, acc[0][1]), acc[0][2] = fmaf(a0, v.z, acc[0][2]), acc[0][3] = fmaf(a0, v.w, acc[0][3]);
-        acc[1][0] = fmaf(a1, v.x, acc[1][0]), acc[1][1] = fmaf(a1, v.y, acc[1][1]), acc[1][2] = fmaf(a1, v.z, acc[1][2]), acc[1][3] = fmaf(a1, v.w, acc[1][3]);
+#pragma unroll 2
+      for (int k = 0; k < 32; k += 4) {
+        const float4 a0 = *reinterpret_cast<const float4*>(lhs + r * M::A_PITCH + k), a1 = *reinterpret_cast<const float4*>(lhs + (r + 1) * M::A_PITCH + k);
+        const float l0[4] = {a0.x, a0.y, a0.z, a0.w}, l1[4] = {a1.x, a1.y, a1.z, a1.w};
+#pragma unroll
+        for (int i = 0; i < 4; ++i) {
+          const float4 v = *reinterpret_cast<const float4*>(rhs + (k + i) * M::A_PITCH + c);
+          acc[0][0] = fmaf(l0[i], v.x, acc[0][0]), acc[0][1] = fmaf(l0[i], v.y, acc[0][1]), acc[0][2] = fmaf(l0[i], v.z, acc[0][2]), acc[0][3] = fmaf(l0[i], v.w, acc[0][3]);
+          acc[1][0] = fmaf(l1[i], v.x, acc[1][0]), acc[1][1] = fmaf(l1[i], v.y, acc[1][1]), acc[1][2] = fmaf(l1[i], v.z, acc[1][2]), acc[1][3] = fmaf(l1[i], v.w, acc[1][3]);
+        }
       }
     };
     float acc[2][4];
