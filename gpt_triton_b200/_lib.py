@@ -61,7 +61,7 @@ class PairAttentionArgs(ctypes.Structure):
 class DeltaArgs(ctypes.Structure):
     _fields_ = _fields("ptr rows; i64 ld off_k off_v off_a off_b off_g; ptr conv_w conv_state; i64 conv_cols taps; ptr mixed; i64 ld_mixed; "
                        "ptr norms gates a_log dt_bias norm_w state y; i64 ld_y; ptr pos_dev; i64 B n start heads kv_heads dim vdim; "
-                       "float eps unit_eps q_scale; int fresh dtype; ptr workspace; i64 workspace_bytes")
+                       "float eps unit_eps q_scale; int fresh dtype; ptr workspace; i64 workspace_bytes; ptr status_word")
 
 
 # name -> (restype, argtypes); must list every function include/b200_gpt.h declares

@@ -17,6 +17,7 @@
 #include <atomic>
 
 #include "mma_sync.cuh"
+#include "sm100_primitives.cuh"
 
 namespace b200 {
 namespace {
@@ -348,19 +349,30 @@ delta_chunk_prepare(b200_delta_args p, int n_chunks) {
 template <int DIM, int VC, int CW>
 struct ScanSmem {
   static constexpr int ROLE_WARPS = 4 * (VC / CW), THREADS = 64 * ROLE_WARPS;
-  static constexpr int KP = DIM * 2 + 16, VP = VC * 2 + 16;  // bytes per row
-  static constexpr int TILE = kC * KP, V_TILE = kC * VP;
-  static constexpr int STAGE = 2 * TILE + V_TILE + kFactorBytes + 64;
-  static constexpr int S_PART = DIM * VP;
-  static constexpr int BYTES = 2 * STAGE + 2 * S_PART + 6 * V_TILE;  // S, R, U, U' in two parts each
+  // a stage: keys, queries (DIM / 64 TMA atoms of 64 rows x 128 bytes each, 128-byte swizzle), 64 columns of values, the record
+  static constexpr int ATOM = kC * 128, TILE = DIM / 64 * ATOM;
+  static constexpr int V_AT = 2 * TILE, RECORD_AT = V_AT + ATOM, FACTOR_AT = RECORD_AT + 2 * kFragBytes;
+  static constexpr int STAGE = (RECORD_AT + kRecordBytes + 1023) / 1024 * 1024, STAGES = VC == 16 ? 3 : 2;
+  static constexpr int TX_BYTES = 2 * TILE + ATOM + kRecordBytes;
+  static constexpr int VP = VC * 2 + 16;  // bytes per row of the tiles below: ldmatrix rows fall into different banks
+  static constexpr int V_TILE = kC * VP, S_PART = DIM * VP;
+  static constexpr int BYTES = STAGES * STAGE + 2 * S_PART + 6 * V_TILE + 1024;  // S, R, U, U' in two parts each; alignment
 };
+
+// size a multiple of 16 bytes, both addresses 16-byte aligned
+__device__ __forceinline__ void bulk_copy(uint32_t dst, const void* src, uint32_t bytes, uint32_t bar) {
+  asm volatile("cp.async.bulk.shared::cluster.global.mbarrier::complete_tx::bytes [%0], [%1], %2, [%3];" ::"r"(dst), "l"(src), "r"(bytes), "r"(bar) : "memory");
+}
 
 template <int DIM, int VC, int CW>
 __global__ void __launch_bounds__(ScanSmem<DIM, VC, CW>::THREADS, 1)
-delta_chunk_scan(b200_delta_args p, int n_chunks, int vblocks) {
+delta_chunk_scan(const __grid_constant__ CUtensorMap map_q, const __grid_constant__ CUtensorMap map_k, const __grid_constant__ CUtensorMap map_v, b200_delta_args p,
+                 int n_chunks, int vblocks) {
   using M = ScanSmem<DIM, VC, CW>;
   constexpr int MT = DIM / 64, NT = CW / 8;  // 16-row state tiles per warp, 8-column tiles per warp
-  extern __shared__ __align__(128) uint8_t smem[];
+  extern __shared__ uint8_t smem_raw[];
+  __shared__ __align__(8) uint64_t full[M::STAGES];  // a stage's copies have landed
+  __shared__ volatile int aborted;
   const int warp = threadIdx.x >> 5, lane = threadIdx.x & 31, g8 = lane >> 2, t4 = lane & 3;
   const bool chain = warp < M::ROLE_WARPS;
   // row group, column group; every other four warps in reverse, so that a scheduler's warps share the triangles' work evenly
@@ -369,33 +381,36 @@ delta_chunk_scan(b200_delta_args p, int n_chunks, int vblocks) {
   const int64_t h = (blockIdx.x / vblocks) % p.heads, b = blockIdx.x / ((int64_t)vblocks * p.heads);
   const int64_t kv = h / (p.heads / p.kv_heads);
   const int c0 = vb * VC, dim = (int)p.dim, vdim = (int)p.vdim;
-  const uint32_t base = (uint32_t)__cvta_generic_to_shared(smem);
-  const uint32_t s_hi = base + 2 * M::STAGE, s_lo = s_hi + M::S_PART;
+  const uint32_t raw = (uint32_t)__cvta_generic_to_shared(smem_raw), base = (raw + 1023u) & ~1023u;
+  uint8_t* smem = smem_raw + (base - raw);
+  const uint32_t s_hi = base + M::STAGES * M::STAGE, s_lo = s_hi + M::S_PART;
   const uint32_t r_hi = s_lo + M::S_PART, r_lo = r_hi + M::V_TILE, u_hi = r_lo + M::V_TILE, u_lo = u_hi + M::V_TILE, w_hi = u_lo + M::V_TILE, w_lo = w_hi + M::V_TILE;
-  const auto* mixed = static_cast<const __nv_bfloat16*>(p.mixed) + b * p.n * p.ld_mixed;
   const uint8_t* records = static_cast<const uint8_t*>(p.workspace) + (b * n_chunks * p.heads + h) * (int64_t)kRecordBytes;
   const int64_t record_step = p.heads * (int64_t)kRecordBytes;
   const int i0 = rg * 16 + g8;  // this thread's tokens of a chunk: i0 and i0 + 8
 
-  // (by the output warps only: the chain has no cycles to spare)
-  const int loader = (int)threadIdx.x - 32 * M::ROLE_WARPS;
+  const uint32_t bar_full = (uint32_t)__cvta_generic_to_shared(full);
+  if (threadIdx.x == 0) {
+    for (int i = 0; i < M::STAGES; ++i) sm100::mbar_init(bar_full + 8 * i, 1);
+    aborted = 0;
+    asm volatile("fence.mbarrier_init.release.cluster;" ::: "memory");
+    sm100::fence_proxy_async_smem();
+  }
+  __syncthreads();
+  // one thread (rows behind the last token and columns beyond a head arrive as zeros)
   auto load_chunk = [&](int chunk, int stage) {
-    const uint32_t dst = base + stage * M::STAGE;
-    const int64_t t0 = (int64_t)chunk * kC;
-    const int n = (int)(p.n - t0 < kC ? p.n - t0 : kC);
-    const auto* src = mixed + t0 * p.ld_mixed;
-    load_tile<DIM>(dst, src + p.off_k + kv * dim, p.ld_mixed, n, dim, loader, 32 * M::ROLE_WARPS);
-    load_tile<DIM>(dst + M::TILE, src + kv * dim, p.ld_mixed, n, dim, loader, 32 * M::ROLE_WARPS);
-    for (int i = loader; i < kC * (VC / 8); i += 32 * M::ROLE_WARPS) {
-      const int r = i / (VC / 8), c = i % (VC / 8);
-      const bool ok = r < n && c0 + c * 8 < vdim;
-      const auto* v = src + p.off_v + h * vdim + c0;
-      cp_async16(dst + 2 * M::TILE + r * M::VP + c * 16, ok ? v + (int64_t)r * p.ld_mixed + c * 8 : mixed, ok);
+    const uint32_t dst = base + stage * M::STAGE, bar = bar_full + 8 * stage;
+    sm100::mbar_arrive_expect_tx(bar, M::TX_BYTES);
+#pragma unroll
+    for (int a = 0; a < DIM / 64; ++a) {
+      sm100::tma_load_4d(dst + a * M::ATOM, &map_k, bar, 64 * a, (int)kv, chunk * kC, (int)b);
+      sm100::tma_load_4d(dst + M::TILE + a * M::ATOM, &map_q, bar, 64 * a, (int)kv, chunk * kC, (int)b);
     }
-    const uint8_t* f = records + chunk * record_step + 2 * kFragBytes;
-    for (int i = loader; i < (kFactorBytes + 64) / 16; i += 32 * M::ROLE_WARPS) cp_async16(dst + 2 * M::TILE + M::V_TILE + i * 16, f + i * 16, true);
-    cp_async_commit();
+    sm100::tma_load_4d(dst + M::V_AT, &map_v, bar, c0, (int)h, chunk * kC, (int)b);
+    bulk_copy(dst + M::RECORD_AT, records + chunk * record_step, kRecordBytes, bar);
   };
+  // address of a 16-byte piece of a row of keys or queries
+  auto piece_at = [](uint32_t tile, int row, int piece) { return tile + (uint32_t)((piece >> 3) * M::ATOM) + swz<128>(row, piece & 7); };
   // accumulators (rows of 16, this warp's columns) as two bf16 parts into a row-major tile
   auto put = [&](uint32_t hi, uint32_t lo, int row, int nt, float a, float c) {
     uint32_t x, y;
@@ -408,13 +423,6 @@ delta_chunk_scan(b200_delta_args p, int n_chunks, int vblocks) {
   auto b_at = [&](int row, int np) {
     return (uint32_t)((row + (lane & 7) + ((lane >> 3) & 1) * 8) * M::VP + (cg * CW + np * 16 + (lane >> 4) * 8) * 2);
   };
-  // T (which = 0) or P (1) of this warp's rows
-  auto load_triangle = [&](int chunk, int which, uint4 (&hi)[4], uint4 (&lo)[4]) {
-    const uint4* frag = reinterpret_cast<const uint4*>(records + chunk * record_step + which * kFragBytes) + block_index(rg, 0) * 64 + lane;
-#pragma unroll
-    for (int kt = 0; kt < 4; ++kt)
-      if (kt <= rg) hi[kt] = __ldg(frag + kt * 64), lo[kt] = __ldg(frag + kt * 64 + 32);
-  };
   // acc = 64 token rows (this warp's 16) times the state in two parts
   auto times_state = [&](uint32_t tile, float (&acc)[NT][4]) {
 #pragma unroll
@@ -424,7 +432,7 @@ delta_chunk_scan(b200_delta_args p, int n_chunks, int vblocks) {
 #pragma unroll
     for (int ks = 0; ks < DIM / 16; ++ks) {
       uint32_t af[4];
-      ldsm4(af, tile + (uint32_t)((rg * 16 + (lane & 15)) * M::KP + (ks * 2 + (lane >> 4)) * 16));
+      ldsm4(af, piece_at(tile, rg * 16 + (lane & 15), ks * 2 + (lane >> 4)));
 #pragma unroll
       for (int np = 0; np < NT / 2; ++np) {
         uint32_t hi[4], lo[4];
@@ -438,12 +446,14 @@ delta_chunk_scan(b200_delta_args p, int n_chunks, int vblocks) {
       }
     }
   };
-  // acc += lhs (two parts, lower triangular) times a tile in two parts, for this warp's rows
-  auto triangular = [&](const uint4 (&ah)[4], const uint4 (&al)[4], uint32_t hi_tile, uint32_t lo_tile, float (&acc)[NT][4]) {
+  // acc += T (which = 0) or P (1) of the stage's record times a tile in two parts, for this warp's rows
+  auto triangular = [&](int stage, int which, uint32_t hi_tile, uint32_t lo_tile, float (&acc)[NT][4]) {
+    const uint4* frag = reinterpret_cast<const uint4*>(smem + stage * M::STAGE + M::RECORD_AT + which * kFragBytes) + block_index(rg, 0) * 64 + lane;
 #pragma unroll
     for (int kt = 0; kt < 4; ++kt) {
       if (kt <= rg) {
-        const uint32_t fh[4] = {ah[kt].x, ah[kt].y, ah[kt].z, ah[kt].w}, fl[4] = {al[kt].x, al[kt].y, al[kt].z, al[kt].w};
+        const uint4 ah = frag[kt * 64], al = frag[kt * 64 + 32];
+        const uint32_t fh[4] = {ah.x, ah.y, ah.z, ah.w}, fl[4] = {al.x, al.y, al.z, al.w};
 #pragma unroll
         for (int np = 0; np < NT / 2; ++np) {
           uint32_t hi[4], lo[4];
@@ -461,6 +471,7 @@ delta_chunk_scan(b200_delta_args p, int n_chunks, int vblocks) {
     }
   };
 
+  int stage = 0;
   if (chain) {
     // this warp's state: rows (rg * MT + mt) * 16 + {g8, g8 + 8}, columns cg * CW + nt * 8 + t4 * 2 + {0, 1} of the block's
     float st[MT][NT][4];
@@ -474,10 +485,7 @@ delta_chunk_scan(b200_delta_args p, int n_chunks, int vblocks) {
           const int r = (rg * MT + mt) * 16 + g8 + (e >> 1) * 8, c = c0 + cg * CW + nt * 8 + t4 * 2 + (e & 1);
           st[mt][nt][e] = !p.fresh && r < dim && c < vdim ? state[(int64_t)r * vdim + c] : 0.f;
         }
-    uint4 th[4], tl[4];
-    load_triangle(0, 0, th, tl);
-    for (int chunk = 0; chunk < n_chunks; ++chunk) {
-      const int stage = chunk & 1;
+    for (int chunk = 0; chunk < n_chunks; ++chunk, stage = stage + 1 == M::STAGES ? 0 : stage + 1) {
 #pragma unroll
       for (int mt = 0; mt < MT; ++mt)
 #pragma unroll
@@ -488,8 +496,8 @@ delta_chunk_scan(b200_delta_args p, int n_chunks, int vblocks) {
         }
       __syncthreads();  // (1) tiles and state parts are in place; everyone is done with the chunk before
       const uint32_t sk = base + stage * M::STAGE;
-      const uint8_t* sv = smem + stage * M::STAGE + 2 * M::TILE;
-      const float* factor = reinterpret_cast<const float*>(sv + M::V_TILE);
+      const uint8_t* sv = smem + stage * M::STAGE + M::V_AT;
+      const float* factor = reinterpret_cast<const float*>(smem + stage * M::STAGE + M::FACTOR_AT);
       // R = V - diag(G r_k) C_k S
       float r[NT][4];
       times_state(sk, r);
@@ -498,8 +506,8 @@ delta_chunk_scan(b200_delta_args p, int n_chunks, int vblocks) {
 #pragma unroll
         for (int nt = 0; nt < NT; ++nt) {
           const int c = cg * CW + nt * 8 + t4 * 2;
-          const float2 v0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sv + i0 * M::VP + c * 2));
-          const float2 v1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sv + (i0 + 8) * M::VP + c * 2));
+          const float2 v0 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sv + swz<128>(i0, c >> 3) + (c & 7) * 2));
+          const float2 v1 = __bfloat1622float2(*reinterpret_cast<const __nv_bfloat162*>(sv + swz<128>(i0 + 8, c >> 3) + (c & 7) * 2));
           put(r_hi, r_lo, i0, nt, fmaf(-g0, r[nt][0], v0.x), fmaf(-g0, r[nt][1], v0.y));
           put(r_hi, r_lo, i0 + 8, nt, fmaf(-g1, r[nt][2], v1.x), fmaf(-g1, r[nt][3], v1.y));
         }
@@ -510,8 +518,7 @@ delta_chunk_scan(b200_delta_args p, int n_chunks, int vblocks) {
       for (int i = 0; i < NT; ++i)
 #pragma unroll
         for (int e = 0; e < 4; ++e) r[i][e] = 0.f;
-      triangular(th, tl, r_hi, r_lo, r);
-      if (chunk + 1 < n_chunks) load_triangle(chunk + 1, 0, th, tl);
+      triangular(stage, 0, r_hi, r_lo, r);
       {
         const float f0 = factor[F_WRITE * kC + i0], f1 = factor[F_WRITE * kC + i0 + 8];
 #pragma unroll
@@ -536,7 +543,7 @@ delta_chunk_scan(b200_delta_args p, int n_chunks, int vblocks) {
         uint32_t kf[MT][4];
 #pragma unroll
         for (int mt = 0; mt < MT; ++mt)
-          ldsm4_trans(kf[mt], sk + (uint32_t)((kk * 16 + (lane & 7) + ((lane >> 4) << 3)) * M::KP + ((rg * MT + mt) * 16 + ((lane >> 3) & 1) * 8) * 2));
+          ldsm4_trans(kf[mt], piece_at(sk, kk * 16 + (lane & 7) + ((lane >> 4) << 3), (rg * MT + mt) * 2 + ((lane >> 3) & 1)));
 #pragma unroll
         for (int np = 0; np < NT / 2; ++np) {
           uint32_t hi[4], lo[4];
@@ -563,17 +570,17 @@ delta_chunk_scan(b200_delta_args p, int n_chunks, int vblocks) {
           if (r < dim && c < vdim) *reinterpret_cast<float2*>(state + (int64_t)r * vdim + c) = make_float2(st[mt][nt][e], st[mt][nt][e + 1]);
         }
   } else {
-    load_chunk(0, 0);
-    for (int chunk = 0; chunk < n_chunks; ++chunk) {
-      const int stage = chunk & 1;
+    const bool loads = warp == M::ROLE_WARPS && lane == 0;
+    if (loads)
+      for (int i = 0; i < M::STAGES - 1 && i < n_chunks; ++i) load_chunk(i, i);
+    for (int chunk = 0; chunk < n_chunks; ++chunk, stage = stage + 1 == M::STAGES ? 0 : stage + 1) {
       const int64_t t0 = (int64_t)chunk * kC;
       const int n = (int)(p.n - t0 < kC ? p.n - t0 : kC);
-      cp_async_wait<0>();
+      // (a copy that never lands would be reported through the status word; the barriers are kept up either way)
+      sm100::mbar_wait(bar_full + 8 * stage, (uint32_t)(chunk / M::STAGES) & 1, &aborted, p.status_word, 81);
       __syncthreads();  // (1)
-      if (chunk + 1 < n_chunks) load_chunk(chunk + 1, stage ^ 1);
-      uint4 ph[4], pl[4];
-      load_triangle(chunk, 1, ph, pl);
-      const float* factor = reinterpret_cast<const float*>(smem + stage * M::STAGE + 2 * M::TILE + M::V_TILE);
+      if (loads && chunk + M::STAGES - 1 < n_chunks) load_chunk(chunk + M::STAGES - 1, stage == 0 ? M::STAGES - 1 : stage - 1);
+      const float* factor = reinterpret_cast<const float*>(smem + stage * M::STAGE + M::FACTOR_AT);
       // O = diag(G r_q) C_q S + P U
       float o[NT][4];
       times_state(base + stage * M::STAGE + M::TILE, o);
@@ -582,7 +589,7 @@ delta_chunk_scan(b200_delta_args p, int n_chunks, int vblocks) {
       for (int nt = 0; nt < NT; ++nt) o[nt][0] *= q0, o[nt][1] *= q0, o[nt][2] *= q1, o[nt][3] *= q1;
       __syncthreads();  // (2)
       __syncthreads();  // (3)
-      triangular(ph, pl, u_hi, u_lo, o);
+      triangular(stage, 1, u_hi, u_lo, o);
 #pragma unroll
       for (int e = 0; e < 2; ++e) {
         const int i = i0 + e * 8;
@@ -595,6 +602,11 @@ delta_chunk_scan(b200_delta_args p, int n_chunks, int vblocks) {
           }
         }
       }
+    }
+  }
+  if (aborted) {  // give copies in flight time to land before the shared memory goes away
+    const long long t = clock64();
+    while (clock64() - t < 2000000LL) {
     }
   }
 }
@@ -676,7 +688,19 @@ int launch_scan(const b200_delta_args& p, int n_chunks, cudaStream_t stream) {
   static std::atomic<bool> done[kMaxDevices];
   if (!opt_in(delta_chunk_scan<DIM, VC, CW>, M::BYTES, done)) return B200_ERR_CUDA;
   const int vblocks = (int)((p.vdim + VC - 1) / VC);
-  delta_chunk_scan<DIM, VC, CW><<<(unsigned)(p.B * p.heads * vblocks), M::THREADS, M::BYTES, stream>>>(p, n_chunks, vblocks);
+  const auto* mixed = static_cast<const __nv_bfloat16*>(p.mixed);
+  CUtensorMap mq, mk, mv;
+  auto map = [&](CUtensorMap* m, const void* ptr, int64_t cols, int64_t heads) {
+    const uint64_t dims[4] = {(uint64_t)cols, (uint64_t)heads, (uint64_t)p.n, (uint64_t)p.B};
+    const uint64_t strides[3] = {(uint64_t)cols * 2, (uint64_t)p.ld_mixed * 2, (uint64_t)(p.n * p.ld_mixed) * 2};
+    const uint32_t box[4] = {64, 1, kC, 1};
+    return sm100::encode_tensor_map(m, ptr, 4, dims, strides, box, B200_BF16, CU_TENSOR_MAP_L2_PROMOTION_L2_256B);
+  };
+  int st = map(&mq, mixed, p.dim, p.kv_heads);
+  if (st == B200_OK) st = map(&mk, mixed + p.off_k, p.dim, p.kv_heads);
+  if (st == B200_OK) st = map(&mv, mixed + p.off_v, p.vdim, p.heads);
+  if (st != B200_OK) return st;
+  delta_chunk_scan<DIM, VC, CW><<<(unsigned)(p.B * p.heads * vblocks), M::THREADS, M::BYTES, stream>>>(mq, mk, mv, p, n_chunks, vblocks);
   note_launches(1);
   return status_from_cuda(cudaGetLastError());
 }

@@ -1033,7 +1033,7 @@ def gated_delta(rows, offsets, conv_w, a_log, dt_bias, norm_w, state, conv_state
     p.a_log, p.dt_bias, p.norm_w, p.state, p.pos_dev = a_log.data_ptr(), dt_bias.data_ptr(), norm_w.data_ptr(), state.data_ptr(), _ptr(pos)
     p.B, p.n, p.start, p.heads, p.kv_heads, p.dim, p.vdim = batch, M // batch, start, heads, kv_heads, dim, vdim
     p.eps, p.unit_eps, p.q_scale, p.dtype = eps, UNIT_EPS, q_scale, dtype_code(rows.dtype)
-    p.fresh = int(pos is None and start == 0)
+    p.fresh, p.status_word = int(pos is None and start == 0), _status_ptr(dev)
     lib = _lib.load()
     p.workspace_bytes = lib.b200_delta_workspace_bytes(ctypes.byref(p))
     ws = torch.empty((p.workspace_bytes,), device=dev, dtype=torch.uint8) if p.workspace_bytes else None

@@ -539,6 +539,7 @@ typedef struct {
   int fresh, dtype;
   void* workspace;
   int64_t workspace_bytes;
+  int* status_word;
 } b200_delta_args;
 int64_t b200_delta_workspace_bytes(const b200_delta_args* args);
 int b200_delta(const b200_delta_args* args, void* stream);
