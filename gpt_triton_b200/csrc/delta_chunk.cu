@@ -9,7 +9,7 @@
 // Every ratio of decays has j <= i: nothing overflows, whatever the decays.  c_q, c_k and v are bf16 and enter the MMAs as
 // they are; what is fp32 by definition (S, T, P, U and V - ...) enters as two bf16 parts (16 bits) and is accumulated in fp32.
 //
-//   delta_conv_kernel     convolution and silu, 16 tokens x 8 channels per thread
+//   delta_conv_kernel     convolution and silu, 32 tokens x 8 channels per thread
 //   delta_chunk_prepare   per (chunk, head), in parallel: gates, unit norms, A, its triangular inverse, P; T and P leave in
 //                         the register layout of the MMAs that read them
 //   delta_chunk_scan      per (sequence, head, column block): the chunks one after the other, S in registers
@@ -27,7 +27,7 @@ using namespace warp_mma;
 constexpr int kC = 64;  // tokens per chunk
 
 // ------------------------------------------------------------------ convolution and silu
-constexpr int kConvTokens = 16, kConvBatch = 8;  // tokens per thread, loads in flight
+constexpr int kConvTokens = 32, kConvBatch = 8;  // tokens per thread, loads in flight
 // a / (1 + exp(-a)) with one ex2 and one reciprocal
 __device__ __forceinline__ float silu_quick(float a) {
   float e, r;
